@@ -158,7 +158,7 @@ class CacheManager:
     def release_behind_window(self, request_id) -> int:
         """Give back the pages that no later query of the request can read.  The next query
         sits at position num_tokens and reads from num_tokens - window + 1 on, and from the start of
-        its own block of `chunk` positions on."""
+        its own block of `chunk` positions on; the pages of the first `keep` tokens stay."""
         rc = self.requests[request_id]
         freed = 0
         for need, pool, table in zip(self.layout.paged_groups, self.pools, rc.block_tables):
@@ -166,8 +166,9 @@ class CacheManager:
                 continue
             first_needed = first_needed_position(need, rc.num_tokens)
             dead_blocks = min(max(first_needed, 0) // self.page_size, len(table))
-            gone = [table[b] for b in range(dead_blocks) if table[b] >= 0]
-            for b in range(dead_blocks):
+            first_block = -(-(getattr(need, "keep", None) or 0) // self.page_size)     # the first tokens' pages stay
+            gone = [table[b] for b in range(first_block, dead_blocks) if table[b] >= 0]
+            for b in range(first_block, dead_blocks):
                 table[b] = -1
             pool.release(gone)
             freed += len(gone)

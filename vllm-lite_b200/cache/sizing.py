@@ -117,7 +117,8 @@ def pages_from_memory(layout: CacheLayout, page_size: int, itemsize: int, free_b
     for need in layout.paged_groups:
         most = per_request
         if need.window is not None:
-            most = min(most, -(-(need.window + (max_step_tokens or max_context)) // page_size) + 1)
+            most = min(most, -(-(need.window + (max_step_tokens or max_context)) // page_size) + 1
+                       + -(-(getattr(need, "keep", None) or 0) // page_size))
         if getattr(need, "chunk", None):
             most = min(most, -(-(need.chunk + (max_step_tokens or max_context)) // page_size) + 1)
         least.append(most)                                    # what one request alone may come to hold

@@ -14,7 +14,8 @@
 // multiplies head h's output for token t by sigmoid(gate[t * gate_stride + h]).  Weighting ATT_SIGMOID replaces the
 // softmax: every visible key weighs sigmoid(s_j + head_bias[h]) by itself and nothing is divided by a sum.
 // `softcap` > 0 bounds a score, s <- softcap tanh(s / softcap); `dist_a`, `dist_b` (a number per query head each) then take
-// dist_a[h] ln(1 + dist_b[h] (i - j)) off the score of a key that lies i - j positions back.
+// dist_a[h] ln(1 + dist_b[h] (i - j)) off the score of a key that lies i - j positions back.  `keep` > 0: a query also reads
+// the request's first `keep` keys, however far behind its window they lie.
 //
 // vl_paged_attention: one block per (token, query head), 16 groups of 8 lanes.
 // Group g owns the keys whose position is g modulo 16 and keeps a running
@@ -50,7 +51,7 @@ paged_attention_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
                        int nq, int nkv, int page_size, int num_pages, float scale, int window,
                        const float* __restrict__ sinks, int chunk, const float* __restrict__ head_bias,
                        const T* __restrict__ gate, int gate_stride, float softcap,
-                       const float* __restrict__ dist_a, const float* __restrict__ dist_b, unsigned* err) {
+                       const float* __restrict__ dist_a, const float* __restrict__ dist_b, int keep, unsigned* err) {
     constexpr int HD = R * 16;
     __shared__ float s_acc[ATT_GROUPS][HD];
     __shared__ float s_m[ATT_GROUPS], s_l[ATT_GROUPS];
@@ -76,9 +77,11 @@ paged_attention_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ ou
     }
     float m = -INFINITY, lsum = 0.f;
 
-    for (int jb = (lo / ATT_GROUPS) * ATT_GROUPS; jb <= pos; jb += ATT_GROUPS) {
+    const int lo_jb = (lo / ATT_GROUPS) * ATT_GROUPS, kept = min(keep, lo);       // kept keys before the window
+    for (int jb = kept > 0 ? 0 : lo_jb; jb <= pos; jb += ATT_GROUPS) {
+        if (jb >= kept && jb < lo_jb) jb = lo_jb;                 // past the kept keys: on to the window
         const int j = jb + g;
-        bool valid = (j >= lo) && (j <= pos);
+        bool valid = (j >= lo || j < kept) && (j <= pos);
         size_t base = 0;
         if (valid) {
             const int blk = j / page_size;
@@ -176,17 +179,17 @@ static int launch_paged_attention(int R, dim3 grid, cudaStream_t s, const T* q, 
                                   const int* req, const int* pos, int nq, int nkv, int page_size,
                                   int num_pages, float scale, int window, const float* sinks, int mode, int chunk,
                                   const float* head_bias, const T* gate, int gate_stride, float softcap,
-                                  const float* dist_a, const float* dist_b, unsigned* err) {
+                                  const float* dist_a, const float* dist_b, int keep, unsigned* err) {
 #define ATT_CASE(RR)                                                                              \
     case RR:                                                                                      \
         if (mode == ATT_SIGMOID)                                                                  \
             paged_attention_kernel<T, RR, ATT_SIGMOID><<<grid, ATT_THREADS, 0, s>>>(              \
                 q, q_stride, out, kc, vc, bt, max_blocks, req, pos, nq, nkv, page_size, num_pages,\
-                scale, window, sinks, chunk, head_bias, gate, gate_stride, softcap, dist_a, dist_b, err);                \
+                scale, window, sinks, chunk, head_bias, gate, gate_stride, softcap, dist_a, dist_b, keep, err);          \
         else                                                                                      \
             paged_attention_kernel<T, RR, ATT_SOFTMAX><<<grid, ATT_THREADS, 0, s>>>(              \
                 q, q_stride, out, kc, vc, bt, max_blocks, req, pos, nq, nkv, page_size, num_pages,\
-                scale, window, sinks, chunk, head_bias, gate, gate_stride, softcap, dist_a, dist_b, err);                \
+                scale, window, sinks, chunk, head_bias, gate, gate_stride, softcap, dist_a, dist_b, keep, err);          \
         break;
     switch (R) {
         ATT_CASE(1) ATT_CASE(2) ATT_CASE(3) ATT_CASE(4) ATT_CASE(5) ATT_CASE(6) ATT_CASE(7) ATT_CASE(8)
@@ -204,8 +207,9 @@ extern "C" int vl_paged_attention(const void* q, int q_stride, void* out, int dt
                                   int T, int nq, int nkv, int hd, int page_size, int num_pages,
                                   float scale, int window, const float* sinks, int mode, int chunk,
                                   const float* head_bias, const void* gate, int gate_stride, float softcap,
-                                  const float* dist_a, const float* dist_b, unsigned* err, void* stream) {
+                                  const float* dist_a, const float* dist_b, int keep, unsigned* err, void* stream) {
     if (T <= 0) return VL_OK;
+    if (keep < 0 || (keep > 0 && chunk > 0)) return VL_ERR_ARGUMENT;
     if ((dist_a == nullptr) != (dist_b == nullptr) || softcap < 0.f) return VL_ERR_ARGUMENT;
     if (hd <= 0 || hd % 16 || hd > ATT_MAX_HD) return VL_ERR_UNSUPPORTED;
     if (nq <= 0 || nkv <= 0 || nq % nkv || page_size <= 0 || max_blocks <= 0) return VL_ERR_ARGUMENT;
@@ -219,13 +223,13 @@ extern "C" int vl_paged_attention(const void* q, int q_stride, void* out, int dt
                                              (const float*)kcache, (const float*)vcache, block_table,
                                              max_blocks, req_index, positions, nq, nkv, page_size,
                                              num_pages, scale, window, sinks, mode, chunk, head_bias,
-                                             (const float*)gate, gate_stride, softcap, dist_a, dist_b, err);
+                                             (const float*)gate, gate_stride, softcap, dist_a, dist_b, keep, err);
     if (dtype == VL_BF16)
         return launch_paged_attention<bf16>(hd / 16, grid, s, (const bf16*)q, q_stride, (bf16*)out,
                                             (const bf16*)kcache, (const bf16*)vcache, block_table,
                                             max_blocks, req_index, positions, nq, nkv, page_size,
                                             num_pages, scale, window, sinks, mode, chunk, head_bias,
-                                            (const bf16*)gate, gate_stride, softcap, dist_a, dist_b, err);
+                                            (const bf16*)gate, gate_stride, softcap, dist_a, dist_b, keep, err);
     return VL_ERR_UNSUPPORTED;
 }
 

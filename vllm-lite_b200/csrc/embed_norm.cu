@@ -26,6 +26,56 @@ __global__ void embed_kernel(const int* __restrict__ ids, const TW* __restrict__
     for (int i = threadIdx.x; i < H; i += blockDim.x) row[i] = to_f32(src[i]) * scale;   // float32; times 1 is exact
 }
 
+// The same with a row of a second table added, hashed from the token before and this one:
+//   x[t] = table[id_t] * scale + pairs[(id_(t-1) mul_prev + id_t mul_cur) mod buckets],  row `buckets` at position 0.
+// The token before a portion's first one is the request's state (an int32 per slot), which the block of that token replaces
+// by the portion's last token; no other block touches it.  A row at a negative position (padding of a replayed step) is
+// zero and touches no state.
+template <typename TW>
+__global__ void embed_pair_kernel(const int* __restrict__ ids, const TW* __restrict__ table, const TW* __restrict__ pairs,
+                                  float* __restrict__ x, int H, int V, float scale, int buckets, long long mul_prev,
+                                  long long mul_cur, int* state, long long state_stride, const int* __restrict__ cu,
+                                  const int* __restrict__ slots, const int* __restrict__ req_index,
+                                  const int* __restrict__ positions, unsigned* err) {
+    __shared__ int s_prev;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, pos = positions[t], id = ids[t];
+    float* row = x + (size_t)t * H;
+    if (pos < 0) {
+        for (int i = threadIdx.x; i < H; i += blockDim.x) row[i] = 0.f;
+        return;
+    }
+    if (threadIdx.x == 0) {
+        const int b = req_index[t], first = cu[b];
+        int prev = t > first ? ids[t - 1] : 0;
+        if (t == first) {
+            int* st = state + (long long)slots[b] * state_stride;
+            prev = *st;
+            *st = ids[cu[b + 1] - 1];
+        }
+        s_prev = prev;
+    }
+    __syncthreads();
+    if (id < 0 || id >= V) {
+        if (threadIdx.x == 0) atomicOr(err, VL_DEV_BAD_TOKEN);
+        for (int i = threadIdx.x; i < H; i += blockDim.x) row[i] = 0.f;
+        return;
+    }
+    const int prev = min(max(s_prev, 0), V - 1);         // (a token before that was refused was flagged at its own place)
+    const long long at = pos == 0 ? buckets : (prev * mul_prev + id * mul_cur) % buckets;
+    const TW* src = table + (size_t)id * H;
+    const TW* add = pairs + (size_t)at * H;
+    if ((H & 3) == 0) {
+        for (int i = 4 * threadIdx.x; i < H; i += 4 * blockDim.x) {
+            const float4 a = Quad<TW>::load(src + i), b = Quad<TW>::load(add + i);
+            Quad<float>::store(row + i, make_float4(a.x * scale + b.x, a.y * scale + b.y, a.z * scale + b.z, a.w * scale + b.w));
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < H; i += blockDim.x) row[i] = to_f32(src[i]) * scale + to_f32(add[i]);
+}
+
 // rows == nullptr: row r of the output is row r of x (and x is updated in place
 // when delta is given).  rows != nullptr: output row r is made from x[rows[r]]
 // (+ delta[rows[r]]) and x is left untouched.
@@ -266,35 +316,51 @@ extern "C" int vl_layernorm_rows(const float* x, const int* rows, const float* w
 // the activation dtype: the next sub-layer's input.  `bias` (or null): a vector added to every row of y first, in float32
 // (the bias of the product that made y, left to this kernel).  The row of y is kept in registers where it fits (H a multiple of
 // 4, at most 256 * 4 * VPT values), else read twice.  The order of the sums depends on the row length alone.
+// With a second row y2 the normed row is s1 * y + s2 * y2, or, given weights w1 and w2, s1 * n(y) w1 + s2 * n(y2) w2 with
+// n(y) = y / sqrt(mean(y^2) + eps): two sub-layers side by side, each normed by itself before they are added.
 template <typename TA>
 __global__ void __launch_bounds__(256)
 rmsnorm_add_kernel(const TA* __restrict__ y, const float* __restrict__ bias, const float* __restrict__ w, float eps, float mult,
-                   float* __restrict__ x, TA* __restrict__ cast, int H, const TA* __restrict__ y2, float s1, float s2) {
+                   float* __restrict__ x, TA* __restrict__ cast, int H, const TA* __restrict__ y2, float s1, float s2,
+                   const float* __restrict__ w1, const float* __restrict__ w2) {
     __shared__ float scratch[32];
     pdl_launch_dependents();
     pdl_wait();
     const int r = blockIdx.x;
     const TA* yr = y + (size_t)r * H;
     const TA* y2r = y2 ? y2 + (size_t)r * H : nullptr;          // the normed row is s1 * y + s2 * y2 (two sub-layers side by side)
+    float f1 = s1, f2 = s2;
+    if (w1) {                                                    // ... each normed by itself first
+        float sa = 0.f, sb = 0.f;
+        for (int i = threadIdx.x; i < H; i += 256) { const float u = to_f32(yr[i]), v = to_f32(y2r[i]); sa += u * u; sb += v * v; }
+        f1 = s1 / sqrtf(block_sum<256>(sa, scratch) / (float)H + eps);
+        f2 = s2 / sqrtf(block_sum<256>(sb, scratch) / (float)H + eps);
+    }
+    auto row = [&](int i) {
+        float d = to_f32(yr[i]);
+        if (y2r) d = w1 ? f1 * d * w1[i] + f2 * to_f32(y2r[i]) * w2[i] : s1 * d + s2 * to_f32(y2r[i]);
+        return d + (bias ? bias[i] : 0.f);
+    };
     float ss = 0.f;
     for (int i = threadIdx.x; i < H; i += 256) {
-        const float d = (y2r ? s1 * to_f32(yr[i]) + s2 * to_f32(y2r[i]) : to_f32(yr[i])) + (bias ? bias[i] : 0.f);
+        const float d = row(i);
         ss += d * d;
     }
     const float inv = 1.0f / sqrtf(block_sum<256>(ss, scratch) / (float)H + eps);
     float* xr = x + (size_t)r * H;
     for (int i = threadIdx.x; i < H; i += 256) {
-        const float d = (y2r ? s1 * to_f32(yr[i]) + s2 * to_f32(y2r[i]) : to_f32(yr[i])) + (bias ? bias[i] : 0.f);
+        const float d = row(i);
         const float v = xr[i] + mult * (d * inv * w[i]);
         xr[i] = v;
         if (cast) cast[(size_t)r * H + i] = from_f32<TA>(v);
     }
 }
 
-template <typename TA, int VPT>
+template <typename TA, int VPT, bool NORMED>
 __global__ void __launch_bounds__(256)
 rmsnorm_add_vec_kernel(const TA* __restrict__ y, const float* __restrict__ bias, const float* __restrict__ w, float eps, float mult,
-                       float* __restrict__ x, TA* __restrict__ cast, int H, const TA* __restrict__ y2, float s1, float s2) {
+                       float* __restrict__ x, TA* __restrict__ cast, int H, const TA* __restrict__ y2, float s1, float s2,
+                   const float* __restrict__ w1, const float* __restrict__ w2) {
     __shared__ float scratch[32];
     pdl_launch_dependents();
     pdl_wait();
@@ -303,6 +369,36 @@ rmsnorm_add_vec_kernel(const TA* __restrict__ y, const float* __restrict__ bias,
     const TA* y2r = y2 ? y2 + (size_t)r * H : nullptr;          // the normed row is s1 * y + s2 * y2
     float4 v[VPT];
     float ss = 0.f;
+    if constexpr (NORMED) {                                      // both normed by themselves first (a kernel of its own: it holds two rows)
+        float4 u[VPT];
+        float sa = 0.f, sb = 0.f;
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) {
+            const int c = threadIdx.x + 256 * i;
+            if (c < H4) {
+                v[i] = Quad<TA>::load(yr + 4 * c);
+                u[i] = Quad<TA>::load(y2r + 4 * c);
+                sa += v[i].x * v[i].x; sa += v[i].y * v[i].y; sa += v[i].z * v[i].z; sa += v[i].w * v[i].w;
+                sb += u[i].x * u[i].x; sb += u[i].y * u[i].y; sb += u[i].z * u[i].z; sb += u[i].w * u[i].w;
+            }
+        }
+        const float f1 = s1 / sqrtf(block_sum<256>(sa, scratch) / (float)H + eps);
+        const float f2 = s2 / sqrtf(block_sum<256>(sb, scratch) / (float)H + eps);
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) {
+            const int c = threadIdx.x + 256 * i;
+            if (c < H4) {
+                const float4 g1 = Quad<float>::load(w1 + 4 * c), g2 = Quad<float>::load(w2 + 4 * c);
+                v[i].x = f1 * v[i].x * g1.x + f2 * u[i].x * g2.x; v[i].y = f1 * v[i].y * g1.y + f2 * u[i].y * g2.y;
+                v[i].z = f1 * v[i].z * g1.z + f2 * u[i].z * g2.z; v[i].w = f1 * v[i].w * g1.w + f2 * u[i].w * g2.w;
+                if (bias) {
+                    const float4 b = Quad<float>::load(bias + 4 * c);
+                    v[i].x += b.x; v[i].y += b.y; v[i].z += b.z; v[i].w += b.w;
+                }
+                ss += v[i].x * v[i].x; ss += v[i].y * v[i].y; ss += v[i].z * v[i].z; ss += v[i].w * v[i].w;
+            }
+        }
+    } else {
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
         const int c = threadIdx.x + 256 * i;
@@ -319,6 +415,7 @@ rmsnorm_add_vec_kernel(const TA* __restrict__ y, const float* __restrict__ bias,
             }
             ss += v[i].x * v[i].x; ss += v[i].y * v[i].y; ss += v[i].z * v[i].z; ss += v[i].w * v[i].w;
         }
+    }
     }
     const float inv = 1.0f / sqrtf(block_sum<256>(ss, scratch) / (float)H + eps);
     float* xr = x + (size_t)r * H;
@@ -338,22 +435,26 @@ rmsnorm_add_vec_kernel(const TA* __restrict__ y, const float* __restrict__ bias,
 
 template <typename TA>
 static int launch_rmsnorm_add(const TA* y, const float* bias, const float* w, float eps, float mult, float* x, TA* cast, int R, int H,
-                              const TA* y2, float s1, float s2, cudaStream_t s) {
+                              const TA* y2, float s1, float s2, const float* w1, const float* w2, cudaStream_t s) {
     const int pieces = (H / 4 + 255) / 256;
-    if (H % 4 == 0 && pieces <= 1) return vl_launch(rmsnorm_add_vec_kernel<TA, 1>, dim3(R), dim3(256), 0, s, y, bias, w, eps, mult, x, cast, H, y2, s1, s2);
-    if (H % 4 == 0 && pieces <= 2) return vl_launch(rmsnorm_add_vec_kernel<TA, 2>, dim3(R), dim3(256), 0, s, y, bias, w, eps, mult, x, cast, H, y2, s1, s2);
-    if (H % 4 == 0 && pieces <= 4) return vl_launch(rmsnorm_add_vec_kernel<TA, 4>, dim3(R), dim3(256), 0, s, y, bias, w, eps, mult, x, cast, H, y2, s1, s2);
-    if (H % 4 == 0 && pieces <= 8) return vl_launch(rmsnorm_add_vec_kernel<TA, 8>, dim3(R), dim3(256), 0, s, y, bias, w, eps, mult, x, cast, H, y2, s1, s2);
-    return vl_launch(rmsnorm_add_kernel<TA>, dim3(R), dim3(256), 0, s, y, bias, w, eps, mult, x, cast, H, y2, s1, s2);
+#define RMS_ADD(VPT)                                                                                                                      \
+    return w1 ? vl_launch(rmsnorm_add_vec_kernel<TA, VPT, true>, dim3(R), dim3(256), 0, s, y, bias, w, eps, mult, x, cast, H, y2, s1, s2, w1, w2) \
+              : vl_launch(rmsnorm_add_vec_kernel<TA, VPT, false>, dim3(R), dim3(256), 0, s, y, bias, w, eps, mult, x, cast, H, y2, s1, s2, w1, w2)
+    if (H % 4 == 0 && pieces <= 1) RMS_ADD(1);
+    if (H % 4 == 0 && pieces <= 2) RMS_ADD(2);
+    if (H % 4 == 0 && pieces <= 4) RMS_ADD(4);
+    if (H % 4 == 0 && pieces <= 8) RMS_ADD(8);
+#undef RMS_ADD
+    return vl_launch(rmsnorm_add_kernel<TA>, dim3(R), dim3(256), 0, s, y, bias, w, eps, mult, x, cast, H, y2, s1, s2, w1, w2);
 }
 
 extern "C" int vl_rmsnorm_add(const void* y, int act_dtype, const float* bias, const float* w, float eps, float mult, float* x, void* cast,
-                              int R, int H, const void* y2, float s1, float s2, void* stream) {
+                              int R, int H, const void* y2, float s1, float s2, const float* w1, const float* w2, void* stream) {
     if (R <= 0) return VL_OK;
-    if (H <= 0) return VL_ERR_ARGUMENT;
+    if (H <= 0 || (w1 == nullptr) != (w2 == nullptr) || (w1 && !y2)) return VL_ERR_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
-    if (act_dtype == VL_F32) return launch_rmsnorm_add<float>((const float*)y, bias, w, eps, mult, x, (float*)cast, R, H, (const float*)y2, s1, s2, s);
-    if (act_dtype == VL_BF16) return launch_rmsnorm_add<bf16>((const bf16*)y, bias, w, eps, mult, x, (bf16*)cast, R, H, (const bf16*)y2, s1, s2, s);
+    if (act_dtype == VL_F32) return launch_rmsnorm_add<float>((const float*)y, bias, w, eps, mult, x, (float*)cast, R, H, (const float*)y2, s1, s2, w1, w2, s);
+    if (act_dtype == VL_BF16) return launch_rmsnorm_add<bf16>((const bf16*)y, bias, w, eps, mult, x, (bf16*)cast, R, H, (const bf16*)y2, s1, s2, w1, w2, s);
     return VL_ERR_UNSUPPORTED;
 }
 
@@ -368,6 +469,23 @@ extern "C" int vl_embed(const int* ids, const void* table, int table_dtype, floa
     else
         return VL_ERR_UNSUPPORTED;
     return vl_launch_status();
+}
+
+extern "C" int vl_embed_pair(const int* ids, const void* table, const void* pairs, int table_dtype, float* x, int T, int H, int V,
+                             float scale, int buckets, long long mul_prev, long long mul_cur, int* state, long long state_stride,
+                             const int* cu, const int* slots, const int* req_index, const int* positions, unsigned* err, void* stream) {
+    if (T <= 0) return VL_OK;
+    if (H <= 0 || V <= 0 || buckets <= 0 || mul_prev < 0 || mul_cur < 0 || mul_prev > 0x7fffffff || mul_cur > 0x7fffffff || state_stride < 1)
+        return VL_ERR_ARGUMENT;
+    if ((((uintptr_t)table | (uintptr_t)pairs | (uintptr_t)x) & 15)) return VL_ERR_ARGUMENT;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (table_dtype == VL_F32)
+        return vl_launch(embed_pair_kernel<float>, dim3(T), dim3(256), 0, s, ids, (const float*)table, (const float*)pairs, x, H, V, scale,
+                         buckets, mul_prev, mul_cur, state, state_stride, cu, slots, req_index, positions, err);
+    if (table_dtype == VL_BF16)
+        return vl_launch(embed_pair_kernel<bf16>, dim3(T), dim3(256), 0, s, ids, (const bf16*)table, (const bf16*)pairs, x, H, V, scale,
+                         buckets, mul_prev, mul_cur, state, state_stride, cu, slots, req_index, positions, err);
+    return VL_ERR_UNSUPPORTED;
 }
 
 extern "C" int vl_add_rmsnorm(float* x, const void* delta, const int* rows, const float* w, void* out,

@@ -23,6 +23,9 @@
 // block; `gate` multiplies head h's output for token t by sigmoid(gate[t * gate_stride + h]); the weighting SIG
 // replaces the softmax: a visible key weighs sigmoid(s_j + head_bias[h]) by itself, nothing is divided by a sum, and
 // partial results of chunks and warps simply add up (they travel with a maximum of 0, so every merge weighs them 1).
+// `keep` > 0: a query also reads the request's first `keep` keys, however far behind its window they lie.  The prefill
+// kernel walks the tiles of the kept keys before those of the window; the decode kernel numbers the keys that a token reads
+// (the kept ones first, then its window) and cuts that number into chunks.
 // Rows of shared-memory tiles are padded by 16 bytes, which makes every 8-row ldmatrix access
 // hit 8 different banks groups for any head size.
 #include "score_shape.cuh"
@@ -82,6 +85,7 @@ struct AttnOptions {
     const bf16* gate; int gate_stride;                   // a gate logit per (token of the step, head), or null
     float cap_l2;                                        // a bound on the scores, times log2 e (0: none): s <- cap tanh(s / cap)
     const float* dist_a; const float* dist_b;            // per query head (or null): a ln(1 + b (i - j)) is taken off the score
+    int keep;                                            // first keys of a request that every query reads (0: none)
 };
 __device__ __forceinline__ float gate_factor(const AttnOptions& op, int tok, int h) {
     return op.gate ? 1.f / (1.f + __expf(-__bfloat162float(op.gate[(size_t)tok * op.gate_stride + h]))) : 1.f;
@@ -94,9 +98,10 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 // Row of the cache ([pages, nkv, page_size, HD] seen as rows of HD) that holds position j of the
 // request, or -1 when j lies outside [first, last] (such rows are filled with zeros and never looked
 // up: their pages may not exist, or may have been given back once a window passed them).
+// Keys before `kept` are looked up too.
 __device__ __forceinline__ int cache_row(const int* table, int max_blocks, int j, int first, int last, int kvh,
-                                         int nkv, int page_size, int num_pages, unsigned* err) {
-    if (j < first || j > last) return -1;
+                                         int nkv, int page_size, int num_pages, unsigned* err, int kept = 0) {
+    if ((j < first && j >= kept) || j > last) return -1;
     const int blk = j / page_size;
     const int page = blk < max_blocks ? table[blk] : -1;
     if (page < 0 || page >= num_pages) {
@@ -157,7 +162,10 @@ flash_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
     int lo = (window > 0 && pos0 - window + 1 > 0) ? pos0 - window + 1 : 0;
     if (op.block > 0) lo = max(lo, pos0 / op.block * op.block);  // the first row's block starts first
     const int blk_hi = op.block > 0 ? hi / op.block * op.block : 0;     // where the last row's block starts
-    const int kt_lo = lo / BN, kt_hi = hi / BN;
+    // tiles in the order of their walk: those of the kept keys that lie before the window's first tile, then the window's
+    const int kt_win = lo / BN, nkeep = min((min(op.keep, lo) + BN - 1) / BN, kt_win);
+    const int kt_lo = 0, kt_hi = hi / BN - kt_win + nkeep;
+    auto tile_of = [&](int i) { return i < nkeep ? i : kt_win + i - nkeep; };
 
     for (int idx = tid; idx < BM * CPR; idx += NTHREADS) {       // the query tile (rows beyond count: zeros)
         const int r = idx / CPR, c = idx - r * CPR;
@@ -166,8 +174,8 @@ flash_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
         cp_async16(Qs + (size_t)r * LDS + c * 8, src, valid);
     }
     if (tid < BN) {
-        s_rows[0][tid] = cache_row(table, max_blocks, kt_lo * BN + tid, lo, hi, kvh, nkv, page_size, num_pages, err);
-        s_rows[1][tid] = cache_row(table, max_blocks, (kt_lo + 1) * BN + tid, lo, hi, kvh, nkv, page_size, num_pages, err);
+        s_rows[0][tid] = cache_row(table, max_blocks, tile_of(0) * BN + tid, lo, hi, kvh, nkv, page_size, num_pages, err, op.keep);
+        s_rows[1][tid] = cache_row(table, max_blocks, tile_of(1) * BN + tid, lo, hi, kvh, nkv, page_size, num_pages, err, op.keep);
     }
     __syncthreads();
     load_kv_tiles(Ks, Vs, kcache, vcache, s_rows[0], BN);
@@ -186,9 +194,10 @@ flash_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
     const float sl2 = shaped ? 1.f : scale_log2;                 // shaped scores are in units of log2 already
     const float toc = two_over_cap(op.cap_l2), da = op.dist_a ? op.dist_a[h] : 0.f, db = op.dist_a ? op.dist_b[h] : 0.f;
 
-    for (int kt = kt_lo; kt <= kt_hi; ++kt) {
-        const int buf = (kt - kt_lo) & 1;
-        if (kt + 1 <= kt_hi) {
+    for (int it = kt_lo; it <= kt_hi; ++it) {
+        const int kt = tile_of(it);
+        const int buf = (it - kt_lo) & 1;
+        if (it + 1 <= kt_hi) {
             load_kv_tiles(Ks + (buf ^ 1) * BN * LDS, Vs + (buf ^ 1) * BN * LDS, kcache, vcache, s_rows[buf ^ 1], BN);
             cp_async_commit();
             cp_async_wait<1>();
@@ -196,10 +205,10 @@ flash_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
             cp_async_wait<0>();
         }
         __syncthreads();
-        // rows of tile kt + 2 (read after the barrier that ends this round; slot `buf` is no longer in use)
-        if (tid < BN && kt + 2 <= kt_hi)
-            s_rows[buf][tid] = cache_row(table, max_blocks, (kt + 2) * BN + tid, lo, hi, kvh, nkv, page_size, num_pages, err);
-        if (kt == kt_lo) {
+        // rows of the tile after the next (read after the barrier that ends this round; slot `buf` is no longer in use)
+        if (tid < BN && it + 2 <= kt_hi)
+            s_rows[buf][tid] = cache_row(table, max_blocks, tile_of(it + 2) * BN + tid, lo, hi, kvh, nkv, page_size, num_pages, err, op.keep);
+        if (it == kt_lo) {
 #pragma unroll
             for (int ks = 0; ks < KSTEPS; ++ks)
                 ldmatrix_x4(qf[ks], Qs + (size_t)(row0 + (lane & 7) + 8 * ((lane >> 3) & 1)) * LDS + ks * 16 + 8 * (lane >> 4));
@@ -241,7 +250,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict_
                     const int j = j_base + n * 8 + (e & 1);
                     const int p = (e < 2) ? pos_a : pos_b;
                     const bool rv = (e < 2) ? row_a : row_b;
-                    if (!rv || j > p || (window > 0 && j <= p - window) || j < ((e < 2) ? blk_a : blk_b)) s[n][e] = -INFINITY;
+                    if (!rv || j > p || (window > 0 && j <= p - window && j >= op.keep) || j < ((e < 2) ? blk_a : blk_b)) s[n][e] = -INFINITY;
                 }
             }
         }
@@ -348,8 +357,9 @@ extern "C" int vl_flash_prefill(const void* q, int q_stride, void* out, const vo
                                 int nq, int nkv, int hd, int page_size, int num_pages, float scale, int window,
                                 unsigned* err, const float* sinks, int weighting, int block, const float* head_bias,
                                 const void* gate, int gate_stride, float softcap, const float* dist_a, const float* dist_b,
-                                void* stream) {
+                                int keep, void* stream) {
     if (num_tiles <= 0) return VL_OK;
+    if (keep < 0 || (keep > 0 && block > 0)) return VL_ERR_ARGUMENT;
     if (softcap < 0.f || (dist_a == nullptr) != (dist_b == nullptr)) return VL_ERR_ARGUMENT;
     if (hd != HD) return VL_ERR_UNSUPPORTED;
     if (nq <= 0 || nkv <= 0 || nq % nkv || page_size <= 0 || max_blocks <= 0 || q_stride % 8) return VL_ERR_ARGUMENT;
@@ -362,7 +372,7 @@ extern "C" int vl_flash_prefill(const void* q, int q_stride, void* out, const vo
     auto kernel = weighting == 1 ? flash_prefill_kernel<true> : flash_prefill_kernel<false>;
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    const AttnOptions op = {weighting, block, head_bias, (const bf16*)gate, gate_stride, softcap * 1.4426950408889634f, dist_a, dist_b};
+    const AttnOptions op = {weighting, block, head_bias, (const bf16*)gate, gate_stride, softcap * 1.4426950408889634f, dist_a, dist_b, keep};
     kernel<<<dim3(nq, num_tiles * parts), NTHREADS, smem, (cudaStream_t)stream>>>(
         (const bf16*)q, q_stride, (bf16*)out, (const bf16*)kcache, (const bf16*)vcache, block_table, max_blocks,
         (const int4*)tiles, parts, nq, nkv, page_size, num_pages, scale * 1.4426950408889634f, window, err, sinks, op);
@@ -504,6 +514,12 @@ flash_decode_kernel(const bf16* __restrict__ q, int q_stride,
     const int nvalid = min(DEC_ROWS, grp - htile * DEC_ROWS);
     int pos = positions[tok];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    if (fz.op.block > 0 && pos >= 0) lo = max(lo, pos / fz.op.block * fz.op.block);
+    // With kept keys the launch works on the number of a key among those the token reads, not on its position: key v is
+    // position v for v < kept and position v + gap behind them (gap = 0 without the option: number and position are one).
+    const int kept = fz.op.keep > 0 ? min(fz.op.keep, lo) : 0, gap = fz.op.keep > 0 ? lo - kept : 0;
+    if (fz.op.keep > 0) { lo = 0; pos -= gap; }
     if ((long long)pos >= (long long)S * chunk) {                // beyond the S chunks the launch was sized for:
         if (tid == 0 && split == 0 && err) atomicOr(err, VL_DEV_BEYOND_BOUND);   // flagged and served like an empty place
         pos = -1;
@@ -516,8 +532,6 @@ flash_decode_kernel(const bf16* __restrict__ q, int q_stride,
         }
         return;
     }
-    int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
-    if (fz.op.block > 0) lo = max(lo, pos / fz.op.block * fz.op.block);
     auto finish = [&](float M, float L, int h) { return decode_finish<SIG>(fz, M, L, tok, h); };
     const int c0 = max(split * chunk, lo);
     const int c1 = min((split + 1) * chunk, pos + 1);
@@ -535,8 +549,10 @@ flash_decode_kernel(const bf16* __restrict__ q, int q_stride,
     const int* table = block_table + (size_t)req_index[tok] * max_blocks;
     const int st0 = c0 / BN, st1 = (c1 - 1) / BN;
 
-    for (int i = tid; i < (st1 - st0 + 1) * BN; i += NTHREADS)
-        s_rows[i] = cache_row(table, max_blocks, st0 * BN + i, c0, pos, kvh, nkv, page_size, num_pages, err);
+    for (int i = tid; i < (st1 - st0 + 1) * BN; i += NTHREADS) {
+        const int v = st0 * BN + i;                              // a key outside [c0, pos] is not looked up
+        s_rows[i] = v < c0 || v > pos ? -1 : cache_row(table, max_blocks, v < kept ? v : v + gap, 0, pos + gap, kvh, nkv, page_size, num_pages, err);
+    }
     // (c0 <= pos always) this chunk holds the token's own position, and this call owns the cache (a call that
     // reads another call's cache finds the token's key there: the owner ran before it)
     const bool has_new = fz.on && fz.slots && pos < c1;
@@ -673,11 +689,13 @@ flash_decode_kernel(const bf16* __restrict__ q, int q_stride,
             }
             const int j0 = st * BN + warp * 16 + g;              // this lane's keys: j0 and j0 + 8
             const bool in0 = j0 >= c0 && j0 < c1, in1 = j0 + 8 >= c0 && j0 + 8 < c1;
+            // how far back the lane's keys lie (numbers differ by the gap where a key is a kept one)
+            const int dist0 = pos - j0 + (j0 < kept ? gap : 0), dist1 = pos - j0 - 8 + (j0 + 8 < kept ? gap : 0);
             if (shaped) {                                        // (uniform) bounded scores, less the bias of the distance
-                sT[0] = in0 ? shape_score(sT[0] * scale_log2, fz.op.cap_l2, toc, da[0], db[0], pos - j0) : -INFINITY;
-                sT[1] = in0 ? shape_score(sT[1] * scale_log2, fz.op.cap_l2, toc, da[1], db[1], pos - j0) : -INFINITY;
-                sT[2] = in1 ? shape_score(sT[2] * scale_log2, fz.op.cap_l2, toc, da[0], db[0], pos - j0 - 8) : -INFINITY;
-                sT[3] = in1 ? shape_score(sT[3] * scale_log2, fz.op.cap_l2, toc, da[1], db[1], pos - j0 - 8) : -INFINITY;
+                sT[0] = in0 ? shape_score(sT[0] * scale_log2, fz.op.cap_l2, toc, da[0], db[0], dist0) : -INFINITY;
+                sT[1] = in0 ? shape_score(sT[1] * scale_log2, fz.op.cap_l2, toc, da[1], db[1], dist0) : -INFINITY;
+                sT[2] = in1 ? shape_score(sT[2] * scale_log2, fz.op.cap_l2, toc, da[0], db[0], dist1) : -INFINITY;
+                sT[3] = in1 ? shape_score(sT[3] * scale_log2, fz.op.cap_l2, toc, da[1], db[1], dist1) : -INFINITY;
             } else {
                 sT[0] = in0 ? sT[0] * scale_log2 : -INFINITY; sT[1] = in0 ? sT[1] * scale_log2 : -INFINITY;
                 sT[2] = in1 ? sT[2] * scale_log2 : -INFINITY; sT[3] = in1 ? sT[3] * scale_log2 : -INFINITY;
@@ -784,7 +802,7 @@ flash_decode_kernel(const bf16* __restrict__ q, int q_stride,
                     const int j = st * BN + kr0 + n * 8 + 2 * t + (e & 1);
                     float v = -INFINITY;
                     if (j >= c0 && j < c1)
-                        v = shaped ? shape_score(s[n][e] * scale_log2, fz.op.cap_l2, toc, da[e >> 1], db[e >> 1], pos - j)
+                        v = shaped ? shape_score(s[n][e] * scale_log2, fz.op.cap_l2, toc, da[e >> 1], db[e >> 1], pos - j + (j < kept ? gap : 0))
                                    : s[n][e] * scale_log2;
                     s[n][e] = v;
                     mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -1071,11 +1089,12 @@ extern "C" int vl_flash_decode(const void* q, int q_stride, const void* kcache, 
                                int chunk, int S, float* part_acc, float* part_ml, unsigned* err,
                                const int* token_index, void* out, int* arrivals, const float* sinks, int weighting,
                                int block, const float* head_bias, const void* gate, int gate_stride, float softcap,
-                               const float* dist_a, const float* dist_b, void* stream) {
+                               const float* dist_a, const float* dist_b, int keep, void* stream) {
+    if (keep < 0 || (keep > 0 && block > 0)) return VL_ERR_ARGUMENT;
     if (softcap < 0.f || (dist_a == nullptr) != (dist_b == nullptr)) return VL_ERR_ARGUMENT;
     DecodeFusion fz = {};
     fz.sinks = sinks;
-    fz.op = AttnOptions{weighting, block, head_bias, (const bf16*)gate, gate_stride, softcap * 1.4426950408889634f, dist_a, dist_b};
+    fz.op = AttnOptions{weighting, block, head_bias, (const bf16*)gate, gate_stride, softcap * 1.4426950408889634f, dist_a, dist_b, keep};
     return launch_flash_decode(q, q_stride, kcache, vcache, block_table, max_blocks, req_index, positions, T, nq, nkv, hd,
                                page_size, num_pages, scale, window, chunk, S, part_acc, part_ml, err, token_index, out,
                                arrivals, fz, stream);

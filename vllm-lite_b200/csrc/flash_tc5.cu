@@ -35,6 +35,8 @@
 // into blocks of that many, counted from position 0, and a query reads no key of an earlier block; with SIG (the kernel's
 // template argument) a visible key weighs sigmoid(s_j + head_bias[h]) by itself: no maximum, no sum, no rescaling, and
 // nothing is divided; `gate` multiplies head h's output for token t by sigmoid(gate[t * gate_stride + h]).
+// `keep` > 0: a query also reads the request's first `keep` keys, however far behind its window they lie; the tiles of the
+// kept keys are walked first, then those of the window.
 // Every wait on an mbarrier is bounded; when one expires the block records VL_DEV_WAIT_EXPIRED,
 // stops, and still frees its TMEM.
 #include "score_shape.cuh"
@@ -127,7 +129,7 @@ flash_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constan
                  int nq, int nkv, int page_size, int num_pages, float scale_log2, int window, unsigned* err,
                  const float* __restrict__ sinks, int mask_block, const float* __restrict__ head_bias,
                  const bf16* __restrict__ gate, int gate_stride, float cap_l2, const float* __restrict__ dist_a,
-                 const float* __restrict__ dist_b) {
+                 const float* __restrict__ dist_b, int keep) {
     // tiles of the 128-byte swizzle must start on 1024-byte boundaries; there is no static shared
     // memory in this kernel, so the array starts the block's window
     extern __shared__ __align__(1024) unsigned char smem[];
@@ -179,7 +181,10 @@ flash_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constan
     const int hi = pos0 + count - 1;                             // the last key any row reads
     int lo = (window > 0 && pos0 - window + 1 > 0) ? pos0 - window + 1 : 0;         // the first key any row reads
     if (mask_block > 0) lo = max(lo, pos0 / mask_block * mask_block);
-    const int jt0 = lo / BN, n_tiles = hi / BN - jt0 + 1;
+    // the walk: `nkeep` tiles of kept keys that lie before the window's first tile, then the window's
+    const int jt_win = lo / BN, nkeep = min((min(keep, lo) + BN - 1) / BN, jt_win);
+    const int n_tiles = hi / BN - jt_win + 1 + nkeep;
+    auto tile_of = [&](int it) { return it < nkeep ? it : jt_win + it - nkeep; };
 
     // the query tile, rows beyond `count` zero, into the swizzled layout
     for (int idx = tid; idx < BM * (HD / 8); idx += NTHREADS) {
@@ -199,8 +204,8 @@ flash_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constan
         // one tile ahead of its use
         auto lookup = [&](int it) -> int {
             if (lane >= nbox || it >= n_tiles) return beyond;
-            const int first = (jt0 + it) * BN + lane * box_rows;
-            if (first > hi || first + box_rows - 1 < lo) return beyond;
+            const int first = tile_of(it) * BN + lane * box_rows;
+            if (first > hi || (first + box_rows - 1 < lo && first >= keep)) return beyond;
             const int blk = first / page_size;
             const int page = blk < max_blocks ? table[blk] : -1;
             if (page < 0 || page >= num_pages) {
@@ -246,7 +251,7 @@ flash_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constan
         }
         // Slots behind the request's last key hold whatever the page's earlier owner left there.  Their
         // probabilities are zero, but 0 * NaN is NaN: zero those rows of V of the last key tile.
-        const int last = n_tiles - 1, first_bad = hi + 1 - (jt0 + last) * BN;
+        const int last = n_tiles - 1, first_bad = hi + 1 - tile_of(last) * BN;
         if (ok && first_bad < BN) {
             ok = __all_sync(0xffffffffu, mbar_wait_bounded(&v_full[last & 1], (unsigned)((last / 2) & 1)));
             if (ok) {
@@ -344,7 +349,7 @@ flash_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constan
             tc5_wait_ld();
             tc5_fence_before();
             mbar_arrive(&s_free[s]);                             // the scores are in registers: the buffer may be written again
-            const int j0 = (jt0 + it) * BN;
+            const int j0 = tile_of(it) * BN;
             if constexpr (SHAPED) {
 #pragma unroll
                 for (int c = 0; c < BN; ++c)
@@ -356,7 +361,7 @@ flash_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constan
             if (edge) {
 #pragma unroll
                 for (int c = 0; c < BN; ++c)
-                    if (j0 + c > qpos || j0 + c < first_key) sv[c] = masked;          // -inf
+                    if (j0 + c > qpos || (j0 + c < first_key && j0 + c >= keep)) sv[c] = masked;          // -inf
             }
             unsigned pk[BN / 2];
             bool bump = false;
@@ -459,8 +464,9 @@ extern "C" int vl_flash_prefill_tc5(const void* q, int q_stride, void* out, cons
                                     int nq, int nkv, int hd, int page_size, int num_pages, float scale, int window,
                                     unsigned* err, const float* sinks, int weighting, int mask_block, const float* head_bias,
                                     const void* gate, int gate_stride, float softcap, const float* dist_a, const float* dist_b,
-                                    void* stream) {
+                                    int keep, void* stream) {
     if (num_tiles <= 0) return VL_OK;
+    if (keep < 0 || (keep > 0 && mask_block > 0)) return VL_ERR_ARGUMENT;
     if (hd != HD) return VL_ERR_UNSUPPORTED;
     if (softcap < 0.f || (dist_a == nullptr) != (dist_b == nullptr)) return VL_ERR_ARGUMENT;
     if (weighting < 0 || weighting > 1 || mask_block < 0 || (gate && gate_stride < nq) || (weighting == 1 && sinks)) return VL_ERR_ARGUMENT;
@@ -493,5 +499,5 @@ extern "C" int vl_flash_prefill_tc5(const void* q, int q_stride, void* out, cons
     return vl_launch(kernel, dim3(nq, num_tiles), dim3(NTHREADS), SMEM_BYTES, (cudaStream_t)stream,
                      map_k, map_v, pages_k, pages_v, use_pages, (const bf16*)q, q_stride, (bf16*)out, block_table, max_blocks, (const int4*)tiles,
                      num_tiles, nq, nkv, page_size, num_pages, scale * 1.4426950408889634f, window, err, sinks, mask_block,
-                     head_bias, (const bf16*)gate, gate_stride, softcap * 1.4426950408889634f, dist_a, dist_b);
+                     head_bias, (const bf16*)gate, gate_stride, softcap * 1.4426950408889634f, dist_a, dist_b, keep);
 }

@@ -243,7 +243,9 @@ gemm_batched_bf16_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict_
             for (int nt = 0; nt < NT; ++nt) {
                 const int n = n0 + wn * WN + nt * 8 + t2;
                 const float v0 = gm_unary(acc[nt][2 * half] * scale, act), v1 = gm_unary(acc[nt][2 * half + 1] * scale, act);
-                if (sizeof(TC) == 2 && pair_ok && n + 1 < N) {          // two bfloat16 in one 4-byte store
+                if (sizeof(TC) == 4 && ((ldc | c_bs | n) & 1) == 0 && n + 1 < N && (((uintptr_t)C) & 7) == 0) {
+                    *reinterpret_cast<float2*>(crow + n) = make_float2(v0, v1);
+                } else if (sizeof(TC) == 2 && pair_ok && n + 1 < N) {   // two bfloat16 in one 4-byte store
                     __nv_bfloat162 pr = __floats2bfloat162_rn(v0, v1);
                     *reinterpret_cast<unsigned*>(crow + n) = *reinterpret_cast<unsigned*>(&pr);
                 } else {
@@ -286,48 +288,58 @@ static bool gm_aligned(const void* A, const void* W, int K, int lda, int ldw, lo
     return !(K % 8 || lda % 8 || ldw % 8 || a_bs % 8 || w_bs % 8 || w_gs % 8 || (((uintptr_t)A | (uintptr_t)W) & 15));
 }
 
-static int launch_batched_mma(const bf16* A, const bf16* W, bf16* C, int M, int N, int K, int lda, int ldw, int ldc,
+template <typename TC>
+static int launch_batched_mma(const bf16* A, const bf16* W, TC* C, int M, int N, int K, int lda, int ldw, int ldc,
                               long long a_bs, long long w_bs, long long c_bs, int batch, const int* tile_group,
                               long long w_gs, int bm, const int* row_index, int index_div, const float* row_scale,
                               int act, float alpha, float limit, float shift, cudaStream_t s) {
     dim3 grid((N + GM_BN - 1) / GM_BN, (M + bm - 1) / bm, batch);
     if (grid.y > 65535 || grid.z > 65535) return VL_ERR_UNSUPPORTED;
     if (bm == 64)
-        return launch_mma_kernel<64, bf16>(grid, s, K, A, W, C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, tile_group, w_gs,
+        return launch_mma_kernel<64, TC>(grid, s, K, A, W, C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, tile_group, w_gs,
                                            row_index, index_div, row_scale, act, alpha, limit, shift);
-    return launch_mma_kernel<16, bf16>(grid, s, K, A, W, C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, tile_group, w_gs,
+    return launch_mma_kernel<16, TC>(grid, s, K, A, W, C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, tile_group, w_gs,
                                        row_index, index_div, row_scale, act, alpha, limit, shift);
 }
 
-template <typename T>
-static int launch_batched(const T* A, const T* W, T* C, int M, int N, int K, int lda, int ldw, int ldc,
+template <typename T, typename TC>
+static int launch_batched(const T* A, const T* W, TC* C, int M, int N, int K, int lda, int ldw, int ldc,
                           long long a_bs, long long w_bs, long long c_bs, int batch, const int* tile_group,
                           long long w_gs, int bm, cudaStream_t s) {
     dim3 grid((N + GB_BN - 1) / GB_BN, (M + bm - 1) / bm, batch);
     if (grid.y > 65535 || grid.z > 65535) return VL_ERR_UNSUPPORTED;
     if (bm == 64)
-        return vl_launch(gemm_batched_nt_kernel<T, T, T, 64>, grid, dim3(256), 0, s, A, W, C, M, N, K, lda, ldw, ldc,
+        return vl_launch(gemm_batched_nt_kernel<T, T, TC, 64>, grid, dim3(256), 0, s, A, W, C, M, N, K, lda, ldw, ldc,
                          a_bs, w_bs, c_bs, tile_group, w_gs);
-    return vl_launch(gemm_batched_nt_kernel<T, T, T, 16>, grid, dim3(256), 0, s, A, W, C, M, N, K, lda, ldw, ldc,
+    return vl_launch(gemm_batched_nt_kernel<T, T, TC, 16>, grid, dim3(256), 0, s, A, W, C, M, N, K, lda, ldw, ldc,
                      a_bs, w_bs, c_bs, tile_group, w_gs);
 }
 
 // bm: rows per tile, 64 or 16.  With tile_group, M is the padded number of sorted rows (a multiple of bm).
-extern "C" int vl_gemm_batched_nt(const void* A, const void* W, void* C, int dtype, int M, int N, int K,
+// c_dtype: the operands' dtype, or float32 (the sums as they are).
+extern "C" int vl_gemm_batched_nt(const void* A, const void* W, void* C, int dtype, int c_dtype, int M, int N, int K,
                                   int lda, int ldw, int ldc, long long a_bs, long long w_bs, long long c_bs,
                                   int batch, const int* tile_group, long long w_gs, int bm, void* stream) {
     if (M <= 0 || N <= 0 || batch <= 0) return VL_OK;
     if (K <= 0 || lda < K || ldw < K || ldc < N || (bm != 64 && bm != 16)) return VL_ERR_ARGUMENT;
     if (tile_group && M % bm) return VL_ERR_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
+    if (c_dtype != dtype && c_dtype != VL_F32) return VL_ERR_UNSUPPORTED;
     if (dtype == VL_F32)
-        return launch_batched<float>((const float*)A, (const float*)W, (float*)C, M, N, K, lda, ldw, ldc,
+        return launch_batched<float, float>((const float*)A, (const float*)W, (float*)C, M, N, K, lda, ldw, ldc,
                                      a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, s);
+    if (dtype == VL_BF16 && c_dtype == VL_F32) {
+        if (gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
+            return launch_batched_mma((const bf16*)A, (const bf16*)W, (float*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs,
+                                      batch, tile_group, w_gs, bm, nullptr, 1, nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f, s);
+        return launch_batched<bf16, float>((const bf16*)A, (const bf16*)W, (float*)C, M, N, K, lda, ldw, ldc,
+                                           a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, s);
+    }
     if (dtype == VL_BF16) {
         if (gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
             return launch_batched_mma((const bf16*)A, (const bf16*)W, (bf16*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs,
                                       batch, tile_group, w_gs, bm, nullptr, 1, nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f, s);
-        return launch_batched<bf16>((const bf16*)A, (const bf16*)W, (bf16*)C, M, N, K, lda, ldw, ldc,
+        return launch_batched<bf16, bf16>((const bf16*)A, (const bf16*)W, (bf16*)C, M, N, K, lda, ldw, ldc,
                                     a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, s);
     }
     return VL_ERR_UNSUPPORTED;

@@ -70,6 +70,7 @@ struct Core {
     int page_size = 16;
     std::vector<Pool> pools;
     std::vector<int> windows;                 // per group, 0 = none
+    std::vector<int> keeps;                   // per group, 0 = none: first tokens of a request that stay readable behind the window
     std::vector<int> chunks;                  // per group, 0 = none: positions in blocks of that many, no key of an earlier block is read
     Pool slots;
     std::unordered_map<long long, Request> requests;
@@ -89,7 +90,7 @@ inline int align4(int n) { return (n + 3) & ~3; }
 extern "C" {
 
 void* vc_create(int page_size, int num_groups, const int* pages_per_group, const int* windows, const int* chunks,
-                int max_requests) {
+                const int* keeps, int max_requests) {
     if (page_size <= 0 || num_groups < 0 || max_requests < 0) return nullptr;
     Core* c = new Core();
     c->page_size = page_size;
@@ -98,6 +99,7 @@ void* vc_create(int page_size, int num_groups, const int* pages_per_group, const
         c->pools.emplace_back(pages_per_group[g]);
         c->windows.push_back(windows ? windows[g] : 0);
         c->chunks.push_back(chunks ? chunks[g] : 0);
+        c->keeps.push_back(keeps ? keeps[g] : 0);
     }
     c->slots = Pool(max_requests);
     return c;
@@ -166,7 +168,7 @@ int vc_append(void* h, long long key, long long count, long long* start) {
 
 // Gives back the pages that no later query of the request can read: the next query sits at
 // position num_tokens and reads from num_tokens - window + 1 on, and from the start of its own block of
-// `chunk` positions on.  *freed = pages returned.
+// `chunk` positions on; the pages of the first `keep` tokens stay.  *freed = pages returned.
 int vc_release_behind_window(void* h, long long key, int* freed) {
     Core* c = static_cast<Core*>(h);
     auto it = c->requests.find(key);
@@ -182,7 +184,7 @@ int vc_release_behind_window(void* h, long long key, int* freed) {
         long long dead = first_needed / c->page_size;
         if (dead > (long long)r.tables[g].size()) dead = (long long)r.tables[g].size();
         std::vector<int> gone;
-        for (long long b = 0; b < dead; ++b)
+        for (long long b = (c->keeps[g] + c->page_size - 1) / c->page_size; b < dead; ++b)
             if (r.tables[g][b] >= 0) { gone.push_back(r.tables[g][b]); r.tables[g][b] = -1; }
         const int rc = c->pools[g].release(gone.data(), (int)gone.size());
         if (rc) return rc;

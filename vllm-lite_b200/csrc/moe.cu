@@ -8,6 +8,8 @@
 //                   `choice_bias` (a number per expert): the choice, also that of the groups, is made on
 //                   score + choice_bias instead of the logits; the weights stay the scores without it.
 //                   `group_top`: a group counts by the sum of its `group_top` largest choice values (1: its largest).
+//                   `extra` columns of z behind the E experts' (at most one): their sigmoid goes to extra_out [T] (the weight of a
+//                   feed-forward that every token passes).
 //                   -> expert ids [T, top], weights float32 [T, top]
 //   vl_moe_align    sorts the T * top (token, choice) pairs by expert into tiles of `bm` rows, every
 //                   expert's rows padded up to whole tiles: sorted_rows[r] = pair or -1,
@@ -16,7 +18,9 @@
 //                   on it: a row's arithmetic does not depend on its place.
 //   vl_moe_gather   rows[r] = weight(pair) * h[token(pair)] (or h itself), zeros for padding rows
 //   vl_moe_combine  out[t] = sum over the token's choices, in the order of the choices, of
-//                   (weight *) result[place[pair]] (+ add[t]: a row that every token gets, added last)
+//                   (weight *) result[place[pair]] (+ add[t]: a row that every token gets, times add_weight[t] when
+//                   given, added last).  A choice whose expert id is `identity_from` or more is an expert without
+//                   tensors whose result is its input, h[t]
 //
 // Padded tokens of a graph step are ordinary rows here: they cost a row of work and nobody reads
 // their result.
@@ -28,10 +32,10 @@
 
 // one warp per token; z [ntok, E]: the router's logits (csrc/gemm_batched.cu: vl_gemm_rows_f32w)
 __global__ void __launch_bounds__(128)
-moe_route_kernel(const float* __restrict__ z, int slices, int ntok, int E, int top,
+moe_route_kernel(const float* __restrict__ z, int slices, int ntok, int E, int ldz, int top,
                  int score_fn, int renorm, int groups, int keep, const float* __restrict__ bias,
                  const float* __restrict__ choice_bias, int group_top, float renorm_eps,
-                 int* __restrict__ ids, float* __restrict__ weights) {
+                 int* __restrict__ ids, float* __restrict__ weights, float* __restrict__ extra_out) {
     extern __shared__ float s_scores[];                  // [4][E], then [4][groups], then [4][E] logits kept for the weights
     pdl_launch_dependents();
     pdl_wait();
@@ -41,8 +45,13 @@ moe_route_kernel(const float* __restrict__ z, int slices, int ntok, int E, int t
     float* sc = s_scores + (size_t)warp * E;
     for (int e = lane; e < E; e += 32) {                 // the logits came as sums over slices of K: added in their order
         float v = 0.f;
-        for (int sl = 0; sl < slices; ++sl) v += z[((size_t)sl * ntok + t) * E + e];
+        for (int sl = 0; sl < slices; ++sl) v += z[((size_t)sl * ntok + t) * ldz + e];
         sc[e] = bias ? v + bias[e] : v;
+    }
+    if (extra_out && lane == 0) {
+        float v = 0.f;
+        for (int sl = 0; sl < slices; ++sl) v += z[((size_t)sl * ntok + t) * ldz + E];
+        extra_out[t] = 1.0f / (1.0f + expf(-v));
     }
     __syncwarp();
     // The choice is made on the logits: both score functions grow with z, and a sigmoid that has
@@ -199,7 +208,8 @@ __global__ void moe_gather_kernel(const T* __restrict__ h, const int* __restrict
 template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ result, const int* __restrict__ place,
                                    const float* __restrict__ weights, int top, int N, int scale_output,
-                                   T* __restrict__ out, const T* __restrict__ add) {
+                                   T* __restrict__ out, const T* __restrict__ add, const float* __restrict__ add_weight,
+                                   const int* __restrict__ ids, int identity_from, const T* __restrict__ h) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -208,9 +218,10 @@ __global__ void moe_combine_kernel(const T* __restrict__ result, const int* __re
             float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
             for (int j = 0; j < top; ++j) {
                 const int r = place[(size_t)t * top + j];
-                if (r < 0) continue;
+                const bool identity = h && ids[(size_t)t * top + j] >= identity_from;
+                if (r < 0 && !identity) continue;
                 float v[8];
-                load8(result + (size_t)r * N + n, v);
+                load8(identity ? h + (size_t)t * N + n : result + (size_t)r * N + n, v);
                 const float w = scale_output ? weights[(size_t)t * top + j] : 1.0f;
 #pragma unroll
                 for (int i = 0; i < 8; ++i) acc[i] += scale_output ? w * v[i] : v[i];
@@ -218,8 +229,9 @@ __global__ void moe_combine_kernel(const T* __restrict__ result, const int* __re
             if (add) {                                       // one more row for every token (an expert that all tokens share)
                 float v[8];
                 load8(add + (size_t)t * N + n, v);
+                const float w = add_weight ? add_weight[t] : 1.0f;
 #pragma unroll
-                for (int i = 0; i < 8; ++i) acc[i] += v[i];
+                for (int i = 0; i < 8; ++i) acc[i] += add_weight ? w * v[i] : v[i];
             }
             store8(out + (size_t)t * N + n, acc);
         }
@@ -229,26 +241,28 @@ __global__ void moe_combine_kernel(const T* __restrict__ result, const int* __re
         float acc = 0.f;
         for (int j = 0; j < top; ++j) {
             const int r = place[(size_t)t * top + j];
-            if (r < 0) continue;
-            const float v = to_f32(result[(size_t)r * N + n]);
+            const bool identity = h && ids[(size_t)t * top + j] >= identity_from;
+            if (r < 0 && !identity) continue;
+            const float v = to_f32(identity ? h[(size_t)t * N + n] : result[(size_t)r * N + n]);
             acc += scale_output ? weights[(size_t)t * top + j] * v : v;
         }
-        if (add) acc += to_f32(add[(size_t)t * N + n]);
+        if (add) acc += (add_weight ? add_weight[t] : 1.0f) * to_f32(add[(size_t)t * N + n]);
         out[(size_t)t * N + n] = from_f32<T>(acc);
     }
 }
 
-extern "C" int vl_moe_route(const float* z, int slices, int T, int E, int top, int score_fn, int renorm, int groups, int keep,
+extern "C" int vl_moe_route(const float* z, int slices, int T, int E, int ldz, int top, int score_fn, int renorm, int groups, int keep,
                             const float* bias, const float* choice_bias, int group_top, float renorm_eps, int* ids,
-                            float* weights, void* stream) {
+                            float* weights, float* extra_out, void* stream) {
     if (T <= 0) return VL_OK;
+    if (ldz < E + (extra_out ? 1 : 0)) return VL_ERR_ARGUMENT;
     if (group_top < 1 || renorm_eps < 0.f) return VL_ERR_ARGUMENT;
     if (E <= 0 || E > MOE_MAX_EXPERTS || top <= 0 || top > E || slices <= 0) return VL_ERR_ARGUMENT;
     if (score_fn != MOE_SCORE_SIGMOID && score_fn != MOE_SCORE_SOFTMAX) return VL_ERR_ARGUMENT;
     if (groups < 1 || E % groups || keep < 1 || keep > groups || keep * (E / groups) < top) return VL_ERR_ARGUMENT;
     return vl_launch(moe_route_kernel, dim3((T + 3) / 4), dim3(128), (size_t)4 * (E + groups + (choice_bias ? E : 0)) * sizeof(float),
-                     (cudaStream_t)stream, z, slices, T, E, top, score_fn, renorm, groups, keep, bias, choice_bias, group_top,
-                     renorm_eps, ids, weights);
+                     (cudaStream_t)stream, z, slices, T, E, ldz, top, score_fn, renorm, groups, keep, bias, choice_bias, group_top,
+                     renorm_eps, ids, weights, extra_out);
 }
 
 // cap = rows of the sorted buffer (a multiple of bm, at least npairs rounded up per expert: npairs + E * (bm - 1)
@@ -277,15 +291,16 @@ extern "C" int vl_moe_gather(const void* h, int dtype, const int* sorted_rows, c
 }
 
 extern "C" int vl_moe_combine(const void* result, int dtype, const int* place, const float* weights, int T, int top,
-                              int N, int scale_output, void* out, const void* add, void* stream) {
+                              int N, int scale_output, void* out, const void* add, const float* add_weight, const int* ids, int identity_from,
+                              const void* h, void* stream) {
     if (T <= 0) return VL_OK;
-    if (top <= 0 || N <= 0) return VL_ERR_ARGUMENT;
+    if (top <= 0 || N <= 0 || (h && !ids)) return VL_ERR_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == VL_F32)
         return vl_launch(moe_combine_kernel<float>, dim3(T, (N + 511) / 512), dim3(128), 0, s, (const float*)result, place, weights, top, N,
-                         scale_output, (float*)out, (const float*)add);
+                         scale_output, (float*)out, (const float*)add, add_weight, ids, identity_from, (const float*)h);
     if (dtype == VL_BF16)
         return vl_launch(moe_combine_kernel<bf16>, dim3(T, (N + 511) / 512), dim3(128), 0, s, (const bf16*)result, place, weights, top, N,
-                         scale_output, (bf16*)out, (const bf16*)add);
+                         scale_output, (bf16*)out, (const bf16*)add, add_weight, ids, identity_from, (const bf16*)h);
     return VL_ERR_UNSUPPORTED;
 }

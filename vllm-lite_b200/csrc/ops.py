@@ -34,7 +34,17 @@ def dtype_code(dtype) -> int:
 _SIGNATURES = {
     ("embed_norm", "vl_embed"): [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
     ("embed_norm", "vl_rmsnorm_add"): [c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p,
-                                       c_float, c_float, c_void_p],
+                                       c_float, c_float, c_void_p, c_void_p, c_void_p],
+    ("embed_norm", "vl_embed_pair"): [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_int, c_longlong,
+                                      c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
+    ("head_work", "vl_head_work"): [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int,
+                                    c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                    c_int, c_int, c_int, c_int, c_longlong, c_void_p, c_void_p],
+    ("head_work", "vl_combine_maps"): [c_void_p, c_void_p, c_int, c_float, c_float, c_float, c_int, c_longlong, c_int, c_int, c_void_p],
+    ("linear_scan", "vl_linear_scan"): [c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
+                                        c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int,
+                                        c_void_p],
+    ("activation", "vl_poly_norm"): [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_void_p],
     ("embed_norm", "vl_add_rmsnorm"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
     ("embed_norm", "vl_add_bias"): [c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p],
     ("embed_norm", "vl_cast"): [c_void_p, c_int, c_void_p, c_int, c_longlong, c_void_p],
@@ -44,7 +54,7 @@ _SIGNATURES = {
     ("attention", "vl_paged_attention"): [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                           c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                           c_float, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p,
-                                          c_void_p, c_void_p],
+                                          c_int, c_void_p, c_void_p],
     ("rope_cache", "vl_head_norm_write"): [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int,
                                            c_float, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_longlong,
                                            c_int, c_void_p, c_void_p],
@@ -73,14 +83,14 @@ _SIGNATURES = {
                                                  c_int, c_int, c_void_p, c_void_p, c_void_p],
     ("flash_attn", "vl_flash_prefill"): [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
                                          c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p,
-                                         c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p],
+                                         c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p],
     ("flash_tc5", "vl_flash_prefill_tc5"): [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
                                             c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p,
-                                            c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p],
+                                            c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p],
     ("flash_attn", "vl_flash_decode"): [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                         c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int,
                                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                        c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p],
+                                        c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p],
     ("flash_attn", "vl_flash_decode_fused"): [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                               c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int,
                                               c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -97,19 +107,20 @@ _SIGNATURES = {
     ("embed_norm", "vl_layernorm_rows"): [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
     ("latent", "vl_latent_norm_write"): [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p,
                                          c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
-    ("gemm_batched", "vl_gemm_batched_nt"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+    ("gemm_batched", "vl_gemm_batched_nt"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                              c_longlong, c_longlong, c_longlong, c_int, c_void_p, c_longlong, c_int, c_void_p],
     ("gemm_batched", "vl_gemm_grouped_fused"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
                                                 c_longlong, c_int, c_void_p, c_int, c_void_p, c_int, c_float, c_float, c_float,
                                                 c_void_p],
-    ("moe", "vl_moe_route"): [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_float,
-                              c_void_p, c_void_p, c_void_p],
+    ("moe", "vl_moe_route"): [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_float,
+                              c_void_p, c_void_p, c_void_p, c_void_p],
     ("gemm_batched", "vl_gemm_rows_f32w"): [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     ("gemm_tc5_grouped", "vl_gemm_bf16_tc5_grouped"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                                                        c_void_p, c_int, c_float, c_float, c_float, c_void_p, c_void_p],
     ("moe", "vl_moe_align"): [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     ("moe", "vl_moe_gather"): [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
-    ("moe", "vl_moe_combine"): [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
+    ("moe", "vl_moe_combine"): [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                                c_int, c_void_p, c_void_p],
     ("gemm_f32", "vl_gemm_f32_nt"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     ("gemm_bf16", "vl_gemm_bf16_small_m"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                             c_void_p, c_int, c_void_p],
@@ -129,7 +140,7 @@ _SIGNATURES = {
                               c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     ("hyper", "vl_dyt_rows"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     ("recurrent", "vl_short_conv"): [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong,
-                                     c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p],
+                                     c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
     ("recurrent", "vl_ssd_scan"): [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                    c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     ("recurrent", "vl_mlstm_scan"): [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
@@ -216,6 +227,22 @@ def embed(ids, table, out, err, scale=1.0):
         raise KernelError(f"out must be [{T}, {H}], got {tuple(out.shape)}")
     _check(_fn("embed_norm", "vl_embed")(_ptr(ids), _ptr(table), dtype_code(table.dtype), _ptr(out), T, H, V,
                                          float(scale), _ptr(err), _stream()), "vl_embed")
+    return out
+
+
+def embed_pair(ids, table, pairs, out, scale, buckets, mul_prev, mul_cur, state, cu, slots, req_index, positions, err):
+    """out[t] = table[id_t] * scale + pairs[row], row = (id_(t-1) mul_prev + id_t mul_cur) mod buckets, or `buckets` at
+    position 0; the token before a portion's first is state[slot, 0] (int32 [slots, n]), replaced by the portion's last."""
+    _need(ids, torch.int32, "ids", 1); _need(table, None, "table", 2); _need(pairs, table.dtype, "pairs", 2)
+    _need(out, torch.float32, "out", 2); _need(state, torch.int32, "state", 2)
+    _need(req_index, torch.int32, "req_index", 1); _need(positions, torch.int32, "positions", 1)
+    T, (V, H) = ids.shape[0], table.shape
+    if out.shape != (T, H) or pairs.shape != (buckets + 1, H) or req_index.shape[0] != T or positions.shape[0] != T:
+        raise KernelError(f"embed_pair: out {tuple(out.shape)}, pairs {tuple(pairs.shape)} for {buckets} buckets of {H}")
+    _seg_args(cu, slots)
+    _check(_fn("embed_norm", "vl_embed_pair")(_ptr(ids), _ptr(table), _ptr(pairs), dtype_code(table.dtype), _ptr(out), T, H, V,
+                                              float(scale), int(buckets), int(mul_prev), int(mul_cur), _ptr(state), state.shape[1],
+                                              _ptr(cu), _ptr(slots), _ptr(req_index), _ptr(positions), _ptr(err), _stream()), "vl_embed_pair")
     return out
 
 
@@ -450,12 +477,23 @@ def _check_score_shape(num_heads, softcap, distance):
     return cap, a, b
 
 
+def _check_keep(keep, window, chunk):
+    """One more option of every attention entry point: a query also reads the request's first `keep` keys, however far
+    behind its window they lie (without a window: nothing changes, every key is read).  Not together with `chunk`."""
+    keep = int(keep or 0) if window else 0
+    if keep < 0 or (keep and chunk):
+        raise KernelError(f"{keep} kept keys go with a window, not with a mask in blocks")
+    return keep
+
+
 def paged_attention(qkv, out, k_cache, v_cache, block_table, req_index, positions,
                     num_heads, num_kv_heads, head_dim, scale, window, err, sinks=None,
-                    weighting="softmax", chunk=None, head_bias=None, gate=None, softcap=None, distance=None):
+                    weighting="softmax", chunk=None, head_bias=None, gate=None, softcap=None, distance=None, keep=None):
     """out [T, nq*hd] = attention of the q part of qkv over the pages of each token's request.
     `sinks` (float32 [nq]): one more term exp(sinks[h]) in every softmax denominator of head h.
-    `weighting`, `chunk`, `head_bias`, `gate`: see `_check_variant`.  `softcap`, `distance`: see `_check_score_shape`."""
+    `weighting`, `chunk`, `head_bias`, `gate`: see `_check_variant`.  `softcap`, `distance`: see `_check_score_shape`.
+    `keep`: see `_check_keep`."""
+    keep = _check_keep(keep, window, chunk)
     _check_sinks(sinks, num_heads)
     cap, dist_a, dist_b = _check_score_shape(num_heads, softcap, distance)
     mode, chunk, gate_stride = _check_variant(qkv, num_heads, weighting, chunk, head_bias, gate, sinks)
@@ -475,7 +513,7 @@ def paged_attention(qkv, out, k_cache, v_cache, block_table, req_index, position
         _ptr(block_table), block_table.shape[1], _ptr(req_index), _ptr(positions),
         T, num_heads, num_kv_heads, head_dim, k_cache.shape[2], k_cache.shape[0],
         float(scale), int(window or 0), _ptr(sinks), mode, chunk, _ptr(head_bias), _ptr(gate), gate_stride,
-        cap, _ptr(dist_a), _ptr(dist_b), _ptr(err), _stream()), "vl_paged_attention")
+        cap, _ptr(dist_a), _ptr(dist_b), keep, _ptr(err), _stream()), "vl_paged_attention")
     return out
 
 
@@ -570,12 +608,13 @@ def _flash_checks(qkv, k_cache, v_cache, block_table, num_heads, num_kv_heads, h
 
 def flash_prefill(qkv, out, k_cache, v_cache, block_table, tiles, num_heads, num_kv_heads, head_dim, scale, window, err,
                   tile_rows=64, sinks=None, weighting="softmax", mask_chunk=None, head_bias=None, gate=None, softcap=None,
-                  distance=None):
+                  distance=None, keep=None):
     """Tensor-core (mma.sync) attention for prompt portions.  `tiles` int32 [n, 4]: (row of the block
     table, index of the tile's first token in the step, tokens (<= tile_rows), position of the first
     token); the tiles of a step cover every token that the kernel is to serve once.
     `weighting`, `mask_chunk` (the `chunk` there), `head_bias`, `gate`: see `_check_variant`; `softcap`, `distance`: see
-    `_check_score_shape`."""
+    `_check_score_shape`; `keep`: see `_check_keep`."""
+    keep = _check_keep(keep, window, mask_chunk)
     _flash_checks(qkv, k_cache, v_cache, block_table, num_heads, num_kv_heads, head_dim)
     _check_sinks(sinks, num_heads)
     mode, mask_chunk, gate_stride = _check_variant(qkv, num_heads, weighting, mask_chunk, head_bias, gate, sinks)
@@ -587,7 +626,7 @@ def flash_prefill(qkv, out, k_cache, v_cache, block_table, tiles, num_heads, num
         _ptr(qkv), qkv.shape[1], _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1],
         _ptr(tiles), tiles.shape[0], int(tile_rows), num_heads, num_kv_heads, head_dim, k_cache.shape[2],
         k_cache.shape[0], float(scale), int(window or 0), _ptr(err), _ptr(sinks), mode, mask_chunk, _ptr(head_bias),
-        _ptr(gate), gate_stride, cap, _ptr(dist_a), _ptr(dist_b), _stream()), "vl_flash_prefill")
+        _ptr(gate), gate_stride, cap, _ptr(dist_a), _ptr(dist_b), keep, _stream()), "vl_flash_prefill")
     return out
 
 
@@ -602,10 +641,12 @@ def flash_tc5_supported(dtype, head_dim, page_size) -> bool:
 
 
 def flash_prefill_tc5(qkv, out, k_cache, v_cache, block_table, tiles, num_heads, num_kv_heads, head_dim, scale, window, err,
-                      sinks=None, weighting="softmax", mask_chunk=None, head_bias=None, gate=None, softcap=None, distance=None):
+                      sinks=None, weighting="softmax", mask_chunk=None, head_bias=None, gate=None, softcap=None, distance=None,
+                      keep=None):
     """Attention for prompt portions on the tcgen05 tensor cores; `tiles` as for `flash_prefill`,
     up to 128 tokens each.  `weighting`, `mask_chunk` (the `chunk` there), `head_bias`, `gate`: see `_check_variant`;
-    `softcap`, `distance`: see `_check_score_shape`."""
+    `softcap`, `distance`: see `_check_score_shape`; `keep`: see `_check_keep`."""
+    keep = _check_keep(keep, window, mask_chunk)
     cap, dist_a, dist_b = _check_score_shape(num_heads, softcap, distance)
     _flash_checks(qkv, k_cache, v_cache, block_table, num_heads, num_kv_heads, head_dim)
     _need(out, torch.bfloat16, "out", 2); _need(tiles, torch.int32, "tiles", 2)
@@ -619,7 +660,7 @@ def flash_prefill_tc5(qkv, out, k_cache, v_cache, block_table, tiles, num_heads,
         _ptr(qkv), qkv.shape[1], _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1],
         _ptr(tiles), tiles.shape[0], num_heads, num_kv_heads, head_dim, k_cache.shape[2], k_cache.shape[0],
         float(scale), int(window or 0), _ptr(err), _ptr(sinks), mode, mask_chunk, _ptr(head_bias), _ptr(gate), gate_stride,
-        cap, _ptr(dist_a), _ptr(dist_b), _stream()), "vl_flash_prefill_tc5")
+        cap, _ptr(dist_a), _ptr(dist_b), keep, _stream()), "vl_flash_prefill_tc5")
     return out
 
 
@@ -658,7 +699,7 @@ def flash_decode_streams(dtype, num_tokens, num_kv_heads, head_dim, page_size, m
 def flash_decode(qkv, out, k_cache, v_cache, block_table, req_index, positions, num_heads, num_kv_heads,
                  head_dim, scale, window, max_context, part_acc, part_ml, err, chunk=DECODE_CHUNK, token_index=None,
                  stream_kernel=None, arrivals=None, fold=None, sinks=None, weighting="softmax", mask_chunk=None,
-                 head_bias=None, gate=None, softcap=None, distance=None):
+                 head_bias=None, gate=None, softcap=None, distance=None, keep=None):
     """Tensor-core version of `decode_attention` (bfloat16): every block takes a chunk of a token's
     keys; the chunks are merged by the block that finishes last (`arrivals`: int32 counters,
     `flash_decode_arrivals` of them, zero before the first call and left zero) or, without
@@ -674,12 +715,15 @@ def flash_decode(qkv, out, k_cache, v_cache, block_table, req_index, positions, 
     written to the cache by this launch (slots None: not written).  The same bits as the two kernels in turn.
     `weighting`, `mask_chunk` (the `chunk` there), `head_bias`, `gate`: see `_check_variant`.  The sigmoid and the gate
     go with the block-per-chunk kernel that merges its chunks itself (`arrivals` given, few enough chunks).
-    `softcap`, `distance` (see `_check_score_shape`) go with the block-per-chunk kernel, merged either way."""
+    `softcap`, `distance` (see `_check_score_shape`) go with the block-per-chunk kernel, merged either way.  `keep` (see
+    `_check_keep`) goes with the block-per-chunk kernel that merges its chunks itself; `max_context` then bounds the number
+    of keys a token reads (window + keep at most), not its position."""
+    keep = _check_keep(keep, window, mask_chunk)
     _flash_checks(qkv, k_cache, v_cache, block_table, num_heads, num_kv_heads, head_dim)
     _check_sinks(sinks, num_heads)
     mode, mask_chunk, gate_stride = _check_variant(qkv, num_heads, weighting, mask_chunk, head_bias, gate, sinks)
     cap, dist_a, dist_b = _check_score_shape(num_heads, softcap, distance)
-    variant = bool(mode or mask_chunk or gate is not None)
+    variant = bool(mode or mask_chunk or gate is not None or keep)
     if (variant or cap or dist_a is not None) and fold is not None:
         raise KernelError("flash_decode: the folded head work goes with the plain softmax")
     if cap or dist_a is not None:
@@ -702,7 +746,7 @@ def flash_decode(qkv, out, k_cache, v_cache, block_table, req_index, positions, 
         raise KernelError(f"flash_decode: scratch too small ({part_acc.numel()} < {need_acc})")
     if variant:
         if stream_kernel or arrivals is None or S > _own_merge_cap(head_dim):
-            raise KernelError("flash_decode: weighting, mask chunk and gate go with the kernel that merges its chunks itself")
+            raise KernelError("flash_decode: weighting, mask chunk, gate and kept keys go with the kernel that merges its chunks itself")
         stream_kernel = False
     if stream_kernel is None:
         stream_kernel = fold is None and flash_decode_streams(qkv.dtype, T, num_kv_heads, head_dim, k_cache.shape[2], max_context)
@@ -723,7 +767,7 @@ def flash_decode(qkv, out, k_cache, v_cache, block_table, req_index, positions, 
         if fold is None:
             _check(_fn("flash_attn", "vl_flash_decode", {"FA_HD": head_dim})(
                 *args, _ptr(out) if arrivals is not None else None, _ptr(arrivals), _ptr(sinks), mode, mask_chunk,
-                _ptr(head_bias), _ptr(gate), gate_stride, cap, _ptr(dist_a), _ptr(dist_b), _stream()), "vl_flash_decode")
+                _ptr(head_bias), _ptr(gate), gate_stride, cap, _ptr(dist_a), _ptr(dist_b), keep, _stream()), "vl_flash_decode")
         else:
             qw, kw, eps, inv_freq, rot, slots = fold
             for t, n in ((qw, "q_weight"), (kw, "k_weight"), (inv_freq, "inv_freq")):
@@ -827,6 +871,16 @@ def scale_softcap(logits, scale, cap):
     return logits
 
 
+def poly_norm(x, coef, eps, out):
+    """out[r] = c0 N(x) + c1 N(x^2) + c2 N(x^3) + c3 with N(v) = v / sqrt(mean(v^2) + eps) over row r; coef float32 [4]."""
+    _need(x, None, "x", 2); _need(out, x.dtype, "out", 2); _need(coef, torch.float32, "coef", 1)
+    if out.shape != x.shape or coef.shape[0] != 4:
+        raise KernelError("poly_norm: out has x's shape, coef four entries")
+    _check(_fn("activation", "vl_poly_norm")(_ptr(x), _ptr(out), dtype_code(x.dtype), x.shape[0], x.shape[1], _ptr(coef), float(eps),
+                                             _stream()), "vl_poly_norm")
+    return out
+
+
 # ---------------------------------------------------------------- layer norm
 def layernorm_add(y, weight, eps, x, cast=None):
     """x[r] += layer_norm(y[r]) * weight (no bias; float32 arithmetic); x float32 [T, H], y in the activation
@@ -846,8 +900,14 @@ def layernorm_add(y, weight, eps, x, cast=None):
 def rmsnorm_add(y, weight, eps, mult, x, cast=None, bias=None, pair=None):
     """x[r] += mult * (y[r] / sqrt(mean(y[r]^2) + eps) * weight), x float32 [R, H], y in the activation dtype; `cast`
     (same dtype as y, or None) receives the new x.  `bias` (float32 [H] or None) is added to every row of y first.
-    `pair` = (y2, s1, s2): the normed row is s1 * y + s2 * y2 (the results of two sub-layers side by side), in float32."""
-    y2, s1, s2 = pair if pair is not None else (None, 1.0, 0.0)
+    `pair` = (y2, s1, s2): the normed row is s1 * y + s2 * y2 (the results of two sub-layers side by side), in float32; with
+    `pair` = (y2, s1, s2, w1, w2) each of the two is first divided by its own root mean square and multiplied by its weight."""
+    y2, s1, s2, w1, w2 = (tuple(pair) + (None, None))[:5] if pair is not None else (None, 1.0, 0.0, None, None)
+    for w in (w1, w2):
+        if w is not None:
+            _need(w, torch.float32, "pair weight", 1)
+            if w.shape[0] != x.shape[1]:
+                raise KernelError("rmsnorm_add: the weights of a pair have one entry per column")
     if y2 is not None:
         _need(y2, y.dtype, "y2", 2)
         if y2.shape != y.shape:
@@ -864,7 +924,8 @@ def rmsnorm_add(y, weight, eps, mult, x, cast=None, bias=None, pair=None):
         if bias.shape[0] != x.shape[1]:
             raise KernelError("rmsnorm_add: the bias has one entry per column")
     _check(_fn("embed_norm", "vl_rmsnorm_add")(_ptr(y), dtype_code(y.dtype), _ptr(bias), _ptr(weight), float(eps), float(mult), _ptr(x),
-                                               _ptr(cast), x.shape[0], x.shape[1], _ptr(y2), float(s1), float(s2), _stream()),
+                                               _ptr(cast), x.shape[0], x.shape[1], _ptr(y2), float(s1), float(s2), _ptr(w1), _ptr(w2),
+                                               _stream()),
            "vl_rmsnorm_add")
     return x
 
@@ -970,15 +1031,15 @@ def sigmoid_gate(x, gate, gate_col=0):
 
 
 def gemm_heads(a, w, out):
-    """One product per head on column slices: a [T, H*K], w [H, N, K], out [T, H*N];
+    """One product per head on column slices: a [T, H*K], w [H, N, K], out [T, H*N] (in a's dtype, or float32);
     out[:, h*N:(h+1)*N] = a[:, h*K:(h+1)*K] @ w[h]^T.  float32 accumulation in a fixed order over K."""
-    _need(a, None, "a", 2); _need(w, a.dtype, "w", 3); _need(out, a.dtype, "out", 2)
+    _need(a, None, "a", 2); _need(w, a.dtype, "w", 3); _need(out, None, "out", 2)
     H, N, K = w.shape
     T = a.shape[0]
     if a.shape[1] != H * K or out.shape != (T, H * N):
         raise KernelError(f"gemm_heads: shapes disagree a{tuple(a.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
     _check(_fn("gemm_batched", "vl_gemm_batched_nt")(
-        _ptr(a), _ptr(w), _ptr(out), dtype_code(a.dtype), T, N, K, H * K, K, H * N, K, N * K, N, H, None, 0,
+        _ptr(a), _ptr(w), _ptr(out), dtype_code(a.dtype), dtype_code(out.dtype), T, N, K, H * K, K, H * N, K, N * K, N, H, None, 0,
         16 if T <= 16 else 64, _stream()), "vl_gemm_batched_nt")
     return out
 
@@ -993,7 +1054,7 @@ def gemm_grouped(rows, w, out, tile_group, bm):
     if rows.shape[1] != K or out.shape != (cap, N) or cap % bm or tile_group.shape[0] < cap // bm:
         raise KernelError("gemm_grouped: shapes disagree")
     _check(_fn("gemm_batched", "vl_gemm_batched_nt")(
-        _ptr(rows), _ptr(w), _ptr(out), dtype_code(rows.dtype), cap, N, K, K, K, N, 0, 0, 0, 1, _ptr(tile_group), N * K,
+        _ptr(rows), _ptr(w), _ptr(out), dtype_code(rows.dtype), dtype_code(rows.dtype), cap, N, K, K, K, N, 0, 0, 0, 1, _ptr(tile_group), N * K,
         int(bm), _stream()), "vl_gemm_batched_nt")
     return out
 
@@ -1051,7 +1112,7 @@ def router_slices(K) -> int:
 
 
 def moe_route(h, router, top, ids, weights, logits, score="sigmoid", renormalize=False, groups=1, keep_groups=1, bias=None,
-              choice_bias=None, group_top=1, renorm_eps=0.0):
+              choice_bias=None, group_top=1, renorm_eps=0.0, extra_out=None):
     """h [T, K], router [E, K] (float32; or bfloat16 as stored, beside bfloat16 rows: products of two bfloat16 numbers
     are exact in float32, so the tensor cores' float32 sums are the 32-bit logits of the rounded rows):
     logits float32 [router_slices(K), T, E] = partial sums of h router^T; ids int32 [T, top] = the experts with
@@ -1061,18 +1122,24 @@ def moe_route(h, router, top, ids, weights, logits, score="sigmoid", renormalize
     `bias` (float32 [E]) is added to the logits before anything else.  "softmax" with `renormalize` is the softmax
     over the chosen logits alone.  `choice_bias` (float32 [E]): experts and groups are chosen by score + choice_bias
     instead (the weights stay the scores without it); `group_top`: a group counts by the sum of that many of its largest
-    choice values; `renorm_eps` is added to the sum that `renormalize` divides by."""
+    choice values; `renorm_eps` is added to the sum that `renormalize` divides by.
+    `extra_out` (float32 [T]): the router has one more row behind the experts', the sigmoid of its product goes there."""
     _need(h, None, "h", 2); _need(router, None, "router", 2); _need(logits, torch.float32, "logits", 3)
     if router.dtype != torch.float32 and router.dtype != h.dtype:
         raise KernelError("moe_route: the router is float32, or bfloat16 beside bfloat16 rows")
     _need(ids, torch.int32, "ids", 2); _need(weights, torch.float32, "weights", 2)
     T, K = h.shape
-    E = router.shape[0]
+    rows = router.shape[0]
+    E = rows if extra_out is None else rows - 1
     slices = router_slices(K)
-    if router.shape[1] != K or ids.shape != (T, top) or weights.shape != (T, top) or logits.shape != (slices, T, E):
+    if extra_out is not None:
+        _need(extra_out, torch.float32, "extra_out", 1)
+        if extra_out.shape[0] != T or E <= 0:
+            raise KernelError("moe_route: extra_out has one number per token")
+    if router.shape[1] != K or ids.shape != (T, top) or weights.shape != (T, top) or logits.shape != (slices, T, rows):
         raise KernelError("moe_route: shapes disagree (logits: [router_slices(K), T, E])")
     _check(_fn("gemm_batched", "vl_gemm_rows_f32w")(_ptr(h), dtype_code(h.dtype), _ptr(router), dtype_code(router.dtype),
-                                                    _ptr(logits), T, E, K, slices, _stream()), "vl_gemm_rows_f32w")
+                                                    _ptr(logits), T, rows, K, slices, _stream()), "vl_gemm_rows_f32w")
     if groups < 1 or E % groups or not 1 <= keep_groups <= groups or keep_groups * (E // groups) < top:
         raise KernelError(f"moe_route: {E} experts in {groups} groups, {keep_groups} kept, top {top}")
     if bias is not None:
@@ -1083,9 +1150,9 @@ def moe_route(h, router, top, ids, weights, logits, score="sigmoid", renormalize
         _need(choice_bias, torch.float32, "choice_bias", 1)
         if choice_bias.shape[0] != E:
             raise KernelError(f"moe_route: the choice bias has {choice_bias.shape[0]} entries for {E} experts")
-    _check(_fn("moe", "vl_moe_route")(_ptr(logits), slices, T, E, int(top), ROUTER_SCORES[score], int(bool(renormalize)),
+    _check(_fn("moe", "vl_moe_route")(_ptr(logits), slices, T, E, rows, int(top), ROUTER_SCORES[score], int(bool(renormalize)),
                                       int(groups), int(keep_groups), _ptr(bias), _ptr(choice_bias), int(group_top),
-                                      float(renorm_eps), _ptr(ids), _ptr(weights), _stream()),
+                                      float(renorm_eps), _ptr(ids), _ptr(weights), _ptr(extra_out), _stream()),
            "vl_moe_route")
 
 
@@ -1135,9 +1202,10 @@ def moe_gather(h, sorted_rows, weights, top, rows, scale_input):
     return rows
 
 
-def moe_combine(result, place, weights, top, out, scale_output, add=None):
+def moe_combine(result, place, weights, top, out, scale_output, add=None, add_weight=None, ids=None, identity_from=0, h=None):
     """out[t] = the sum over token t's choices (in their order) of (weight *) result[place[t, j]]; `add` [T, N]: one more
-    row per token, added last (a feed-forward that every token passes)."""
+    row per token, added last (a feed-forward that every token passes), times add_weight[t] (float32 [T]) when given.
+    `h` [T, N] with `ids`: a choice whose expert is `identity_from` or more gives the token's own row h[t]."""
     _need(result, None, "result", 2); _need(out, result.dtype, "out", 2); _need(weights, torch.float32, "weights")
     T, N = out.shape
     if result.shape[1] != N or place.shape[0] < T * top:
@@ -1146,8 +1214,17 @@ def moe_combine(result, place, weights, top, out, scale_output, add=None):
         _need(add, out.dtype, "add", 2)
         if add.shape != out.shape:
             raise KernelError("moe_combine: the added rows have the output's shape")
+    if add_weight is not None:
+        _need(add_weight, torch.float32, "add_weight", 1)
+        if add is None or add_weight.shape[0] != T:
+            raise KernelError("moe_combine: a weight per token for the added rows")
+    if h is not None:
+        _need(h, out.dtype, "h", 2); _need(ids, torch.int32, "ids", 2)
+        if h.shape != out.shape or ids.shape != (T, top):
+            raise KernelError("moe_combine: the rows of identity experts have the output's shape")
     _check(_fn("moe", "vl_moe_combine")(_ptr(result), dtype_code(result.dtype), _ptr(place), _ptr(weights), T, int(top), N,
-                                        int(bool(scale_output)), _ptr(out), _ptr(add), _stream()), "vl_moe_combine")
+                                        int(bool(scale_output)), _ptr(out), _ptr(add), _ptr(add_weight), _ptr(ids),
+                                        int(identity_from), _ptr(h), _stream()), "vl_moe_combine")
     return out
 
 
@@ -1410,14 +1487,14 @@ def _seg_args(cu, slots):
 
 
 def short_conv(x, col0, C, weight, bias, state, state_off, cu, slots, out, act=True, longest=None, in_bias=None):
-    """out float32 [T, C] = act(causal convolution over time of columns col0 .. col0+C of x [T, ld]); weight float32
+    """out [T, C] (float32 or x's dtype) = act(causal convolution over time of columns col0 .. col0+C of x [T, ld]); weight float32
     [C, taps]; the last taps-1 inputs live at `state_off` of every request's state row [(taps-1), C].  `longest`: a
     bound on the tokens one request brings (default: all of them).  `in_bias` (float32 [C] or None) is added to the
     rows of x as they are read, before the convolution; the state keeps them with it."""
     _need(x, None, "x", 2); _need(weight, torch.float32, "weight", 2)
     taps = weight.shape[1]
     if out is not None:                         # None: only the new state is made (the rows were computed elsewhere)
-        _need(out, torch.float32, "out", 2)
+        _need(out, None, "out", 2)
     if weight.shape[0] != C or (out is not None and out.shape != (x.shape[0], C)):
         raise KernelError("short_conv: shapes disagree")
     for t, n in ((bias, "bias"), (in_bias, "in_bias")):
@@ -1430,7 +1507,7 @@ def short_conv(x, col0, C, weight, bias, state, state_off, cu, slots, out, act=T
     _check(_fn("recurrent", "vl_short_conv")(_ptr(x), dtype_code(x.dtype), x.shape[1], col0, C, _ptr(weight), _ptr(bias),
                                              _ptr(in_bias), taps,
                                              sp, stride, _ptr(cu), _ptr(slots), B, int(longest or max(x.shape[0], 1)), _ptr(out),
-                                             int(bool(act)), _stream()), "vl_short_conv")
+                                             dtype_code(out.dtype) if out is not None else F32, int(bool(act)), _stream()), "vl_short_conv")
     if out is not None and int(longest or x.shape[0]) > 64:
         global launch_count
         launch_count += 1           # requests cut among blocks: the new state is a launch of its own
@@ -1575,4 +1652,101 @@ def gate_norm(y, gate, gate_col, gate_kind, gate_first, weight, eps, out, part):
     _check(_fn("recurrent", "vl_gate_norm")(_ptr(y), _ptr(gate), dtype_code(out.dtype), ld, gate_col, GATES[gate_kind if gate is not None else None],
                                             int(bool(gate_first)), _ptr(weight), weight.shape[0], float(eps), _ptr(out), T, W,
                                             part, _stream()), "vl_gate_norm")
+    return out
+
+
+# ---------------------------------------------------------------- head work, maps, element-wise recurrences
+def head_work(rows, bias, positions, slots, q_weight, k_weight, eps, rotary, q_factor, q_out, k_cache, v_cache, num_heads,
+              num_kv_heads, maps, dim, vdim, err, whole=False, true_dim=None):
+    """The head work of an attention (csrc/head_work.cu): rows [T, >= (nq + nkv) maps dim + nkv vdim] = q | k | v (plus
+    `bias`), a norm per map of a head (weights float32 [dim]) or over all of q and all of k (`whole`; weights of all their
+    columns), the rotation of neighbours (2i, 2i + 1) by `rotary` = (inv_freq, rot), query head h times q_factor[h]; q to
+    q_out [T, nq maps, P] (map m at feature m dim, zeros elsewhere), [k_1 .. k_maps | 0] and [v | 0] to the caches
+    [pages, nkv, page_size, P] at `slots`.  k_cache None: rows hold q alone (a call that reads another call's cache).
+    dim and vdim are multiples of 8; `true_dim` (default dim) counts the features that are not padding."""
+    _need(rows, None, "rows", 2); _need(positions, torch.int32, "positions", 1); _need(q_out, rows.dtype, "q_out", 3)
+    T = rows.shape[0]
+    P = q_out.shape[2]
+    n = int(true_dim or dim)
+    has_kv = k_cache is not None
+    width = num_heads * maps * dim + (num_kv_heads * (maps * dim + vdim) if has_kv else 0)
+    if rows.shape[1] < width or rows.shape[1] % 8 or positions.shape[0] != T or q_out.shape[:2] != (T, num_heads * maps):
+        raise KernelError(f"head_work: rows {tuple(rows.shape)}, q_out {tuple(q_out.shape)}; {width} columns are wanted")
+    if bias is not None:
+        _need(bias, torch.float32, "bias", 1)
+        if bias.shape[0] < width:
+            raise KernelError("head_work: the bias has one entry per column")
+    if (q_weight is None) != (k_weight is None):
+        raise KernelError("head_work: norms on q and k come together")
+    if q_weight is not None:
+        _need(q_weight, torch.float32, "q_weight", 1); _need(k_weight, torch.float32, "k_weight", 1)
+        if q_weight.shape[0] != (num_heads * dim if whole else dim) or k_weight.shape[0] != (num_kv_heads * dim if whole else dim):
+            raise KernelError("head_work: the norm weights do not match")
+    if q_factor is not None:
+        _need(q_factor, torch.float32, "q_factor", 1)
+        if q_factor.shape[0] != num_heads:
+            raise KernelError("head_work: q_factor has one number per query head")
+    inv_freq, rot = rotary if rotary is not None else (None, 0)
+    if inv_freq is not None:
+        _need(inv_freq, torch.float32, "inv_freq", 1)
+        if inv_freq.shape[0] * 2 != rot or rot > n:
+            raise KernelError("head_work: inv_freq must have rot / 2 entries, rot at most the head size")
+    page_size, num_slots = 1, 0
+    if has_kv:
+        _need(k_cache, rows.dtype, "k_cache", 4); _need(v_cache, rows.dtype, "v_cache", 4)
+        if k_cache.shape != v_cache.shape or k_cache.shape[1] != num_kv_heads or k_cache.shape[3] != P:
+            raise KernelError(f"cache {tuple(k_cache.shape)} does not match kv heads {num_kv_heads} x {P}")
+        _need(slots, torch.int32, "slots", 1)
+        if slots.shape[0] != T:
+            raise KernelError("head_work: one slot per token")
+        page_size = k_cache.shape[2]
+        num_slots = k_cache.shape[0] * page_size
+    _check(_fn("head_work", "vl_head_work")(
+        _ptr(rows), rows.shape[1], dtype_code(rows.dtype), _ptr(bias), _ptr(positions), _ptr(slots) if has_kv else None, _ptr(q_weight),
+        _ptr(k_weight), float(eps), int(bool(whole)), n, num_heads * n, num_kv_heads * n, _ptr(inv_freq), int(rot), _ptr(q_factor),
+        _ptr(q_out), _ptr(k_cache), _ptr(v_cache), T, num_heads, num_kv_heads, maps, dim, vdim, P, int(has_kv), page_size, num_slots,
+        _ptr(err), _stream()), "vl_head_work")
+    return q_out
+
+
+def combine_maps(a, lam, factor, eps, true_vdim, out):
+    """a [T, 2 nq, P] (map m of head h in row 2 h + m), out [T, nq * V]: (a_1 - lam a_2) divided by its root mean square over
+    `true_vdim` features (eps inside the root), times `factor`; V a multiple of 8."""
+    _need(a, None, "a", 3); _need(out, a.dtype, "out", 2)
+    T, maps, P = a.shape
+    V = out.shape[1] // (maps // 2)
+    if maps % 2 or out.shape != (T, maps // 2 * V):
+        raise KernelError("combine_maps: two maps per head, out [T, heads * V]")
+    _check(_fn("head_work", "vl_combine_maps")(_ptr(a), _ptr(out), dtype_code(a.dtype), float(lam), float(factor), float(eps), int(true_vdim),
+                                               T * (maps // 2), P, V, _stream()), "vl_combine_maps")
+    return out
+
+
+LINEAR_SCANS = {"min_gru": 0, "gated_lru": 1}
+
+
+def linear_scan(kind, proj, biases, state, state_off, cu, slots, out, conv=None, gates=None, block=0, decay=None, longest=None):
+    """S_t = a_t S_(t-1) + b_t per channel from state[slot, state_off : state_off + C] (float32), out [T, C] = S * gate; a, b
+    and the gate as csrc/linear_scan.cu makes them.  "min_gru": proj [T, >= 3 C] = z | x | g, biases (z, x).  "gated_lru":
+    proj [T, >= C] = y first, conv [T, C], gates float32 [T, 2 C] in blocks of `block`, biases (r, i, y), decay float32 [C]."""
+    _need(proj, None, "proj", 2); _need(out, proj.dtype, "out", 2)
+    T, C = out.shape
+    if kind not in LINEAR_SCANS or proj.shape[0] != T:
+        raise KernelError(f"linear_scan: kind {kind!r} / shapes disagree")
+    biases = tuple(biases) + (None,) * (3 - len(biases))
+    for t, n in tuple(zip(biases, ("bias 0", "bias 1", "bias 2"))) + ((decay, "decay"),):
+        if t is not None:
+            _need(t, torch.float32, n, 1)
+            if t.shape[0] != C:
+                raise KernelError(f"linear_scan: {n} has one entry per channel")
+    if kind == "gated_lru":
+        _need(conv, proj.dtype, "conv", 2); _need(gates, torch.float32, "gates", 2)
+        if conv.shape != (T, C) or gates.shape != (T, 2 * C) or decay is None:
+            raise KernelError("linear_scan: conv [T, C], gates [T, 2 C], decay [C]")
+    B = _seg_args(cu, slots)
+    sp, stride = _state_args(state, state_off, C)
+    _check(_fn("linear_scan", "vl_linear_scan")(
+        LINEAR_SCANS[kind], _ptr(proj), proj.shape[1], dtype_code(proj.dtype), _ptr(conv), C, _ptr(gates), 2 * C, int(block), _ptr(biases[0]),
+        _ptr(biases[1]), _ptr(biases[2]), _ptr(decay), sp, stride, _ptr(cu), _ptr(slots), B, int(longest or max(T, 1)), _ptr(out), C,
+        _stream()), "vl_linear_scan")
     return out

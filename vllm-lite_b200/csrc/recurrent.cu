@@ -77,11 +77,11 @@ static inline bool scan_shape(int N, int P, ScanShape* sh) {
 // the state it rewrites); mode 1: outputs only; mode 2: the new state only (a launch of its own after mode 1, when
 // requests are cut among several blocks: the blocks that read the old state must have finished).
 #define CONV_TOKENS 64
-template <typename TP>
+template <typename TP, typename TO>
 __global__ void __launch_bounds__(256)
 short_conv_kernel(const TP* __restrict__ in, int ld, int col0, int C, const float* __restrict__ w,
                   const float* __restrict__ bias, const float* __restrict__ in_bias, int taps, float* __restrict__ state,
-                  long long state_stride, const int* __restrict__ cu, const int* __restrict__ slots, float* __restrict__ out,
+                  long long state_stride, const int* __restrict__ cu, const int* __restrict__ slots, TO* __restrict__ out,
                   int act, int mode) {
     pdl_launch_dependents();
     pdl_wait();
@@ -103,7 +103,7 @@ short_conv_kernel(const TP* __restrict__ in, int ld, int col0, int C, const floa
                 const float v = at >= 0 ? to_f32(in[(size_t)(s0 + at) * ld + col0 + c]) + ib : st[(size_t)(at + back) * C + c];
                 acc += w[(size_t)c * taps + j] * v;
             }
-            out[(size_t)(s0 + t) * C + c] = act ? silu_f(acc) : acc;
+            out[(size_t)(s0 + t) * C + c] = from_f32<TO>(act ? silu_f(acc) : acc);
         }
     }
     if (mode == 1) return;
@@ -118,9 +118,10 @@ short_conv_kernel(const TP* __restrict__ in, int ld, int col0, int C, const floa
 
 extern "C" int vl_short_conv(const void* in, int dtype, int ld, int col0, int C, const float* w, const float* bias,
                              const float* in_bias, int taps, float* state, long long state_stride, const int* cu, const int* slots,
-                             int B, int longest, float* out, int act, void* stream) {
+                             int B, int longest, void* out, int out_dtype, int act, void* stream) {
     if (B <= 0 || C <= 0) return VL_OK;
     if (taps <= 0 || col0 < 0 || col0 + C > ld || longest <= 0) return VL_ERR_ARGUMENT;
+    if (out && out_dtype != VL_F32 && out_dtype != dtype) return VL_ERR_UNSUPPORTED;       // float32, or the dtype of the rows
     cudaStream_t s = (cudaStream_t)stream;
     const int cuts = (longest + CONV_TOKENS - 1) / CONV_TOKENS;
     // without `out` only the new state is made (the caller computed the rows itself, from the old state)
@@ -129,11 +130,14 @@ extern "C" int vl_short_conv(const void* in, int dtype, int ld, int col0, int C,
         dim3 grid((C + 31) / 32, B, mode == 1 ? cuts : 1), block(32, 8);
         int rc;
         if (dtype == VL_F32)
-            rc = vl_launch(short_conv_kernel<float>, grid, block, 0, s, (const float*)in, ld, col0, C, w, bias, in_bias, taps, state,
-                           state_stride, cu, slots, out, act, mode);
+            rc = vl_launch(short_conv_kernel<float, float>, grid, block, 0, s, (const float*)in, ld, col0, C, w, bias, in_bias, taps, state,
+                           state_stride, cu, slots, (float*)out, act, mode);
+        else if (dtype == VL_BF16 && out_dtype == VL_BF16)
+            rc = vl_launch(short_conv_kernel<bf16, bf16>, grid, block, 0, s, (const bf16*)in, ld, col0, C, w, bias, in_bias, taps, state,
+                           state_stride, cu, slots, (bf16*)out, act, mode);
         else if (dtype == VL_BF16)
-            rc = vl_launch(short_conv_kernel<bf16>, grid, block, 0, s, (const bf16*)in, ld, col0, C, w, bias, in_bias, taps, state,
-                           state_stride, cu, slots, out, act, mode);
+            rc = vl_launch(short_conv_kernel<bf16, float>, grid, block, 0, s, (const bf16*)in, ld, col0, C, w, bias, in_bias, taps, state,
+                           state_stride, cu, slots, (float*)out, act, mode);
         else
             return VL_ERR_UNSUPPORTED;
         if (rc) return rc;

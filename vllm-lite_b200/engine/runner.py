@@ -21,7 +21,7 @@ from ..cache import make_cache_manager
 from ..cache.manager import CacheLayout, OutOfPages
 from ..cache.storage import CacheStorage
 from ..parts.base import QUERY_TILE, BuildContext, Entry, GroupView, StepBatch, Workspace
-from ..parts.model import CausalLM, cache_needs
+from ..parts.model import CausalLM, cache_needs, cache_sources
 
 
 class StepError(RuntimeError):
@@ -85,7 +85,7 @@ class ModelRunner:
         self.page_size = int(page_size)
         torch.cuda.set_device(self.device)
         self.model = CausalLM(plan, weights, BuildContext(self.device, dtype))
-        self.layout = CacheLayout.from_needs(cache_needs(plan), [c.cache_of for c in plan.order])
+        self.layout = CacheLayout.from_needs(cache_needs(plan), cache_sources(plan))
         self.max_context = int(max_context or plan.max_position_embeddings)
         if own_weights:
             weights.clear()

@@ -53,6 +53,21 @@ def _pair_order(head_dim, rotary_dim, device):
     return idx
 
 
+def neighbour_order(size, rotary_dim, interleaved, device):
+    """The order of a head's features that puts the pairs a rotation turns side by side, (2i, 2i + 1), where the head-work
+    kernel (`ops.head_work`) wants them: pairs (i, i + rotary_dim/2) move, interleaved ones lie so already.  q.k does not
+    change when q and k are permuted alike."""
+    idx = torch.arange(size, device=device)
+    if not interleaved:
+        half = rotary_dim // 2
+        idx[:rotary_dim] = torch.stack([torch.arange(half, device=device), torch.arange(half, rotary_dim, device=device)], dim=1).reshape(-1)
+    return idx
+
+
+def round_up(n, to):
+    return -(-n // to) * to
+
+
 @MIXERS.register("gqa_attention")
 class GqaAttention:
     graph_safe = True          # launches only stream-ordered kernels: a step can be captured in a CUDA graph
@@ -74,7 +89,13 @@ class GqaAttention:
                       spec.distance_bias[1]: TensorDecl((spec.num_heads,), init="rate")})
         if spec.gate is not None:
             d[spec.gate] = TensorDecl((spec.num_heads * vd, spec.hidden_size))
-        if spec.qk_norm is not None:
+        for name in (spec.head_temp, spec.sink):
+            if name is not None:
+                d[name] = TensorDecl((spec.num_heads,), init="norm" if name == spec.head_temp else "unit")
+        if spec.qk_norm is not None and spec.whole_norm:
+            for side, rows in zip(spec.norm_prefixes, (qd, kd)):
+                d[side + spec.qk_norm.tensor] = TensorDecl((rows,), init="norm")
+        elif spec.qk_norm is not None:
             for side in spec.norm_prefixes:
                 for name, decl in NORMS.get(spec.qk_norm.kind).declare(spec.qk_norm).items():
                     d[side + name] = decl
@@ -92,7 +113,8 @@ class GqaAttention:
 
     @staticmethod
     def cache_need(spec: AttentionSpec):
-        return PagedKV(spec.num_kv_heads, GqaAttention.padded_head_dim(spec), spec.window)
+        return PagedKV(spec.num_kv_heads, GqaAttention.padded_head_dim(spec), spec.window,
+                       keep=spec.keep_first if spec.window is not None else None)
 
     def __init__(self, spec: AttentionSpec, weights: dict, ctx):
         import dataclasses
@@ -101,8 +123,18 @@ class GqaAttention:
         # an attention with options on its scores or around them runs its own sequence of kernels (`_call_with_options`);
         # with a query factor or a value norm the head work is a kernel of its own, which knows the heads' true sizes
         self.own_head_work = spec.q_temp is not None or spec.v_norm is not None
-        self.with_options = bool(self.own_head_work or spec.softcap or spec.distance_bias is not None or spec.unit_sink
-                                 or spec.gate is not None)
+        # ... and so is it with a norm over the whole projection or a factor per head (`ops.head_work`: bias, norm, rotation,
+        # factor and the cache rows in one pass, from rows of unpadded heads)
+        self.row_work = bool(spec.whole_norm or spec.head_temp is not None)
+        self.with_options = bool(self.own_head_work or self.row_work or spec.softcap or spec.distance_bias is not None
+                                 or spec.unit_sink or spec.sink is not None or spec.keep_first or spec.gate is not None)
+        if self.row_work and (self.own_head_work or (spec.qk_norm is not None and (spec.qk_norm.kind != "rms_norm" or spec.qk_norm.offset
+                                                     or spec.qk_norm.scalar or not spec.qk_norm.has_weight))):
+            raise ValueError("a whole-row norm or a factor per head goes with plain RMS norms, no query factor and no value norm")
+        if spec.whole_norm and spec.qk_norm is None:
+            raise ValueError("whole_norm says where qk_norm runs; there is none")
+        if spec.unit_sink and spec.sink is not None:
+            raise ValueError("a sink of score 0 and a learned one")
         if self.own_head_work and (spec.position is not None or spec.bias or
                                    (spec.qk_norm is not None and spec.qk_norm.kind != "rms_norm")):
             raise ValueError("a query factor or a value norm goes with RMS head norms, no rotation and no projection bias")
@@ -113,6 +145,10 @@ class GqaAttention:
         check_attention_sizes(spec)
         self.spec = spec
         self.dtype = ctx.dtype
+        self.scale = spec.scale
+        if self.row_work:
+            self._bind_row_work(weights, ctx)
+            return
         nq, nkv = spec.num_heads, spec.num_kv_heads
         qn, kn, vn, on = spec.names
         wq, wk, wv, wo = weights[qn], weights[kn], weights[vn], weights[on]
@@ -146,7 +182,7 @@ class GqaAttention:
         self.distance = None
         if spec.distance_bias is not None:
             self.distance = (f32(weights[spec.distance_bias[0]]), f32(weights[spec.distance_bias[1]]))
-        self.sinks = torch.zeros(nq, dtype=torch.float32, device=ctx.device) if spec.unit_sink else None
+        self.sinks = self._sinks(weights, ctx)
         self.o_proj = Linear(wo.contiguous(), weights[spec.bias_names[3]].float() if spec.out_bias else None)
         self.q_norm = self.k_norm = None
         # The kernel that rotates and writes the cache also applies an RMS norm to every head.  A head norm
@@ -189,7 +225,58 @@ class GqaAttention:
             pos = dataclasses.replace(spec.position, head_dim=pd, rotary_dim=spec.position.dim, interleaved=False) \
                 if hasattr(spec.position, "rotary_dim") else spec.position
             self.position = POSITIONS.get(pos.kind)(pos, sub_weights(weights, "rotary."), ctx)
-        self.scale = spec.scale
+
+    def _sinks(self, weights, ctx):
+        s = self.spec
+        if s.sink is not None:
+            return weights[s.sink].to(device=ctx.device, dtype=torch.float32).contiguous()
+        return torch.zeros(s.num_heads, dtype=torch.float32, device=ctx.device) if s.unit_sink else None
+
+    def _bind_row_work(self, weights, ctx):
+        """Weights for `ops.head_work`: rows of q, k and v with heads rounded up to 8 features (the kernel lays them out in
+        the attention's padded heads), the pairs of the rotation side by side; a gate's rows follow the padded heads."""
+        s, ts = self.spec, self.true_spec
+        nq, nkv, hd, vd, pd = s.num_heads, s.num_kv_heads, ts.head_dim, ts.v_head_dim or ts.head_dim, s.head_dim
+        self.D, self.V = round_up(hd, 8), round_up(vd, 8)
+        f32 = lambda t: t.to(device=ctx.device, dtype=torch.float32).contiguous()
+        rot = ts.position
+        order = neighbour_order(hd, rot.dim if rot is not None else 0, rot is None or rot.interleaved, weights[s.names[0]].device)
+        heads = lambda t, n: _pad_heads(t.reshape((n, hd) + tuple(t.shape[1:]))[:, order].reshape(t.shape), n, hd, self.D)
+        parts = [heads(weights[s.names[0]], nq), heads(weights[s.names[1]], nkv), _pad_heads(weights[s.names[2]], nkv, vd, self.V)]
+        self.row_bias = None
+        if s.bias:
+            qb, kb, vb = (weights[n].float() for n in s.bias_names[:3])
+            self.row_bias = f32(torch.cat([heads(qb, nq), heads(kb, nkv), _pad_heads(vb, nkv, vd, self.V)]))
+        self.gate_col = None
+        if s.gate is not None:
+            self.gate_col = sum(p.shape[0] for p in parts)
+            parts.append(_pad_heads(weights[s.gate], nq, vd, pd))
+        self.qkv_proj = Linear(torch.cat(parts, dim=0).contiguous())
+        wo = weights[s.names[3]]
+        if vd != pd:
+            wo = _pad_heads(wo.t().contiguous(), nq, vd, pd).t()
+        self.o_proj = Linear(wo.contiguous(), weights[s.bias_names[3]].float() if s.out_bias else None)
+        self.head_weights = (None, None)
+        if s.qk_norm is not None:
+            qw, kw = (f32(weights[side + s.qk_norm.tensor]) for side in s.norm_prefixes)
+            self.head_weights = (heads(qw, nq), heads(kw, nkv)) if s.whole_norm else (heads(qw, 1), heads(kw, 1))
+            self.head_weights = tuple(w.contiguous() for w in self.head_weights)
+        self.q_factor = f32(weights[s.head_temp]) if s.head_temp is not None else None
+        self.distance = None
+        if s.distance_bias is not None:
+            self.distance = (f32(weights[s.distance_bias[0]]), f32(weights[s.distance_bias[1]]))
+        self.sinks = self._sinks(weights, ctx)
+        self.rotary = None
+        if rot is not None:
+            table = POSITIONS.get(rot.kind)(rot, sub_weights(weights, "rotary."), ctx)
+            self.rotary = table.fused_rotary()
+            if self.rotary is None:
+                raise TypeError(f"position kind {rot.kind!r} offers no table of frequencies to the head-work kernel")
+
+    def take_out_bias(self):
+        """Hands the output projection's bias to the caller (a block whose norm reads the product anyway)."""
+        bias, self.o_proj.bias = self.o_proj.bias, None
+        return bias
 
     def factors_norms(self, M) -> bool:
         """For M rows: the input may come as `ScaledRows` and the result may go `into_stream`."""
@@ -203,7 +290,13 @@ class GqaAttention:
         group = step.groups[cache.group]
         qkv = self.qkv_proj(h, step, "attn.qkv")
         slots = group.slots if cache.writes else None
-        if self.own_head_work:
+        if self.row_work:
+            q = step.workspace.get(step.tag + "attn.q", (qkv.shape[0], s.num_heads, s.head_dim), self.dtype)
+            ops.head_work(qkv, self.row_bias, step.positions, slots, self.head_weights[0], self.head_weights[1],
+                          ts.qk_norm.eps if ts.qk_norm is not None else 0.0, self.rotary, self.q_factor, q, cache.k, cache.v,
+                          s.num_heads, s.num_kv_heads, 1, self.D, self.V, step.err, whole=ts.whole_norm, true_dim=ts.head_dim)
+            q = q.view(qkv.shape[0], s.num_heads * s.head_dim)
+        elif self.own_head_work:
             qk = ts.qk_norm
             ops.head_norm_write(qkv, step.positions, slots, self.head_weights[0], self.head_weights[1],
                                 qk.eps if qk is not None else 0.0, ts.head_dim if qk is not None else 0,
@@ -221,8 +314,8 @@ class GqaAttention:
             ops.qk_norm_rope_write(qkv, step.positions, slots, qw, kw, eps, inv_freq, rot, cache.k, cache.v,
                                    s.num_heads, s.num_kv_heads, s.head_dim, step.err)
         out = step.workspace.get(step.tag + "attn.out", (qkv.shape[0], s.num_heads * s.head_dim), self.dtype)
-        attention_dispatch.run(qkv, out, cache, group, step, s, self.scale, sinks=self.sinks, softcap=ts.softcap,
-                               distance=self.distance)
+        attention_dispatch.run(q if self.row_work else qkv, out, cache, group, step, s, self.scale, sinks=self.sinks,
+                               softcap=ts.softcap, distance=self.distance, keep=ts.keep_first)
         if self.gate_col is not None:
             ops.sigmoid_gate(out, qkv, self.gate_col)
         return self.o_proj(out, step, "attn.o")

@@ -70,8 +70,14 @@ def _variant_decode_ok(ops, spec, num_tokens, max_context, mask_chunk) -> bool:
     return -(-int(max_context) // chunk) <= ops.flash_decode_own_merge_cap(spec.head_dim)
 
 
+def _merges_itself(ops, spec, num_tokens, max_keys) -> bool:
+    """Whether the block-per-chunk kernel merges the chunks of so many keys itself, which kept keys ask for."""
+    chunk = ops.decode_chunk_for(num_tokens, spec.num_kv_heads, max_keys, head_dim=spec.head_dim)
+    return -(-int(max_keys) // chunk) <= ops.flash_decode_own_merge_cap(spec.head_dim)
+
+
 def run(qkv, out, cache, group, step, spec, scale, fold=None, sinks=None, weighting="softmax", chunk=None,
-        head_bias=None, gate=None, softcap=None, distance=None):
+        head_bias=None, gate=None, softcap=None, distance=None, keep=None):
     """`spec`: anything with num_heads, num_kv_heads, head_dim and window.
     `fold` (only where `folds_head_work` said so): (q_weight, k_weight, eps, inv_freq, rotary_dim, slots) of the
     head work that the mixer left undone.
@@ -80,11 +86,13 @@ def run(qkv, out, cache, group, step, spec, scale, fold=None, sinks=None, weight
     itself; `chunk`: positions in blocks of that many, no key of an earlier block is read; `gate` [T, >= num_heads]:
     head h's output is multiplied by sigmoid(gate[t, h]).
     `softcap` c: score <- c tanh(score / c); `distance` (a, b), float32 [num_heads] each: a[h] ln(1 + b[h] (i - j)) is
-    taken off the score of the key j that query i reads."""
+    taken off the score of the key j that query i reads; `keep`: beside the window, the first `keep` keys stay visible."""
     from ..csrc import ops
-    if softcap or distance is not None:
+    if not spec.window:
+        keep = None
+    if softcap or distance is not None or keep:
         return _run_shaped(ops, qkv, out, cache, group, step, spec, scale, sinks, weighting, chunk, head_bias, gate,
-                           softcap, distance)
+                           softcap, distance, keep)
     if weighting != "softmax" or chunk is not None or head_bias is not None or gate is not None:
         return _run_variant(ops, qkv, out, cache, group, step, spec, scale, weighting, chunk, head_bias, gate, sinks)
     if fold is not None and not folds_head_work(qkv.dtype, step, spec, group, qkv.shape[0]):
@@ -137,19 +145,26 @@ def _run_variant(ops, q, out, cache, group, step, spec, scale, weighting, chunk,
                                weighting=weighting, chunk=chunk, head_bias=head_bias, gate=gate)
 
 
-def _run_shaped(ops, q, out, cache, group, step, spec, scale, sinks, weighting, chunk, head_bias, gate, softcap, distance):
-    """Attention whose scores are capped or lose a bias that grows with the distance: in bfloat16 the tensor-core kernels
+def _run_shaped(ops, q, out, cache, group, step, spec, scale, sinks, weighting, chunk, head_bias, gate, softcap, distance, keep):
+    """Attention whose scores are capped or lose a bias that grows with the distance, or whose window leaves the first keys
+    visible (the decode kernel then cuts the keys a token reads into chunks, not its positions): in bfloat16 the tensor-core kernels
     for portions of prompts (tcgen05 for long portions of heads of 64 or 128, else mma.sync) and the block-per-chunk kernel
     for single tokens (a mixed step launches both); in float32, for
     other head sizes, or together with another weighting, a chunked mask or a gate per head, the one kernel whose sums
     depend on positions alone."""
-    shape = dict(softcap=softcap, distance=distance)
+    shape = dict(softcap=softcap, distance=distance, keep=keep)
     plain = weighting == "softmax" and chunk is None and head_bias is None and gate is None
+    # what bounds the decode launch: the context, or the most keys a token reads
+    bound = lambda context: min(int(context), int(spec.window) + int(keep)) if keep else context
+    if keep and step.max_query_len == 1:
+        plain = plain and _merges_itself(ops, spec, q.shape[0], bound(group.max_context))
+    elif keep and step.single_tokens is not None:
+        plain = plain and _merges_itself(ops, spec, step.single_tokens.shape[0], bound(step.single_context))
     if plain and ops.flash_supported(q.dtype, spec.head_dim):
         args = (q, out, cache.k, cache.v, group.block_table, step.req_index, step.positions,
                 spec.num_heads, spec.num_kv_heads, spec.head_dim, scale, spec.window)
         if step.max_query_len == 1:
-            return _decode(ops, args, step, spec, group, q.shape[0], group.max_context, sinks=sinks, shape=shape)
+            return _decode(ops, args, step, spec, group, q.shape[0], bound(group.max_context), sinks=sinks, shape=shape)
         if step.query_tiles is not None:
             tile_args = (q, out, cache.k, cache.v, group.block_table, step.query_tiles, spec.num_heads, spec.num_kv_heads,
                          spec.head_dim, scale, spec.window, step.err)
@@ -158,10 +173,10 @@ def _run_shaped(ops, q, out, cache, group, step, spec, scale, sinks, weighting, 
             else:
                 ops.flash_prefill(*tile_args, tile_rows=QUERY_TILE, sinks=sinks, **shape)
             if step.single_tokens is not None:
-                _decode(ops, args, step, spec, group, step.single_tokens.shape[0], step.single_context,
+                _decode(ops, args, step, spec, group, step.single_tokens.shape[0], bound(step.single_context),
                         token_index=step.single_tokens, sinks=sinks, shape=shape)
             return out
     return ops.paged_attention(q, out, cache.k, cache.v, group.block_table, step.req_index, step.positions,
                                spec.num_heads, spec.num_kv_heads, spec.head_dim, scale, spec.window, step.err, sinks=sinks,
                                weighting=weighting, chunk=chunk, head_bias=head_bias, gate=gate, softcap=softcap,
-                               distance=distance)
+                               distance=distance, keep=keep)

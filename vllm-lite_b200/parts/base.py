@@ -173,11 +173,15 @@ class StreamSink:
 @dataclass
 class ScaledPair:
     """The results of two sub-layers side by side, not yet added: the sum is a_scale * a + b_scale * b.  A mixer that says
-    `returns_pair` hands this to a block whose next norm says `takes_pair`; the norm's kernel forms the sum as it reads."""
+    `returns_pair` hands this to a block whose next norm says `takes_pair`; the norm's kernel forms the sum as it reads.
+    With weights (float32) and `eps`, each of the two is an RMS norm's input: n(a) * a_weight and n(b) * b_weight are added."""
     a: torch.Tensor
     a_scale: float
     b: torch.Tensor
     b_scale: float
+    a_weight: Optional[torch.Tensor] = None
+    b_weight: Optional[torch.Tensor] = None
+    eps: float = 0.0
 
 
 def sub_weights(weights: dict, prefix: str) -> dict:

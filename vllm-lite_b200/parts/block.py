@@ -144,7 +144,10 @@ class PostNormBlock:
             y = self.mixer(residual.x, step, cache)
         else:
             h, buf = self._stream_input(residual, step)
-            y = self.mixer(h, step, cache)
+            if getattr(self.mixer, "returns_pair", False) and getattr(self.norm1, "takes_pair", False):
+                y = self.mixer(h, step, cache, as_pair=True)      # two mixers side by side: the norm's kernel adds them as it reads
+            else:
+                y = self.mixer(h, step, cache)
         # the feed-forward reads the new stream in the activation dtype; after the last norm of the block only a
         # following block that asks for it does
         residual.cast = self.norm1.add_normed(y, residual.x, step, buf, **kw, **({} if self.bias1 is None else {"bias": self.bias1}))

@@ -21,7 +21,9 @@ the step is router, sort, two products and the sum: five launches instead of sev
 
 Options of the router (`ops.moe_route`): a bias on the logits, a bias on the scores that only the choice sees, groups of
 neighbouring experts that count by their largest or by the sum of their largest choice values, renormalised weights.
-A `shared` feed-forward (any registered kind) runs for every token beside the experts and is added to their sum.
+A `shared` feed-forward (any registered kind) runs for every token beside the experts and is added to their sum, times
+sigmoid(W_sg h) with `shared_gate` (one more row of the router's product).  `identity` experts are router outputs behind the
+experts' without tensors: the sort passes over them and the last kernel adds the token's own row, weighted.
 """
 from __future__ import annotations
 
@@ -42,13 +44,16 @@ class RoutedExperts:
     def declare(spec: RoutedExpertsSpec) -> dict:
         gate, up, down = spec.names
         I, H = spec.intermediate_size, spec.hidden_size
-        d = {spec.router: TensorDecl((spec.num_experts, H))}
+        outputs = spec.num_experts + spec.identity
+        d = {spec.router: TensorDecl((outputs, H))}
         if spec.router_bias is not None:
-            d[spec.router + spec.router_bias] = TensorDecl((spec.num_experts,))
+            d[spec.router + spec.router_bias] = TensorDecl((outputs,))
         if spec.choice_bias is not None:
-            d[spec.choice_bias] = TensorDecl((spec.num_experts,), init="unit")
+            d[spec.choice_bias] = TensorDecl((outputs,), init="unit")
         if spec.shared is not None:
             d.update(prefixed(FEED_FORWARDS.get(spec.shared.kind).declare(spec.shared), spec.shared_prefix))
+            if spec.shared_gate is not None:
+                d[spec.shared_gate] = TensorDecl((1, H))
         for e in range(spec.num_experts):
             p = spec.expert_prefix.format(e)
             d.update({p + up: TensorDecl((I, H)), p + down: TensorDecl((H, I))})
@@ -58,11 +63,16 @@ class RoutedExperts:
 
     def __init__(self, spec: RoutedExpertsSpec, weights: dict, ctx):
         from ..csrc import ops
-        if not 0 < spec.top <= spec.num_experts:
-            raise ValueError(f"routed experts: top {spec.top} of {spec.num_experts} experts")
-        if spec.groups < 1 or spec.num_experts % spec.groups or not 1 <= spec.keep_groups <= spec.groups \
-                or spec.keep_groups * (spec.num_experts // spec.groups) < spec.top:
-            raise ValueError(f"routed experts: {spec.num_experts} experts in {spec.groups} groups of which {spec.keep_groups} "
+        outputs = spec.num_experts + spec.identity           # what the router chooses from
+        if spec.identity < 0 or spec.num_experts < 1 or not 0 < spec.top <= outputs:
+            raise ValueError(f"routed experts: top {spec.top} of {spec.num_experts} + {spec.identity} experts")
+        if spec.shared_gate is not None and spec.shared is None:
+            raise ValueError("routed experts: a gate on a shared feed-forward that is not there")
+        if spec.identity and spec.scale_input:
+            raise ValueError("routed experts: identity experts go with weights on the experts' outputs")
+        if spec.groups < 1 or outputs % spec.groups or not 1 <= spec.keep_groups <= spec.groups \
+                or spec.keep_groups * (outputs // spec.groups) < spec.top:
+            raise ValueError(f"routed experts: {outputs} experts in {spec.groups} groups of which {spec.keep_groups} "
                              f"are kept cannot offer {spec.top} choices")
         known = ops.ACTIVATIONS if spec.gated else ops.UNARY_ACTIVATIONS
         if spec.activation not in known or spec.score not in ops.ROUTER_SCORES:
@@ -77,6 +87,8 @@ class RoutedExperts:
         # bfloat16 rows stays as it is: the products of two bfloat16 numbers are exact in float32, so the tensor
         # cores add the same numbers as a float32 product of the widened matrix would.
         r = weights[spec.router]
+        if spec.shared_gate is not None:                     # the shared feed-forward's gate: one more row
+            r = torch.cat([r, weights[spec.shared_gate].to(r.dtype)], dim=0)
         keep = r.dtype == torch.bfloat16 and ctx.dtype == torch.bfloat16 and spec.hidden_size % 8 == 0
         self.router = r.contiguous() if keep else r.to(device=ctx.device, dtype=torch.float32).contiguous()
         self.router_bias = None
@@ -122,9 +134,13 @@ class RoutedExperts:
         sorted_rows = ws.get(tag + "moe.sorted", (cap,), torch.int32)
         tile_group = ws.get(tag + "moe.tiles", (cap // bm,), torch.int32)
         place = ws.get(tag + "moe.place", (pairs,), torch.int32)
-        logits = ws.get(tag + "moe.logits", (ops.router_slices(H), T, E), torch.float32)
+        logits = ws.get(tag + "moe.logits", (ops.router_slices(H), T, self.router.shape[0]), torch.float32)
+        share = ws.get(tag + "moe.share", (T,), torch.float32) if s.shared_gate is not None else None
         ops.moe_route(h, self.router, top, ids, weights, logits, s.score, s.renormalize, s.groups, s.keep_groups,
-                      bias=self.router_bias, choice_bias=self.choice_bias, group_top=s.group_top, renorm_eps=s.renorm_eps)
+                      bias=self.router_bias, choice_bias=self.choice_bias, group_top=s.group_top, renorm_eps=s.renorm_eps, extra_out=share)
+        last = dict(add_weight=share)
+        if s.identity:
+            last.update(ids=ids, identity_from=E, h=h)
         ops.moe_align(ids, E, bm, sorted_rows, tile_group, place)
         act = ws.get(tag + "moe.act", (cap, I), self.dtype)
         if big:
@@ -134,7 +150,7 @@ class RoutedExperts:
                                  weights if s.scale_input else None, s.activation, s.alpha, s.limit, s.up_shift)
             res = ops.gemm_grouped_tc5(act, self.down, ws.get(tag + "moe.down", (cap, H), self.dtype), tile_group, step.err)
             return ops.moe_combine(res, place, weights, top, ws.get(tag + "moe.out", (T, H), self.dtype), not s.scale_input,
-                                   add=self._shared(h, step))
+                                   add=self._shared(h, step), **last)
         if self.fused:
             ops.gemm_grouped_fused(h, self.gate_up, act, tile_group, bm, sorted_rows, top,
                                    weights if s.scale_input else None, s.activation, s.alpha, s.limit, s.up_shift)
@@ -147,7 +163,7 @@ class RoutedExperts:
                 ops.unary_act(gu, act, s.activation)
         res = ops.gemm_grouped(act, self.down, ws.get(tag + "moe.down", (cap, H), self.dtype), tile_group, bm)
         out = ws.get(tag + "moe.out", (T, H), self.dtype)
-        return ops.moe_combine(res, place, weights, top, out, not s.scale_input, add=self._shared(h, step))
+        return ops.moe_combine(res, place, weights, top, out, not s.scale_input, add=self._shared(h, step), **last)
 
     def _shared(self, h, step):
         """The shared feed-forward's rows (None without one): the kernel that sums a token's choices adds them last."""

@@ -7,7 +7,7 @@ the activation is one kernel on the stacked result and adds the two projections'
 the down projection's bias is added by the linear layer.
 The SwiGLU part (`parts/mlp.py`) is the bias-free special case whose activation the product kernels
 fuse; this part serves what that one does not take.  Without a gate (`gated` False) it is down(f(up(h))) with f a
-function of one argument (the square of max(v, 0))."""
+function of one argument (the square of max(v, 0)), or of the whole row (a polynomial of normed powers, `ops.poly_norm`)."""
 from __future__ import annotations
 
 import torch
@@ -26,7 +26,10 @@ class GatedMlp:
         gate, up, down = spec.names
         I, H = spec.intermediate_size, spec.hidden_size
         if not spec.gated:
-            return {up: TensorDecl((I, H)), down: TensorDecl((H, I))}
+            d = {up: TensorDecl((I, H)), down: TensorDecl((H, I))}
+            if spec.activation == "poly_norm":
+                d[spec.coef] = TensorDecl((4,), init="norm")
+            return d
         d = {gate: TensorDecl((I, H)), up: TensorDecl((I, H)), down: TensorDecl((H, I))}
         if spec.bias:
             d.update({gate + spec.bias_suffix: TensorDecl((I,)), up + spec.bias_suffix: TensorDecl((I,)),
@@ -35,7 +38,7 @@ class GatedMlp:
 
     def __init__(self, spec: GatedMlpSpec, weights: dict, ctx):
         from ..csrc import ops
-        known = ops.ACTIVATIONS if spec.gated else ops.UNARY_ACTIVATIONS
+        known = ops.ACTIVATIONS if spec.gated else tuple(ops.UNARY_ACTIVATIONS) + ("poly_norm",)
         if spec.activation not in known or (spec.bias and not spec.gated):
             raise ValueError(f"gated_mlp: activation {spec.activation!r} ({'with' if spec.gated else 'without'} a gate); "
                              f"known: {', '.join(known)}")
@@ -45,6 +48,11 @@ class GatedMlp:
         if not spec.gated:
             self.gate_up_bias = None
             self.gate_up = Linear(weights[up])
+            self.coef = None
+            if spec.activation == "poly_norm":
+                if not spec.eps > 0:
+                    raise ValueError(f"gated_mlp: normed powers need a positive eps, got {spec.eps}")
+                self.coef = weights[spec.coef].to(device=ctx.device, dtype=torch.float32).contiguous()
             self.down = Linear(weights[down])
             return
         b = spec.bias_suffix
@@ -59,6 +67,8 @@ class GatedMlp:
         gu = self.gate_up(h, step, "mlp.gate_up")
         act = step.workspace.get(step.tag + "mlp.act", (gu.shape[0], self.spec.intermediate_size), gu.dtype)
         s = self.spec
+        if not s.gated and self.coef is not None:
+            return self.down(ops.poly_norm(gu, self.coef, s.eps, act), step, "mlp.down")
         if not s.gated:
             return self.down(ops.unary_act(gu, act, s.activation), step, "mlp.down")
         ops.gated_act(gu, act, s.activation, 0, s.alpha, s.limit, s.up_shift, bias=self.gate_up_bias)

@@ -6,6 +6,7 @@ from __future__ import annotations
 
 import torch
 
+from ..cache.spec import widened
 from .base import BuildContext, Residual, prefixed, sub_weights
 from .registry import BLOCKS, EMBEDDINGS, HEADS, NORMS
 from .spec import ModelPlan, TensorDecl
@@ -24,12 +25,27 @@ def declare_model(plan: ModelPlan) -> dict:
 
 def cache_needs(plan: ModelPlan) -> list:
     """The need of every entry of the running order (None for an entry that
-    keeps nothing or that reads another entry's cache)."""
+    keeps nothing or that reads another entry's cache; what such a reader can reach is
+    kept by the owner), then the embedding's, if it keeps something (`cache_sources` beside it)."""
     needs = []
     for call in plan.order:
         block = plan.layers[call.layer]
-        needs.append(None if call.cache_of is not None else BLOCKS.get(block.kind).cache_need(block))
+        need = BLOCKS.get(block.kind).cache_need(block)
+        if call.cache_of is not None:
+            needs[call.cache_of] = widened(needs[call.cache_of], need)
+            need = None
+        needs.append(need)
+    emb = plan.embedding_spec
+    own = getattr(EMBEDDINGS.get(emb.kind), "cache_need", None)
+    if own is not None:
+        needs.append(own(emb))
     return needs
+
+
+def cache_sources(plan: ModelPlan) -> list:
+    """For every entry of `cache_needs`: the earlier entry whose cache it reads, or None."""
+    sources = [c.cache_of for c in plan.order]
+    return sources + [None] * (len(cache_needs(plan)) - len(sources))
 
 
 class CausalLM:
@@ -51,7 +67,10 @@ class CausalLM:
         the running order with the stream brought up to date (a reader for tests and comparisons)."""
         ws = step.workspace
         x = ws.get(step.tag + "residual", (step.num_tokens, self.plan.hidden_size), torch.float32)
-        self.embedding(step, x)
+        if getattr(self.embedding, "keeps_state", False):
+            self.embedding(step, x, caches[len(self.plan.order)])
+        else:
+            self.embedding(step, x)
         residual = Residual(x)
         order = self.plan.order
         for i, (call, cache) in enumerate(zip(order, caches)):

@@ -43,7 +43,10 @@ class RmsNorm:
         from ..csrc import ops
         from .base import ScaledPair
         if isinstance(y, ScaledPair):
-            ops.rmsnorm_add(y.a, self.weight, self.spec.eps, mult, x, cast, bias=bias, pair=(y.b, y.a_scale, y.b_scale))
+            if y.a_weight is not None and y.eps != self.spec.eps:
+                raise NotImplementedError("the norms of a pair and the norm of their sum share one eps")
+            ops.rmsnorm_add(y.a, self.weight, self.spec.eps, mult, x, cast, bias=bias,
+                            pair=(y.b, y.a_scale, y.b_scale, y.a_weight, y.b_weight))
         else:
             ops.rmsnorm_add(y, self.weight, self.spec.eps, mult, x, cast, bias=bias)
         return cast

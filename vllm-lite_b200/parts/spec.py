@@ -53,6 +53,18 @@ class NormSpec:
 
 
 @dataclass(frozen=True)
+class RotaryScaling:
+    """How rotary frequencies are slowed down for long contexts.  `original` None: every frequency divided by `factor`.
+    Else by wavelength l = 2 pi / f against the context the model was first trained for: f as it is where
+    l < original / high, f / factor where l > original / low, between the two (1 - s) f / factor + s f with
+    s = (original / l - low) / (high - low)."""
+    factor: float
+    low: float = 1.0
+    high: float = 1.0
+    original: Optional[float] = None
+
+
+@dataclass(frozen=True)
 class RotarySpec:
     """Rotary position encoding of the first `rotary_dim` features of each head; inv_freq[i] =
     theta^(-2i / rotary_dim).  Feature i turns with feature i + rotary_dim/2 (rotate-half), or, when
@@ -62,6 +74,7 @@ class RotarySpec:
     rotary_dim: Optional[int] = None
     kind: str = "rotary"
     interleaved: bool = False
+    scaling: Optional[RotaryScaling] = None
 
     @property
     def dim(self) -> int:
@@ -86,7 +99,13 @@ class AttentionSpec:
     of the key j that query i reads;
     `unit_sink`: the softmax denominator holds one more term exp(0) = 1, with no key and no value;
     `gate` (a tensor name): the concatenated heads are multiplied element by element by sigmoid(W_g h),
-    W_g [num_heads * value size, hidden], before the output projection.
+    W_g [num_heads * value size, hidden], before the output projection;
+    `whole_norm`: `qk_norm` (an RMS norm) runs over the whole q row and the whole k row at once, before the heads are told
+    apart; its weights have num_heads * head_dim and num_kv_heads * head_dim entries (`qk_norm.size` stays head_dim);
+    `head_temp` (a tensor name, [num_heads]): head h's scores are multiplied by its number;
+    `sink` (a tensor name, [num_heads]): the softmax denominator of head h holds one more term exp(sink_h), with no key, no
+    value and no scale;
+    `keep_first`: beside a window, the first that many keys of the sequence stay visible to every query.
     """
     hidden_size: int
     num_heads: int
@@ -111,6 +130,57 @@ class AttentionSpec:
     distance_bias: Optional[Tuple[str, str]] = None
     unit_sink: bool = False
     gate: Optional[str] = None
+    whole_norm: bool = False
+    head_temp: Optional[str] = None
+    sink: Optional[str] = None
+    keep_first: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class DifferentialAttentionSpec:
+    """Attention whose heads are the difference of two softmax maps over the same values.
+
+    q has num_heads x 2 x dim rows and k num_kv_heads x 2 x dim, head by head as [map 1, map 2]; v num_kv_heads x vdim.
+    `qk_norm` (an RMS norm over dim, its two weights shared by all heads and maps) and `position` act on every map of every
+    head; score = scale q.k over the last `window` keys.  With a_1, a_2 the maps' outputs of a head and
+    lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff (one number; four tensors of dim entries): o = a_1 - lambda a_2, then
+    o / sqrt(mean(o^2) + eps) over the head's values, times (1 - diff); out = W_o concat.
+    `own_kv` False: no key and value tensors; the call reads the cache of an earlier call of this kind (`LayerCall.cache_of`).
+    `names`: (q, k, v, o); a bias is `<name><bias_suffix>` (q, k, v); the norm weights `<name><norm_suffix>`."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    dim: int
+    vdim: int
+    eps: float
+    diff: float
+    scale: Optional[float] = None
+    qk_norm: Optional[NormSpec] = None
+    position: Optional[RotarySpec] = None
+    window: Optional[int] = None
+    keep_first: Optional[int] = None
+    bias: bool = True
+    own_kv: bool = True
+    names: Tuple[str, str, str, str] = ("q", "k", "v", "o")
+    lambda_names: Tuple[str, str, str, str] = ("lq1", "lk1", "lq2", "lk2")
+    bias_suffix: str = ".b"
+    norm_suffix: str = ".norm"
+    kind: str = "differential_attention"
+
+
+@dataclass(frozen=True)
+class PairEmbeddingSpec:
+    """x[t] = table[id_t] * scale + pairs[r_t] (float32), r_t = (id_(t-1) mul_prev + id_t mul_cur) mod buckets, and row
+    `buckets` (the table's last) for a sequence's first token.  The token before is part of the request's state."""
+    vocab_size: int
+    hidden_size: int
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+    scale: float = 1.0
+    tensor: str = "embed"
+    pair_tensor: str = "bigram"
+    kind: str = "pair_embedding"
 
 
 @dataclass(frozen=True)
@@ -183,7 +253,9 @@ class GatedMlpSpec:
     u' = clamp(u, -limit, limit), g' sigmoid(alpha g') (u' + up_shift)) and optional bias vectors on all
     three projections.  `names`: (gate, up, down) relative to the part's prefix; a bias is `<name><bias_suffix>`.
     `gated` False: down(f(up(h))) with f a function of one argument ("relu2": the square of max(v, 0)); there is no gate
-    matrix and no bias."""
+    matrix and no bias.
+    Activation "poly_norm" (ungated) takes the whole row: c_0 N(z) + c_1 N(z^2) + c_2 N(z^3) + c_3, powers element by element,
+    N(v) = v / sqrt(mean(v^2) + eps) over the row; its four numbers are the tensor `coef`."""
     hidden_size: int
     intermediate_size: int
     activation: str = "silu"
@@ -195,6 +267,8 @@ class GatedMlpSpec:
     bias_suffix: str = ".b"
     kind: str = "gated_mlp"
     gated: bool = True
+    coef: str = "act"
+    eps: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -214,6 +288,9 @@ class RoutedExpertsSpec:
     largest).  `renorm_eps` is added to the sum that `renormalize` divides by.
     `shared`: the description of one more feed-forward (any registered kind) that runs for every token and is added; its
     tensors lie under `shared_prefix`.
+    `identity`: the router has that many more outputs behind the experts' (scores, correction and choice run over all of
+    them); such an expert has no tensors and its result is its input.
+    `shared_gate` (a tensor name, [1, hidden]): the shared feed-forward's result is multiplied by sigmoid(W_sg h).
     Tensors: `router`, and per expert i `expert_prefix.format(i)` + gate / up / down of `names`."""
     hidden_size: int
     intermediate_size: int
@@ -241,6 +318,8 @@ class RoutedExpertsSpec:
     renorm_eps: float = 0.0
     shared: Optional[object] = None
     shared_prefix: str = "shared."
+    identity: int = 0
+    shared_gate: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -375,15 +454,49 @@ class TimeMixSpec:
 
 
 @dataclass(frozen=True)
+class MinGruSpec:
+    """A minimal gated recurrence (minGRU): the gates depend on the token at hand, not on the state; `width` channels, one by one.
+
+    z = sigmoid(W_z h + b_z), u = W_x h + b_x, c = u + 1/2 where u >= 0 and sigmoid(u) where u < 0;
+    S <- (1 - z) S + z c from zero;  out = W_o (S * silu(W_g h)).  `names`: (z, x, g, o); biases `<name><bias_suffix>` (z, x)."""
+    hidden_size: int
+    width: int
+    names: Tuple[str, str, str, str] = ("z", "x", "g", "o")
+    bias_suffix: str = ".b"
+    kind: str = "min_gru"
+
+
+@dataclass(frozen=True)
+class GatedLruSpec:
+    """A real-gated linear recurrent unit behind a short convolution, beside a gelu branch (the recurrent block of Griffin).
+
+    y = gelu_tanh(W_y h + b_y); u = causal convolution of `conv` taps per channel of W_x h + b_x (with bias, no activation);
+    in each of `blocks` equal parts of the channels r = sigmoid(A_r u + b_r), i = sigmoid(A_i u + b_i), square matrices;
+    log a = -rate r softplus(lam), S <- a S + sqrt(1 - a^2) i u from zero;  out = W_o (S * y).
+    `names`: (y, x, conv, r, i, lam, o); a bias is `<name><bias_suffix>`."""
+    hidden_size: int
+    width: int
+    blocks: int
+    conv: int
+    rate: float = 8.0
+    names: Tuple[str, ...] = ("y", "x", "conv", "ra", "ri", "lam", "o")
+    bias_suffix: str = ".b"
+    kind: str = "gated_lru"
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec:
     """Two mixers side by side on the same input: left_scale * left(h) + right_scale * right(h).  Each keeps its own
-    cache or state; their tensors lie under `prefixes`."""
+    cache or state; their tensors lie under `prefixes`.  `out_norms`: two RMS norms over the model width, each side's result
+    is normed by its own before the two are scaled and added (tensors `out_norm_prefixes`)."""
     left: object
     right: object
     left_scale: float = 1.0
     right_scale: float = 1.0
     prefixes: Tuple[str, str] = ("left.", "right.")
     kind: str = "parallel_mixer"
+    out_norms: Optional[Tuple[NormSpec, NormSpec]] = None
+    out_norm_prefixes: Tuple[str, str] = ("left.out", "right.out")
 
 
 @dataclass(frozen=True)
