@@ -193,3 +193,32 @@ def test_native_decode_step_equals_its_parts():
         small.decode_step(["p", "q"], [1, 2], 2, 8, 1000, np.zeros(4096, dtype=np.int32))
     assert small.free_pages() == [0, 7] and small.requests["p"].num_tokens == 4
     assert before == (a.free_pages(), [a.requests[r].num_tokens for r in ids])
+
+
+def test_first_tokens_stay_behind_a_window(make):
+    """Pages wholly behind the window are given back, those of the first `keep` tokens are not."""
+    m = make(layout(PagedKV(2, 16, window=10, keep=5), PagedKV(2, 16, window=10)), page_size=4, num_pages=[12, 12], max_requests=2)
+    m.admit("a")
+    m.append("a", 30)
+    m.release_behind_window("a")                       # the next query sits at 30 and reads 21..: pages 0..4 are dead
+    kept, plain = m.requests["a"].block_tables
+    assert [p >= 0 for p in kept] == [True, True, False, False, False, True, True, True]      # 5 tokens: two pages
+    assert [p >= 0 for p in plain] == [False] * 5 + [True] * 3
+    m.check_invariants()
+    m.append("a", 10)
+    m.release_behind_window("a")
+    assert [p >= 0 for p in m.requests["a"].block_tables[0]] == [True, True] + [False] * 5 + [True] * 3
+    m.free("a")
+    assert m.free_pages() == [12, 12]
+    m.check_invariants()
+
+
+def test_an_owner_keeps_what_its_readers_reach():
+    from vllm_lite_b200.cache.spec import widened
+    kv = lambda **k: PagedKV(2, 16, **k)
+    assert widened(kv(window=8), kv(window=20)) == kv(window=20) and widened(kv(window=20), kv(window=8)) == kv(window=20)
+    assert widened(kv(window=8), kv()) == kv() and widened(kv(), kv(window=8)) == kv()
+    assert widened(kv(window=8, keep=2), kv(window=8, keep=5)) == kv(window=8, keep=5)
+    assert widened(kv(chunk=8), kv(window=4)) == kv() and widened(kv(chunk=8), kv(chunk=8)) == kv(chunk=8)
+    with pytest.raises(ValueError):
+        widened(kv(window=8), PagedKV(4, 16, window=8))
