@@ -431,7 +431,7 @@ TIMED_OPS = ("paged_attention", "flash_prefill", "flash_prefill_tc5", "flash_dec
              "moe_gather", "moe_combine", "gated_act", "silu_mul", "scale_softcap", "embed", "cast", "add_bias",
              "hc_step", "dyt_rows", "short_conv", "ssd_scan", "mlstm_scan", "delta_scan", "gate_norm", "scaled_sum",
              "token_shift", "rows_norm_rope_write", "conv_rows_norm_rope_write", "rmsnorm_add", "unary_act",
-             "head_norm_write", "rope_heads", "sigmoid_gate", "token_shift_multi", "decay_scan", "decay_from_raw")
+             "head_norm_write", "rope_heads", "sigmoid_gate", "token_shift_multi", "decay_scan", "decay_from_raw", "head_work", "combine_maps", "linear_scan", "poly_norm", "embed_pair")
 
 
 def kikepel_config(size, layers):
@@ -445,10 +445,11 @@ def kikepel_config(size, layers):
                 layers=[dict(type=kinds[i % 4][0], mixer=mix, mlp=kinds[i % 4][1]) for i in range(layers)])
 
 
-def timed_step(runner, entries):
+def timed_step(runner, entries, suffix=None):
     """One step with every kernel of csrc/ops.py between two CUDA events.  The launches queue up behind a
     kernel that only waits, so that the events see the kernels back to back and not the host's pace.
-    Returns {op: [launches, microseconds]} (library products through torch.mm are 'library_mm')."""
+    Returns {op: [launches, microseconds]} (library products through torch.mm are 'library_mm').  `suffix`(options of a
+    launch) -> what is added to its name, for launches that are to be listed apart."""
     import torch
     from vllm_lite_b200.csrc import ops
     from vllm_lite_b200.parts import matmul
@@ -461,7 +462,8 @@ def timed_step(runner, entries):
             e1.record()
             # an attention launch whose scores are capped or biased by the distance is listed apart
             shaped = k.get("softcap") or k.get("distance") is not None
-            records.append((name + "+shape" if shaped else name, e0, e1))
+            apart = suffix(k) if suffix is not None else ("+shape" if shaped else "")
+            records.append((name + apart, e0, e1))
             return r
         return inner
     for name in TIMED_OPS:
@@ -987,6 +989,166 @@ def puturax_bench(args):
     return 0
 
 
+# ---------------------------------------------------------------------------------------------------
+# --pafelorn: the Pafelorn decoder (differential attention, half of its layers reading an earlier layer's keys; windowed
+# attention with a factor and a sink per head beside a minimal gated recurrence; windowed attention with kept first tokens,
+# capped scores and an output gate beside a gated linear recurrent unit; normed powers, or experts with identity experts and a
+# gated shared one) beside the Qwen3 decoder at equal width, depth, heads and active feed-forward width
+# ---------------------------------------------------------------------------------------------------
+# name: (width, heads, kv heads, value head size = 2 dims of a differential map = head size elsewhere, window, kept, recurrence
+#        width, its blocks, taps, dense ff, expert ff, experts, top, identity, shared ff, vocab)
+PAFELORN_SIZES = {"2k": (2048, 16, 4, 128, 1024, 4, 2048, 16, 4, 8192, 1024, 32, 4, 8, 1024, 65536),
+                  "4k": (4096, 32, 8, 128, 2048, 128, 4096, 16, 4, 12288, 1408, 64, 6, 16, 1408, 65536),
+                  "4k-h64": (4096, 64, 8, 64, 512, 4, 5120, 40, 4, 8192, 2048, 32, 4, 4, 2048, 65536)}
+
+
+def pafelorn_config(size, layers):
+    W, H, KV, D, win, keep, C, blocks, taps, ff, eff, E, top, ident, sff, vocab = PAFELORN_SIZES[size]
+    def rot(n, **sc):
+        return dict(dims=n, base=500000.0, scaling=dict(factor=4.0, **sc))
+    def differential(**kv):
+        return dict(heads=H, kv_heads=KV, dim=D // 2, vdim=D, scale=(D // 2) ** -0.5, diff=0.4, mask=dict(size=16384), rot=rot(D // 2), **kv)
+    left = dict(heads=H, kv_heads=KV, dim=D, vdim=D, scale=D ** -0.5)
+    par = dict(left=dict(left, mask=dict(size=win), rot=rot(D, low=1.0, high=4.0, original=4096)), right=dict(width=C), left_scale=0.7, right_scale=0.6)
+    par2 = dict(left=dict(left, softcap=30.0, mask=dict(size=win, keep_first=keep), rot=rot(D // 2)), right=dict(width=C, blocks=blocks, conv=taps))
+    dense = dict(kind="dense", ff=ff)
+    moe = dict(kind="moe", expert=dict(ff=eff, limit=7.0), router=dict(experts=E, top=top, identity=ident), shared=dict(ff=sff, limit=7.0))
+    kinds = [("attention", lambda i: differential(), dense), ("parallel", lambda i: par, moe),
+             ("attention", lambda i: differential(kv_from=i - 2), moe), ("parallel_2", lambda i: par2, moe)]
+    return dict(architecture="Pafelorn", vocab=vocab, width=W, norm=dict(eps=1e-6), logit_softcap=30.0,
+                embedding=dict(scale=1.0, bigram=dict(buckets=50021, mul_prev=31, mul_cur=7)), max_position_embeddings=16384,
+                layers=[dict(type=kinds[i % 4][0], mixer=kinds[i % 4][1](i), mlp=kinds[i % 4][2]) for i in range(layers)])
+
+
+def pafelorn_bench(args):
+    import torch
+    from vllm_lite_b200.engine import LLMEngine, StepEntry, random_model
+    size, layers = args.pafelorn, args.layers or 8
+    W, H, KV, D, win, keep, C, blocks, taps, ff, eff, E, top, ident, sff, vocab = PAFELORN_SIZES[size]
+    context, pk = args.context, peaks()
+    warmup = max(args.warmup, 3)
+    qwen = dict(QWEN3_8B, num_hidden_layers=layers, hidden_size=W, num_attention_heads=H, num_key_value_heads=KV,
+                head_dim=D, intermediate_size=top * eff + sff, vocab_size=vocab, max_position_embeddings=16384)
+    apart = lambda k: "+keep" if k.get("keep") else ("+sink" if k.get("sinks") is not None else "")
+    results = {}
+    for name, cfg in (("pafelorn", pafelorn_config(size, layers)), ("qwen3", qwen)):
+        _, plan, weights = random_model(cfg, seed=0, dtype="bfloat16", device="cuda:0")
+        for key in weights:                               # corrections smaller than the scores: the tokens spread over the experts
+            if key.endswith(".correction"):
+                weights[key] = weights[key] * 0.01
+        slack = 256
+        pages = 64 * (-(-(context + slack) // args.block_size) + 1) + PREFILL_TOKENS // args.block_size + 64
+        engine = LLMEngine(plan=plan, weights=weights, dtype="bfloat16", kv_blocks=pages, block_size=args.block_size,
+                           max_batch_size=64, max_num_batched_tokens=PREFILL_TOKENS, prefill_chunk_size=PREFILL_TOKENS,
+                           max_model_len=context + slack)
+        del weights
+        runner, sampler = engine.runner, engine.sampler
+        for t in runner.storage.paged:
+            t.normal_()
+        res = {}
+        clocks = ClockSampler().start()
+        w0 = time.time()
+        pms = prefill_run(runner, vocab)
+        res["prefill"] = {"tokens": PREFILL_TOKENS, "ms": round(pms, 3), "tokens_per_s": round(PREFILL_TOKENS / pms * 1e3, 1)}
+        for b in (8, 64):
+            ms, launches, _ = decode_run(runner, sampler, b, context, warmup, args.steps, "random", vocab, f"d{b}.")
+            res[f"decode_b{b}"] = {"ms_per_step": round(ms, 4), "tokens_per_s": round(b * 1e3 / ms, 1), "launches": round(launches)}
+        clocks.stop()
+        res["clocks"] = clocks.summary(w0, time.time())
+        gen = torch.Generator().manual_seed(5)
+        prompt = torch.randint(0, vocab, (PREFILL_TOKENS,), generator=gen).tolist()
+        res["kernels_prefill"] = timed_step(runner, [StepEntry("kp", prompt, [PREFILL_TOKENS - 1])], apart)
+        runner.release("kp")
+        ids = [f"kd{i}" for i in range(64)]
+        for rid in ids:
+            runner.cache.admit(rid)
+            runner.cache.append(rid, context - 1)
+        runner.storage.zero_slots(runner.cache.take_fresh_slots())
+        res["kernels_decode_b64"] = timed_step(runner, [StepEntry(rid, [i], [0]) for i, rid in enumerate(ids)], apart)
+        for rid in ids:
+            runner.release(rid)
+        runner.check_device_errors()
+        res["weights_GB"] = round(sum(p.numel() * p.element_size() for p in _tensors_of(runner.model)) / 1e9, 2)
+        results[name] = res
+        del engine, runner, sampler
+        torch.cuda.empty_cache()
+    print(json.dumps({"pafelorn_bench": size, "layers": layers, "context": context, "steps": args.steps, "warmup": warmup,
+                      "dtype": "bf16", "data": "synthetic (random weights, uniform token ids)",
+                      "config": {"pafelorn": dict(zip(("width", "heads", "kv_heads", "head", "window", "keep_first", "rec_width", "rec_blocks",
+                                                       "taps", "dense_ff", "expert_ff", "experts", "top", "identity", "shared_ff", "vocab"),
+                                                      PAFELORN_SIZES[size])),
+                                 "qwen3": {k_: qwen[k_] for k_ in ("hidden_size", "num_attention_heads", "num_key_value_heads",
+                                                                    "head_dim", "intermediate_size", "vocab_size")}},
+                      "results": results, "roofline": pafelorn_roofline(size, layers, context, results, pk)}))
+    return 0
+
+
+def pafelorn_roofline(size, layers, context, results, pk):
+    """The new kernels against their rooflines, beside the like kernels of the closest model: algorithmic bytes or flops over
+    the launches' time between CUDA events."""
+    W, H, KV, D, win, keep, C, blocks, taps, ff, eff, E, top, ident, sff, vocab = PAFELORN_SIZES[size]
+    T, B = PREFILL_TOKENS, 64
+    px, q = results["pafelorn"], results["qwen3"]
+    us = lambda res, step, names: sum(res[step].get(n, [0, 0.0])[1] for n in names)
+    count = lambda res, step, name: res[step].get(name, [0, 0.0])[0]
+    tf = lambda flops, micro: round(flops / (micro * 1e-6) / 1e12, 1) if micro else None
+    gb = lambda nbytes, micro: round(nbytes / (micro * 1e-6) / 1e9, 1) if micro else None
+    each = lambda micro, n: round(micro / n, 1) if n else None
+    att = ("paged_attention", "flash_prefill", "flash_prefill_tc5", "flash_decode")
+    n_diff = sum(1 for i in range(layers) if i % 4 in (0, 2))
+    n_par, n_par2 = sum(1 for i in range(layers) if i % 4 == 1), sum(1 for i in range(layers) if i % 4 == 3)
+    causal = T * (T + 1) // 2
+    w = min(win, T)
+    inside = w * (w + 1) // 2 + (T - w) * w                       # (query, key) pairs inside the window
+    kept = sum(min(keep, max(0, t - win + 1)) for t in range(T))
+    reach = min(win, context)
+    roof = {"peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"], "source": pk["source"]}}
+    kinds = (("differential", "", n_diff, 2, causal, context), ("window, sink", "+sink", n_par, 1, inside, reach),
+             ("window, kept, capped", "+keep", n_par2, 1, inside + kept, reach + keep))
+    for step, fig in (("kernels_prefill", "attention_prefill_tflops"), ("kernels_decode_b64", "attention_decode_gbs")):
+        r = {}
+        for label, suffix, n, maps, pairs, keys in kinds:
+            t = us(px, step, tuple(a + suffix for a in att))
+            # a map of a differential head: dim multiply-adds a score (its half of the row), 2 dim for the values
+            r[label] = tf(n * pairs * H * (6.0 * D if maps == 2 else 4.0 * D), t) if step == "kernels_prefill" else gb(n * B * keys * 2.0 * KV * D * 2.0, t)
+            r[label + ", us a layer"] = each(t, n)
+        t = us(q, step, att)
+        r["qwen3"] = tf(layers * causal * H * 4.0 * D, t) if step == "kernels_prefill" else gb(layers * B * context * 2.0 * KV * D * 2.0, t)
+        r["qwen3, us a layer"] = each(t, layers)
+        roof[fig] = r
+    n_rec, n_moe, n_dense = n_par + n_par2, layers - sum(1 for i in range(layers) if i % 4 == 0), sum(1 for i in range(layers) if i % 4 == 0)
+    own = sum(1 for i in range(layers) if i % 4 == 0)
+    for step, rows in (("kernels_prefill", T), ("kernels_decode_b64", B)):
+        r = {}
+        # head work: q, k, v in; q (a differential map's row twice as wide), k, v out
+        nbytes = rows * 2.0 * D * (own * (3 * H + 4 * KV) + (n_diff - own) * 3 * H + n_rec * (2 * H + 4 * KV))
+        r["head_work_gbs"] = gb(nbytes, us(px, step, ("head_work",)))
+        r["qwen3_qk_norm_rope_write_gbs"] = gb(count(q, step, "qk_norm_rope_write") * rows * (H + 2 * KV) * D * 4.0, us(q, step, ("qk_norm_rope_write",)))
+        r["combine_maps_gbs"] = gb(n_diff * rows * H * D * 6.0, us(px, step, ("combine_maps",)))
+        r["sigmoid_gate_gbs"] = gb(n_par2 * rows * H * D * 6.0, us(px, step, ("sigmoid_gate",)))
+        r["rmsnorm_add_gbs"] = gb(rows * W * 2.0 * (layers * 6 + n_rec + (layers) * 6), us(px, step, ("rmsnorm_add",)))
+        r["qwen3_add_rmsnorm_gbs"] = gb(count(q, step, "add_rmsnorm") * rows * W * 12.0, us(q, step, ("add_rmsnorm",)))
+        r["poly_norm_gbs"] = gb(n_dense * rows * ff * 4.0, us(px, step, ("poly_norm",)))
+        r["short_conv_gbs"] = gb(n_par2 * rows * C * 4.0, us(px, step, ("short_conv",)))
+        state = 8.0 * C * (B if rows == B else 1)
+        r["linear_scan_gbs"] = gb(n_par * (rows * C * 8.0 + state) + n_par2 * (rows * C * 14.0 + state), us(px, step, ("linear_scan",)))
+        t = us(px, step, ("gemm_heads",))
+        r["gate_products"] = {"tflops": tf(n_par2 * rows * 4.0 * C * (C // blocks), t), "us_a_layer": each(t, n_par2),
+                              "gbs": gb(n_par2 * (rows * C * 10.0 + 4.0 * C * (C // blocks)), t)}
+        r["us_a_step"] = {n: px[step][n][1] for n in px[step]}
+        roof[step] = r
+    grouped = ("gemm_grouped", "gemm_grouped_fused", "gemm_grouped_tc5")
+    share = E / (E + ident)                                       # of the choices, those that reach an expert with tensors
+    q_layer = (H + 2 * KV) * D * W + W * H * D + 3 * W * (top * eff + sff)
+    roof["expert_products_prefill_tflops"] = {
+        "pafelorn": tf(n_moe * 2.0 * T * top * share * 3 * W * eff, us(px, "kernels_prefill", grouped)),
+        "qwen3 (all dense products of the layers)": tf(layers * 2.0 * T * q_layer, us(q, "kernels_prefill", ("gemm_bf16_tc5", "gemm_bf16_tc5_pair", "library_mm")))}
+    roof["expert_products_decode_gbs"] = {
+        "pafelorn (experts that 64 tokens can reach)": gb(n_moe * min(E, B * top) * 3.0 * W * eff * 2, us(px, "kernels_decode_b64", grouped)),
+        "qwen3 (all products)": gb(q["weights_GB"] * 1e9 - 2.0 * vocab * W * 2, us(q, "kernels_decode_b64", ("library_mm", "gemm_bf16_small_m")))}
+    return roof
+
+
 def _tensors_of(model):
     """Every device tensor that the parts of a model hold (weights as they are resident)."""
     import torch
@@ -1039,6 +1201,9 @@ def main(argv=None):
     ap.add_argument("--puturax", default=None, choices=sorted(PUTURAX_SIZES), metavar="SIZE",
                     help="instead of the default workload: the Puturax decoder at layer sizes " + ", ".join(sorted(PUTURAX_SIZES))
                          + " beside the Qwen3 decoder at equal width, depth, heads and active feed-forward width")
+    ap.add_argument("--pafelorn", default=None, choices=sorted(PAFELORN_SIZES), metavar="SIZE",
+                    help="instead of the default workload: the Pafelorn decoder at layer sizes " + ", ".join(sorted(PAFELORN_SIZES))
+                         + " beside the Qwen3 decoder at equal width, depth, heads and active feed-forward width")
     ap.add_argument("--kikepel", default=None, choices=sorted(KIKEPEL_SIZES), metavar="SIZE",
                     help="instead of the default workload: the Kikepel decoder at layer sizes " + ", ".join(sorted(KIKEPEL_SIZES))
                          + " beside the Qwen3 decoder at equal width, depth and heads: prefill of 2,048 tokens, decode at batch 8 "
@@ -1061,6 +1226,8 @@ def main(argv=None):
         return sodonex_bench(args)
     if args.puturax:
         return puturax_bench(args)
+    if args.pafelorn:
+        return pafelorn_bench(args)
     import torch
     from vllm_lite_b200.csrc import ops
     from vllm_lite_b200.engine import LLMEngine, random_model

@@ -100,7 +100,7 @@ CONFIGS = {
 PAGE = {"A": 8, "B": 16, "C": 64, "D": 4}
 SEED = {"A": 61, "B": 62, "C": 63, "D": 64}
 # max |engine - plain| / max |plain| over a row of logits
-TOL = {"float32": 4e-5, "bfloat16": 5e-2}
+TOL = {"float32": 8e-5, "bfloat16": 5e-2}
 CASES = [(w, d) for w in ("A", "B", "C", "D") for d in ("float32", "bfloat16")]
 
 
