@@ -773,6 +773,113 @@ def test_element_wise_recurrences(dtype, kind, C, blocks):
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("kind", ["min_gru", "gated_lru"])
+@pytest.mark.parametrize("n", [128, 129, 1024, 1025, 2500])
+def test_long_stretches_do_not_depend_on_the_number_of_blocks(kind, n):
+    """A long portion alone (one cluster walks it), as a portion of a launch whose longest request is longer, and in two portions
+    cut at a stretch's border: the same bits; and the plain recurrence."""
+    o, C, dtype = ops(), 70, torch.bfloat16
+    ld = 3 * C if kind == "min_gru" else C
+    proj, u, gates = rand((n, ld), 20, dtype, 1.5), rand((n, C), 22, dtype), rand((n, 2 * C), 24)
+    b0, b1, b2 = (rand((C,), 26 + i, scale=0.5) for i in range(3))
+    decay = -8.0 * torch.nn.functional.softplus(rand((C,), 29) * 2 - 5)
+
+    def run(lo, hi, state, longest):
+        step = mini_step([hi - lo], [0], [lo])
+        out = torch.full((hi - lo, C), float("nan"), dtype=dtype, device=DEV)
+        kw = {} if kind == "min_gru" else dict(conv=u[lo:hi].contiguous(), gates=gates[lo:hi].contiguous(), block=C // 2, decay=decay)
+        o.linear_scan(kind, proj[lo:hi].contiguous(), (b0, b1) if kind == "min_gru" else (b0, b1, b2), state, 0, step.cu_seqlens,
+                      step.state_slots, out, longest=longest, **kw)
+        return out
+
+    fresh = lambda: torch.zeros((1, C), dtype=torch.float32, device=DEV)
+    sa, sb, sc = fresh(), fresh(), fresh()
+    whole = run(0, n, sa, n)
+    assert torch.equal(whole, run(0, n, sb, n + 3000)) and torch.equal(sa, sb)
+    cut = n // 2 // 128 * 128
+    if cut:
+        assert torch.equal(whole, torch.cat([run(0, cut, sc, cut), run(cut, n, sc, n - cut)])) and torch.equal(sa, sc)
+    d = lambda t: t.double().cpu()
+    x = d(proj)
+    if kind == "min_gru":
+        z = torch.sigmoid(x[:, :C] + d(b0))
+        S = P.linear_recurrence(1 - z, z * P.candidate(x[:, C:2 * C] + d(b1)))
+    else:
+        g = d(gates).view(n, 2, 2, C // 2)
+        r, i = torch.sigmoid(g[:, :, 0].reshape(n, C) + d(b0)), torch.sigmoid(g[:, :, 1].reshape(n, C) + d(b1))
+        S = P.linear_recurrence(torch.exp(d(decay) * r), torch.sqrt(-torch.expm1(2 * d(decay) * r)) * i * d(u))
+    close(sa[0], S[-1], torch.float32, "state", tol=1e-5)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype,out_dtype", [(torch.float32, torch.float32), (torch.bfloat16, torch.float32), (torch.bfloat16, torch.bfloat16)])
+@pytest.mark.parametrize("taps", [1, 2, 3, 4, 5])
+@pytest.mark.parametrize("C,col0", [(64, 8), (40, 0), (36, 4), (1100, 16), (7, 3)])
+def test_convolution_in_portions(dtype, out_dtype, taps, C, col0):
+    """Both kernels of the short convolution (16-byte accesses, and any size): biases on its rows and on its sums, an
+    activation, requests in portions, single tokens and portions of several runs."""
+    n, cuts = [83, 42], ([1, 2], [1, 0], [2, 1], [1, 39], [78, 0])
+    ld = col0 + C + (5 if C == 7 else 8)
+    x = [rand((n[b], ld), 130 + b, dtype) for b in (0, 1)]
+    w, bias, ib = rand((C, taps), 132), rand((C,), 133), rand((C,), 134)
+    state = torch.zeros((3, 4 + max(taps - 1, 1) * C + (-(taps - 1) * C) % 4), dtype=torch.float32, device=DEV)
+    slots = [2, 0]
+    for act in (False, True):
+        state.zero_()
+
+        def fn(live, lens, starts):
+            step = mini_step(lens, [slots[b] for b in live], starts)
+            rows = torch.cat([x[b][s:s + c] for b, s, c in zip(live, starts, lens)]).contiguous()
+            out = torch.full((rows.shape[0], C), float("nan"), dtype=out_dtype, device=DEV)
+            ops().short_conv(rows, col0, C, w, bias, state, 4, step.cu_seqlens, step.state_slots, out, act=act, longest=max(lens), in_bias=ib)
+            return out
+
+        got = in_portions(n, fn, cuts)
+        for b in (0, 1):
+            src = x[b].double().cpu()[:, col0:col0 + C] + ib.double().cpu()
+            want = P.causal_conv(src, w.cpu(), bias.cpu())
+            want = torch.nn.functional.silu(want) if act else want
+            close(got[b], want, dtype, f"convolution of request {b}", tol=3e-6 if out_dtype == torch.float32 else 8e-3)
+            if taps > 1:
+                kept = state[slots[b], 4:4 + (taps - 1) * C].view(taps - 1, C)
+                close(kept, src[-(taps - 1):], torch.float32, "kept inputs", tol=1e-6)
+        assert float(state[1].abs().max()) == 0.0 and float(state[:, :4].abs().max()) == 0.0
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("T,H_,K,N", [(512, 3, 64, 128), (700, 2, 136, 272), (1030, 5, 40, 100), (600, 1, 256, 512), (16, 4, 64, 128), (100, 4, 24, 48)])
+def test_product_per_block_with_float32_sums(T, H_, K, N):
+    """The gates' product: bfloat16 operands, the float32 sums as they are, few rows and many."""
+    a, w = rand((T, H_ * K), 140, torch.bfloat16), rand((H_, N, K), 141, torch.bfloat16, 0.2)
+    out = torch.full((T, H_ * N), float("nan"), device=DEV)
+    ops().gemm_heads(a, w, out)
+    want = torch.einsum("thk,hnk->thn", a.double().cpu().view(T, H_, K), w.double().cpu()).reshape(T, H_ * N)
+    close(out, want, torch.float32, "product", tol=2e-6)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("window", [1, 17, 64, 200])
+@pytest.mark.parametrize("H_,G_,D_,page", [(4, 2, 16, 8), (8, 2, 64, 64), (40, 2, 32, 16)])
+def test_single_tokens_count_the_keys_of_a_window(window, H_, G_, D_, page):
+    """The decode kernel with chunks over the readable keys instead of positions, on pages of which those behind the window are
+    given back."""
+    dtype, lens, new = torch.bfloat16, [300, 83, 1200, 5, 64], [1, 1, 1, 1, 1]
+    scale = 2.0 * D_ ** -0.5
+    seqs, kc, vc, table, req, pos, q = masked_case(dtype, H_, G_, D_, page, lens, new, window, 0, 4)
+    sink = rand((H_,), 81)
+    wants = want_masked(seqs, lens, new, req, q, H_, D_, scale, None, window, 0, sink.cpu())
+    e = torch.zeros(1, dtype=torch.int32, device=DEV)
+    for chunk in (64, 256):
+        out = torch.full((5, H_ * D_), float("nan"), dtype=dtype, device=DEV)
+        S, na, nm = ops().decode_attention_scratch(5, H_, D_, window, chunk)
+        arrivals = torch.zeros(ops().flash_decode_arrivals(5, H_, G_), dtype=torch.int32, device=DEV)
+        ops().flash_decode(q, out, kc, vc, table, ints(req), ints(pos), H_, G_, D_, scale, window, window, torch.empty(na, device=DEV),
+                           torch.empty(nm, device=DEV), e, chunk=chunk, arrivals=arrivals, sinks=sink, numbered=True)
+        assert int(e.item()) == 0 and int(arrivals.abs().max()) == 0
+        check_masked(out, wants, dtype, f"chunks of {chunk}", 1.5e-2)
+
+
+@pytest.mark.gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("kind,C,blocks,conv,W", [("min_gru", 40, 1, 1, 64), ("min_gru", 18, 1, 1, 72), ("min_gru", 320, 1, 1, 128), ("gated_lru", 36, 3, 3, 64),
                                                   ("gated_lru", 30, 5, 5, 72), ("gated_lru", 96, 1, 1, 96), ("gated_lru", 256, 4, 4, 128), ("gated_lru", 64, 8, 2, 64)])

@@ -262,14 +262,14 @@ extern "C" int vl_sigmoid_gate(void* x, int ldx, const void* g, int ldg, int gco
 // A polynomial of normed powers, row by row:
 //   out = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3,   N(v) = v / sqrt(mean(v^2) + eps) over the row's n values
 // (powers element by element; float32 inside).  The row is kept in registers where it fits (VPT groups of four values a
-// thread, 256 threads), else read twice.  The order of the sums depends on the row length alone.
+// thread, NT threads), else read twice.  The order of the sums depends on the row length alone.
 __device__ __forceinline__ float poly_value(float z, float f1, float f2, float f3, float c3) {
     return z * (f1 + z * (f2 + z * f3)) + c3;
 }
-template <typename T, int VPT>
-__global__ void __launch_bounds__(256)
+template <typename T, int VPT, int NT>
+__global__ void __launch_bounds__(NT)
 poly_norm_kernel(const T* __restrict__ in, T* __restrict__ out, int n, const float* __restrict__ coef, float eps) {
-    __shared__ float scratch[32];
+    __shared__ float s_part[3][NT / 32];
     pdl_launch_dependents();
     pdl_wait();
     const T* x = in + (size_t)blockIdx.x * n;
@@ -280,42 +280,46 @@ poly_norm_kernel(const T* __restrict__ in, T* __restrict__ out, int n, const flo
     if (VPT > 0) {
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
-            const int c = 4 * (threadIdx.x + 256 * i);
-            if (c < n) {
-                v[i] = Quad<T>::load(x + c);
-                add(v[i].x); add(v[i].y); add(v[i].z); add(v[i].w);
-            }
+            const int c = 4 * (threadIdx.x + NT * i);
+            v[i] = c < n ? Quad<T>::load(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) { add(v[i].x); add(v[i].y); add(v[i].z); add(v[i].w); }
     } else {
-        for (int i = threadIdx.x; i < n; i += 256) add(to_f32(x[i]));
+        for (int i = threadIdx.x; i < n; i += NT) add(to_f32(x[i]));
     }
-    s2 = block_sum<256>(s2, scratch);
-    s4 = block_sum<256>(s4, scratch);
-    s6 = block_sum<256>(s6, scratch);
+    s2 = warp_sum(s2); s4 = warp_sum(s4); s6 = warp_sum(s6);
+    if ((threadIdx.x & 31) == 0) { s_part[0][threadIdx.x >> 5] = s2; s_part[1][threadIdx.x >> 5] = s4; s_part[2][threadIdx.x >> 5] = s6; }
+    __syncthreads();
+    s2 = s4 = s6 = 0.f;
+#pragma unroll
+    for (int k = 0; k < NT / 32; ++k) { s2 += s_part[0][k]; s4 += s_part[1][k]; s6 += s_part[2][k]; }
     const float inv = 1.f / (float)n;
     const float f1 = coef[0] / sqrtf(s2 * inv + eps), f2 = coef[1] / sqrtf(s4 * inv + eps), f3 = coef[2] / sqrtf(s6 * inv + eps), c3 = coef[3];
     if (VPT > 0) {
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
-            const int c = 4 * (threadIdx.x + 256 * i);
+            const int c = 4 * (threadIdx.x + NT * i);
             if (c < n)
                 Quad<T>::store(o + c, make_float4(poly_value(v[i].x, f1, f2, f3, c3), poly_value(v[i].y, f1, f2, f3, c3),
                                                   poly_value(v[i].z, f1, f2, f3, c3), poly_value(v[i].w, f1, f2, f3, c3)));
         }
     } else {
-        for (int i = threadIdx.x; i < n; i += 256) o[i] = from_f32<T>(poly_value(to_f32(x[i]), f1, f2, f3, c3));
+        for (int i = threadIdx.x; i < n; i += NT) o[i] = from_f32<T>(poly_value(to_f32(x[i]), f1, f2, f3, c3));
     }
 }
 
 template <typename T>
 static int launch_poly_norm(const T* in, T* out, int rows, int n, const float* coef, float eps, cudaStream_t s) {
-    const int pieces = (n / 4 + 255) / 256;
     const bool vec = n % 4 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0;
-    if (vec && pieces <= 1) return vl_launch(poly_norm_kernel<T, 1>, dim3(rows), dim3(256), 0, s, in, out, n, coef, eps);
-    if (vec && pieces <= 4) return vl_launch(poly_norm_kernel<T, 4>, dim3(rows), dim3(256), 0, s, in, out, n, coef, eps);
-    if (vec && pieces <= 8) return vl_launch(poly_norm_kernel<T, 8>, dim3(rows), dim3(256), 0, s, in, out, n, coef, eps);
-    if (vec && pieces <= 16) return vl_launch(poly_norm_kernel<T, 16>, dim3(rows), dim3(256), 0, s, in, out, n, coef, eps);
-    return vl_launch(poly_norm_kernel<T, 0>, dim3(rows), dim3(256), 0, s, in, out, n, coef, eps);
+#define POLY(VPT, NT) return vl_launch(poly_norm_kernel<T, VPT, NT>, dim3(rows), dim3(NT), 0, s, in, out, n, coef, eps)
+    if (vec && n <= 1024) POLY(1, 256);
+    if (vec && n <= 4096) POLY(4, 256);
+    if (vec && n <= 8192) POLY(4, 512);
+    if (vec && n <= 12288) POLY(6, 512);
+    if (vec && n <= 16384) POLY(8, 512);
+    POLY(0, 256);
+#undef POLY
 }
 
 extern "C" int vl_poly_norm(const void* in, void* out, int dtype, int rows, int n, const float* coef, float eps, void* stream) {

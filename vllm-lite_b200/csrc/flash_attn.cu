@@ -25,7 +25,7 @@
 // partial results of chunks and warps simply add up (they travel with a maximum of 0, so every merge weighs them 1).
 // `keep` > 0: a query also reads the request's first `keep` keys, however far behind its window they lie.  The prefill
 // kernel walks the tiles of the kept keys before those of the window; the decode kernel numbers the keys that a token reads
-// (the kept ones first, then its window) and cuts that number into chunks.
+// (the kept ones first, then its window) and cuts that number into chunks (`numbered`, also for a window alone).
 // Rows of shared-memory tiles are padded by 16 bytes, which makes every 8-row ldmatrix access
 // hit 8 different banks groups for any head size.
 #include "score_shape.cuh"
@@ -86,6 +86,7 @@ struct AttnOptions {
     float cap_l2;                                        // a bound on the scores, times log2 e (0: none): s <- cap tanh(s / cap)
     const float* dist_a; const float* dist_b;            // per query head (or null): a ln(1 + b (i - j)) is taken off the score
     int keep;                                            // first keys of a request that every query reads (0: none)
+    int numbered;                                        // (decode) the launch counts the keys a token reads, not positions
 };
 __device__ __forceinline__ float gate_factor(const AttnOptions& op, int tok, int h) {
     return op.gate ? 1.f / (1.f + __expf(-__bfloat162float(op.gate[(size_t)tok * op.gate_stride + h]))) : 1.f;
@@ -372,7 +373,7 @@ extern "C" int vl_flash_prefill(const void* q, int q_stride, void* out, const vo
     auto kernel = weighting == 1 ? flash_prefill_kernel<true> : flash_prefill_kernel<false>;
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    const AttnOptions op = {weighting, block, head_bias, (const bf16*)gate, gate_stride, softcap * 1.4426950408889634f, dist_a, dist_b, keep};
+    const AttnOptions op = {weighting, block, head_bias, (const bf16*)gate, gate_stride, softcap * 1.4426950408889634f, dist_a, dist_b, keep, 0};
     kernel<<<dim3(nq, num_tiles * parts), NTHREADS, smem, (cudaStream_t)stream>>>(
         (const bf16*)q, q_stride, (bf16*)out, (const bf16*)kcache, (const bf16*)vcache, block_table, max_blocks,
         (const int4*)tiles, parts, nq, nkv, page_size, num_pages, scale * 1.4426950408889634f, window, err, sinks, op);
@@ -516,10 +517,11 @@ flash_decode_kernel(const bf16* __restrict__ q, int q_stride,
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     if (fz.op.block > 0 && pos >= 0) lo = max(lo, pos / fz.op.block * fz.op.block);
-    // With kept keys the launch works on the number of a key among those the token reads, not on its position: key v is
+    // `numbered`: the launch works on the number of a key among those the token reads, not on its position (kept keys need
+    // it; a window much shorter than the context gains by it, as no block is started for positions behind it): key v is
     // position v for v < kept and position v + gap behind them (gap = 0 without the option: number and position are one).
-    const int kept = fz.op.keep > 0 ? min(fz.op.keep, lo) : 0, gap = fz.op.keep > 0 ? lo - kept : 0;
-    if (fz.op.keep > 0) { lo = 0; pos -= gap; }
+    const int kept = fz.op.numbered ? min(fz.op.keep, lo) : 0, gap = fz.op.numbered ? lo - kept : 0;
+    if (fz.op.numbered) { lo = 0; pos -= gap; }
     if ((long long)pos >= (long long)S * chunk) {                // beyond the S chunks the launch was sized for:
         if (tid == 0 && split == 0 && err) atomicOr(err, VL_DEV_BEYOND_BOUND);   // flagged and served like an empty place
         pos = -1;
@@ -1089,12 +1091,12 @@ extern "C" int vl_flash_decode(const void* q, int q_stride, const void* kcache, 
                                int chunk, int S, float* part_acc, float* part_ml, unsigned* err,
                                const int* token_index, void* out, int* arrivals, const float* sinks, int weighting,
                                int block, const float* head_bias, const void* gate, int gate_stride, float softcap,
-                               const float* dist_a, const float* dist_b, int keep, void* stream) {
-    if (keep < 0 || (keep > 0 && block > 0)) return VL_ERR_ARGUMENT;
+                               const float* dist_a, const float* dist_b, int keep, int numbered, void* stream) {
+    if (keep < 0 || (keep > 0 && block > 0) || (keep > 0 && !numbered) || (numbered && (window <= 0 || block > 0 || !out))) return VL_ERR_ARGUMENT;
     if (softcap < 0.f || (dist_a == nullptr) != (dist_b == nullptr)) return VL_ERR_ARGUMENT;
     DecodeFusion fz = {};
     fz.sinks = sinks;
-    fz.op = AttnOptions{weighting, block, head_bias, (const bf16*)gate, gate_stride, softcap * 1.4426950408889634f, dist_a, dist_b, keep};
+    fz.op = AttnOptions{weighting, block, head_bias, (const bf16*)gate, gate_stride, softcap * 1.4426950408889634f, dist_a, dist_b, keep, numbered};
     return launch_flash_decode(q, q_stride, kcache, vcache, block_table, max_blocks, req_index, positions, T, nq, nkv, hd,
                                page_size, num_pages, scale, window, chunk, S, part_acc, part_ml, err, token_index, out,
                                arrivals, fz, stream);

@@ -284,6 +284,115 @@ static int launch_mma_kernel(dim3 grid, cudaStream_t s, int K, Args... args) {
     return vl_launch(kern, grid, dim3(128), smem, s, args..., nst);
 }
 
+// The plain batched product for many rows (one matrix per batch on column slices of wide activations, e.g. the gates of a
+// recurrence in blocks of channels): tiles of 128 x 128, eight warps of 32 x 64, a ring of up to three stages of 64 columns
+// of K.  Sums run over K in steps of 16 in order, as in the kernel above.
+#define GW_BM 128
+#define GW_BN 128
+#define GW_NST 3
+template <typename TC>
+__global__ void __launch_bounds__(256)
+gemm_batched_bf16_wide_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, TC* __restrict__ C, int M, int N, int K,
+                              int lda, int ldw, int ldc, long long a_bs, long long w_bs, long long c_bs, int nst) {
+    extern __shared__ __align__(16) unsigned char gw_smem[];
+    bf16 (*As)[GW_BM][GM_LDS] = reinterpret_cast<bf16 (*)[GW_BM][GM_LDS]>(gw_smem);
+    bf16 (*Ws)[GW_BN][GM_LDS] = reinterpret_cast<bf16 (*)[GW_BN][GM_LDS]>(gw_smem + (size_t)nst * GW_BM * GM_LDS * sizeof(bf16));
+    pdl_launch_dependents();
+    pdl_wait();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wm = warp & 3, wn = warp >> 2;
+    const int m0 = blockIdx.y * GW_BM, n0 = blockIdx.x * GW_BN;
+    const bf16* Ab = A + (size_t)blockIdx.z * a_bs;
+    const bf16* Wb = W + (size_t)blockIdx.z * w_bs;
+    TC* Cb = C + (size_t)blockIdx.z * c_bs;
+    float acc[2][8][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f; }
+    const int KT = (K + GM_BK - 1) / GM_BK;
+    auto load_stage = [&](int st, int kt) {
+        constexpr int CHK = GM_BK / 8;
+#pragma unroll
+        for (int i = 0; i < GW_BM * CHK / 256; ++i) {
+            const int idx = tid + 256 * i, r = idx / CHK, c = idx % CHK, k = kt * GM_BK + c * 8;
+            const bool oka = m0 + r < M && k < K, okw = n0 + r < N && k < K;
+            gm_cp_async16(&As[st][r][c * 8], oka ? Ab + (size_t)(m0 + r) * lda + k : Ab, oka);
+            gm_cp_async16(&Ws[st][r][c * 8], okw ? Wb + (size_t)(n0 + r) * ldw + k : Wb, okw);
+        }
+    };
+    for (int s = 0; s < nst - 1; ++s) {
+        if (s < KT) load_stage(s, s);
+        gm_commit();
+    }
+    for (int kt = 0; kt < KT; ++kt) {
+        if (nst == 2) gm_wait<0>(); else gm_wait<1>();
+        __syncthreads();
+        const int nk = kt + nst - 1;
+        if (nk < KT) load_stage(nk % nst, nk);
+        gm_commit();
+        const int st = kt % nst;
+#pragma unroll
+        for (int kk = 0; kk < GM_BK / 16; ++kk) {
+            unsigned a[2][4];
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+                gm_ldmatrix_x4(a[i], &As[st][wm * 32 + i * 16 + (lane & 15)][kk * 16 + (lane >> 4) * 8]);
+#pragma unroll
+            for (int np = 0; np < 4; ++np) {
+                unsigned b[4];
+                gm_ldmatrix_x4(b, &Ws[st][wn * 64 + np * 16 + (lane & 7) + ((lane >> 4) << 3)][kk * 16 + ((lane >> 3) & 1) * 8]);
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    gm_mma16816(acc[i][2 * np], a[i], b[0], b[1]);
+                    gm_mma16816(acc[i][2 * np + 1], a[i], b[2], b[3]);
+                }
+            }
+        }
+    }
+    gm_wait<0>();
+    const int g = lane >> 2, t2 = (lane & 3) * 2;
+    const bool even = ((ldc | c_bs) & 1) == 0 && (((uintptr_t)C) & (2 * sizeof(TC) - 1)) == 0;
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int m = m0 + wm * 32 + i * 16 + g + half * 8;
+            if (m >= M) continue;
+            TC* crow = Cb + (size_t)m * ldc;
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt) {
+                const int n = n0 + wn * 64 + nt * 8 + t2;
+                const float v0 = acc[i][nt][2 * half], v1 = acc[i][nt][2 * half + 1];
+                if (even && n + 1 < N) {
+                    if (sizeof(TC) == 4) {
+                        *reinterpret_cast<float2*>(crow + n) = make_float2(v0, v1);
+                    } else {
+                        __nv_bfloat162 pr = __floats2bfloat162_rn(v0, v1);
+                        *reinterpret_cast<unsigned*>(crow + n) = *reinterpret_cast<unsigned*>(&pr);
+                    }
+                } else {
+                    if (n < N) crow[n] = from_f32<TC>(v0);
+                    if (n + 1 < N) crow[n + 1] = from_f32<TC>(v1);
+                }
+            }
+        }
+}
+#define GW_MIN_ROWS 512
+template <typename TC>
+static int launch_batched_wide(const bf16* A, const bf16* W, TC* C, int M, int N, int K, int lda, int ldw, int ldc, long long a_bs,
+                               long long w_bs, long long c_bs, int batch, cudaStream_t s) {
+    const dim3 grid((N + GW_BN - 1) / GW_BN, (M + GW_BM - 1) / GW_BM, batch);
+    const int KT = (K + GM_BK - 1) / GM_BK, nst = KT < 2 ? 2 : (KT > GW_NST ? GW_NST : KT);
+    const size_t stage = (size_t)(GW_BM + GW_BN) * GM_LDS * sizeof(bf16);
+    static bool ready = false;                               // per instantiation
+    if (!ready) {
+        cudaError_t e = cudaFuncSetAttribute(gemm_batched_bf16_wide_kernel<TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(GW_NST * stage));
+        if (e != cudaSuccess) return (int)e;
+        ready = true;
+    }
+    return vl_launch(gemm_batched_bf16_wide_kernel<TC>, grid, dim3(256), nst * stage, s, A, W, C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, nst);
+}
+
 static bool gm_aligned(const void* A, const void* W, int K, int lda, int ldw, long long a_bs, long long w_bs, long long w_gs) {
     return !(K % 8 || lda % 8 || ldw % 8 || a_bs % 8 || w_bs % 8 || w_gs % 8 || (((uintptr_t)A | (uintptr_t)W) & 15));
 }
@@ -329,6 +438,9 @@ extern "C" int vl_gemm_batched_nt(const void* A, const void* W, void* C, int dty
         return launch_batched<float, float>((const float*)A, (const float*)W, (float*)C, M, N, K, lda, ldw, ldc,
                                      a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, s);
     if (dtype == VL_BF16 && c_dtype == VL_F32) {
+        if (!tile_group && M >= GW_MIN_ROWS && N >= 96 && (M + GW_BM - 1) / GW_BM <= 65535 && batch <= 65535 &&
+            gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
+            return launch_batched_wide((const bf16*)A, (const bf16*)W, (float*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, batch, s);
         if (gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
             return launch_batched_mma((const bf16*)A, (const bf16*)W, (float*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs,
                                       batch, tile_group, w_gs, bm, nullptr, 1, nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f, s);

@@ -90,7 +90,7 @@ _SIGNATURES = {
     ("flash_attn", "vl_flash_decode"): [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                         c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int,
                                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                        c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p],
+                                        c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p],
     ("flash_attn", "vl_flash_decode_fused"): [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                               c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int,
                                               c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -699,7 +699,7 @@ def flash_decode_streams(dtype, num_tokens, num_kv_heads, head_dim, page_size, m
 def flash_decode(qkv, out, k_cache, v_cache, block_table, req_index, positions, num_heads, num_kv_heads,
                  head_dim, scale, window, max_context, part_acc, part_ml, err, chunk=DECODE_CHUNK, token_index=None,
                  stream_kernel=None, arrivals=None, fold=None, sinks=None, weighting="softmax", mask_chunk=None,
-                 head_bias=None, gate=None, softcap=None, distance=None, keep=None):
+                 head_bias=None, gate=None, softcap=None, distance=None, keep=None, numbered=False):
     """Tensor-core version of `decode_attention` (bfloat16): every block takes a chunk of a token's
     keys; the chunks are merged by the block that finishes last (`arrivals`: int32 counters,
     `flash_decode_arrivals` of them, zero before the first call and left zero) or, without
@@ -717,13 +717,14 @@ def flash_decode(qkv, out, k_cache, v_cache, block_table, req_index, positions, 
     go with the block-per-chunk kernel that merges its chunks itself (`arrivals` given, few enough chunks).
     `softcap`, `distance` (see `_check_score_shape`) go with the block-per-chunk kernel, merged either way.  `keep` (see
     `_check_keep`) goes with the block-per-chunk kernel that merges its chunks itself; `max_context` then bounds the number
-    of keys a token reads (window + keep at most), not its position."""
+    of keys a token reads (window + keep at most), not its position.  `numbered`: the same for a window without kept keys."""
     keep = _check_keep(keep, window, mask_chunk)
+    numbered = bool(keep or (numbered and window))
     _flash_checks(qkv, k_cache, v_cache, block_table, num_heads, num_kv_heads, head_dim)
     _check_sinks(sinks, num_heads)
     mode, mask_chunk, gate_stride = _check_variant(qkv, num_heads, weighting, mask_chunk, head_bias, gate, sinks)
     cap, dist_a, dist_b = _check_score_shape(num_heads, softcap, distance)
-    variant = bool(mode or mask_chunk or gate is not None or keep)
+    variant = bool(mode or mask_chunk or gate is not None or numbered)
     if (variant or cap or dist_a is not None) and fold is not None:
         raise KernelError("flash_decode: the folded head work goes with the plain softmax")
     if cap or dist_a is not None:
@@ -746,7 +747,7 @@ def flash_decode(qkv, out, k_cache, v_cache, block_table, req_index, positions, 
         raise KernelError(f"flash_decode: scratch too small ({part_acc.numel()} < {need_acc})")
     if variant:
         if stream_kernel or arrivals is None or S > _own_merge_cap(head_dim):
-            raise KernelError("flash_decode: weighting, mask chunk, gate and kept keys go with the kernel that merges its chunks itself")
+            raise KernelError("flash_decode: weighting, mask chunk, gate and numbered keys go with the kernel that merges its chunks itself")
         stream_kernel = False
     if stream_kernel is None:
         stream_kernel = fold is None and flash_decode_streams(qkv.dtype, T, num_kv_heads, head_dim, k_cache.shape[2], max_context)
@@ -767,7 +768,8 @@ def flash_decode(qkv, out, k_cache, v_cache, block_table, req_index, positions, 
         if fold is None:
             _check(_fn("flash_attn", "vl_flash_decode", {"FA_HD": head_dim})(
                 *args, _ptr(out) if arrivals is not None else None, _ptr(arrivals), _ptr(sinks), mode, mask_chunk,
-                _ptr(head_bias), _ptr(gate), gate_stride, cap, _ptr(dist_a), _ptr(dist_b), keep, _stream()), "vl_flash_decode")
+                _ptr(head_bias), _ptr(gate), gate_stride, cap, _ptr(dist_a), _ptr(dist_b), keep, int(numbered),
+                _stream()), "vl_flash_decode")
         else:
             qw, kw, eps, inv_freq, rot, slots = fold
             for t, n in ((qw, "q_weight"), (kw, "k_weight"), (inv_freq, "inv_freq")):
@@ -1508,7 +1510,9 @@ def short_conv(x, col0, C, weight, bias, state, state_off, cu, slots, out, act=T
                                              _ptr(in_bias), taps,
                                              sp, stride, _ptr(cu), _ptr(slots), B, int(longest or max(x.shape[0], 1)), _ptr(out),
                                              dtype_code(out.dtype) if out is not None else F32, int(bool(act)), _stream()), "vl_short_conv")
-    if out is not None and int(longest or x.shape[0]) > 64:
+    wide = (out is not None and taps <= 4 and C % 8 == 0 and x.shape[1] % 8 == 0 and col0 % 8 == 0 and stride % 4 == 0
+            and (x.data_ptr() | out.data_ptr() | sp) % 16 == 0)       # (csrc/recurrent.cu: one launch for any step)
+    if out is not None and not wide and int(longest or x.shape[0]) > 64:
         global launch_count
         launch_count += 1           # requests cut among blocks: the new state is a launch of its own
     return out

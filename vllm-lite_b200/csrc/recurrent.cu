@@ -10,7 +10,7 @@
 //                   first token; the last taps-1 inputs of every channel are part of the state (`longest`: a bound
 //                   on the tokens a request brings, which says how many blocks share a request).  `in_bias`: a
 //                   number per channel added to every input row as it is read (the bias of the product that made
-//                   the rows, left to this kernel); the state keeps the rows with it
+//                   the rows, left to this kernel); the state keeps the rows with it.  Two kernels, the same bits
 //   vl_token_shift  h[t] = x[t] + (x[t-1] - x[t]) mu, the row before a portion's first token being part of the state
 //   vl_ssd_scan     S <- exp(-exp(A_log) dt) S + dt B x^T,  y = S^T C + D x          (S: N x P per head, dt =
 //                   softplus(raw + bias); heads share B and C in groups)
@@ -116,6 +116,90 @@ short_conv_kernel(const TP* __restrict__ in, int ld, int col0, int C, const floa
     }
 }
 
+// The same with 16-byte accesses, for 1 to 4 taps, channels in eights and everything on 16-byte boundaries: a thread owns 8
+// channels and CONV_RUN neighbouring tokens of one request, whose rows (and the taps - 1 before them) are loaded together and
+// pass through a window in registers; a channel's sum runs over the taps in the same order.  The thread of a request's first
+// tokens alone touches the state: it reads the old rows, then leaves the portion's last inputs, so one launch serves any step.
+#define CONV_RUN 8
+#define CONV_VEC_THREADS 128
+template <typename TP, typename TO, int TAPS>
+__global__ void __launch_bounds__(CONV_VEC_THREADS)
+short_conv_vec_kernel(const TP* __restrict__ in, int ld, int col0, int C, const float* __restrict__ w,
+                      const float* __restrict__ bias, const float* __restrict__ in_bias, float* state,
+                      long long state_stride, const int* __restrict__ cu, const int* __restrict__ slots, TO* __restrict__ out, int act) {
+    constexpr int BACK = TAPS - 1;
+    pdl_launch_dependents();
+    const int b = blockIdx.y, s0 = cu[b], n = cu[b + 1] - s0;
+    const int first = blockIdx.z * CONV_RUN, c = 8 * (blockIdx.x * CONV_VEC_THREADS + threadIdx.x);
+    if (n <= 0 || first >= n || c >= C) return;
+    float wt[TAPS][8], ib[8], bs[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        ib[i] = in_bias ? in_bias[c + i] : 0.f;
+        bs[i] = bias ? bias[c + i] : 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) wt[j][i] = w[(size_t)(c + i) * TAPS + j];
+    }
+    pdl_wait();
+    float* st = state + (long long)slots[b] * state_stride + c;
+    const TP* src = in + (size_t)s0 * ld + col0 + c;
+    const int m = min(CONV_RUN, n - first);
+    float x[CONV_RUN + BACK][8];                                      // the rows first - BACK .. first + CONV_RUN - 1
+#pragma unroll
+    for (int k = 0; k < CONV_RUN + BACK; ++k) {
+        const int at = first - BACK + k;
+        if (at < 0) {
+            load8(st + (size_t)(at + BACK) * C, x[k]);
+        } else if (at < first + m) {
+            load8(src + (size_t)at * ld, x[k]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) x[k][i] += ib[i];
+        }
+    }
+    if (BACK > 0 && first == 0) {                                     // the new state: the last BACK inputs of old rows and portion
+        float keep[BACK > 0 ? BACK : 1][8];
+#pragma unroll
+        for (int j = 0; j < BACK; ++j) {
+            const int at = n - BACK + j;
+            if (at < 0) {
+                load8(st + (size_t)(at + BACK) * C, keep[j]);
+            } else {
+                load8(src + (size_t)at * ld, keep[j]);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) keep[j][i] += ib[i];
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < BACK; ++j) store8(st + (size_t)j * C, keep[j]);
+    }
+#pragma unroll
+    for (int k = 0; k < CONV_RUN; ++k) {
+        if (k >= m) break;
+        float acc[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            acc[i] = bs[i];
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) acc[i] += wt[j][i] * x[k + j][i];
+            if (act) acc[i] = silu_f(acc[i]);
+        }
+        store8(out + (size_t)(s0 + first + k) * C + c, acc);
+    }
+}
+template <typename TP, typename TO>
+static int launch_short_conv_vec(const TP* in, int ld, int col0, int C, const float* w, const float* bias, const float* in_bias, int taps,
+                                 float* state, long long state_stride, const int* cu, const int* slots, int B, int longest, TO* out,
+                                 int act, cudaStream_t s) {
+    const dim3 grid((C / 8 + CONV_VEC_THREADS - 1) / CONV_VEC_THREADS, B, (longest + CONV_RUN - 1) / CONV_RUN), block(CONV_VEC_THREADS);
+#define CONV_VEC(TAPS) return vl_launch(short_conv_vec_kernel<TP, TO, TAPS>, grid, block, 0, s, in, ld, col0, C, w, bias, in_bias, state, \
+                                        state_stride, cu, slots, out, act)
+    if (taps == 1) CONV_VEC(1);
+    if (taps == 2) CONV_VEC(2);
+    if (taps == 3) CONV_VEC(3);
+    CONV_VEC(4);
+#undef CONV_VEC
+}
+
 extern "C" int vl_short_conv(const void* in, int dtype, int ld, int col0, int C, const float* w, const float* bias,
                              const float* in_bias, int taps, float* state, long long state_stride, const int* cu, const int* slots,
                              int B, int longest, void* out, int out_dtype, int act, void* stream) {
@@ -123,6 +207,17 @@ extern "C" int vl_short_conv(const void* in, int dtype, int ld, int col0, int C,
     if (taps <= 0 || col0 < 0 || col0 + C > ld || longest <= 0) return VL_ERR_ARGUMENT;
     if (out && out_dtype != VL_F32 && out_dtype != dtype) return VL_ERR_UNSUPPORTED;       // float32, or the dtype of the rows
     cudaStream_t s = (cudaStream_t)stream;
+    const int runs = (longest + CONV_RUN - 1) / CONV_RUN;
+    if (out && taps <= 4 && C % 8 == 0 && ld % 8 == 0 && col0 % 8 == 0 && state_stride % 4 == 0 && B <= 65535 && runs <= 65535 &&
+        (((uintptr_t)in | (uintptr_t)out | (uintptr_t)state) & 15) == 0) {
+#define CONV_TRY(TP, TO)                                                                                                               \
+        return launch_short_conv_vec<TP, TO>((const TP*)in, ld, col0, C, w, bias, in_bias, taps, state, state_stride, cu, slots, B,   \
+                                             longest, (TO*)out, act, s)
+        if (dtype == VL_F32) CONV_TRY(float, float);
+        if (dtype == VL_BF16 && out_dtype == VL_BF16) CONV_TRY(bf16, bf16);
+        if (dtype == VL_BF16) CONV_TRY(bf16, float);
+#undef CONV_TRY
+    }
     const int cuts = (longest + CONV_TOKENS - 1) / CONV_TOKENS;
     // without `out` only the new state is made (the caller computed the rows itself, from the old state)
     for (int pass = out ? 0 : 1; pass < (cuts > 1 || !out ? 2 : 1); ++pass) {

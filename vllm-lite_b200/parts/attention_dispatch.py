@@ -100,8 +100,15 @@ def run(qkv, out, cache, group, step, spec, scale, fold=None, sinks=None, weight
     args = (qkv, out, cache.k, cache.v, group.block_table, step.req_index, step.positions,
             spec.num_heads, spec.num_kv_heads, spec.head_dim, scale, spec.window)
     if ops.flash_supported(qkv.dtype, spec.head_dim):
+        # a window much shorter than the context: single tokens count the keys they read, so that no block is started for
+        # positions behind the window (64 tokens x 4 key heads x 4,096 positions, window 1,024: 87 -> 47 us)
+        def single(tokens, context, **kw):
+            short = fold is None and spec.window and 2 * int(spec.window) <= int(context) and not getattr(spec, "shared_row", False)
+            if short and _merges_itself(ops, spec, tokens, spec.window):
+                return _decode(ops, args, step, spec, group, tokens, int(spec.window), sinks=sinks, shape=dict(numbered=True), **kw)
+            return _decode(ops, args, step, spec, group, tokens, context, sinks=sinks, **kw)
         if step.max_query_len == 1:
-            return _decode(ops, args, step, spec, group, qkv.shape[0], group.max_context, fold=fold, sinks=sinks)
+            return single(qkv.shape[0], group.max_context, fold=fold)
         if step.query_tiles is not None:
             tile_args = (qkv, out, cache.k, cache.v, group.block_table, step.query_tiles,
                          spec.num_heads, spec.num_kv_heads, spec.head_dim, scale, spec.window, step.err)
@@ -110,8 +117,7 @@ def run(qkv, out, cache, group, step, spec, scale, fold=None, sinks=None, weight
             else:
                 ops.flash_prefill(*tile_args, tile_rows=QUERY_TILE, sinks=sinks)
             if step.single_tokens is not None:
-                _decode(ops, args, step, spec, group, step.single_tokens.shape[0], step.single_context,
-                        token_index=step.single_tokens, sinks=sinks)
+                single(step.single_tokens.shape[0], step.single_context, token_index=step.single_tokens)
             return out
     return ops.paged_attention(*args, step.err, sinks=sinks)
 
