@@ -774,7 +774,7 @@ def test_element_wise_recurrences(dtype, kind, C, blocks):
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("kind", ["min_gru", "gated_lru"])
-@pytest.mark.parametrize("n", [128, 129, 1024, 1025, 2500])
+@pytest.mark.parametrize("n", [64, 65, 512, 513, 1024, 2500])
 def test_long_stretches_do_not_depend_on_the_number_of_blocks(kind, n):
     """A long portion alone (one cluster walks it), as a portion of a launch whose longest request is longer, and in two portions
     cut at a stretch's border: the same bits; and the plain recurrence."""
@@ -796,7 +796,7 @@ def test_long_stretches_do_not_depend_on_the_number_of_blocks(kind, n):
     sa, sb, sc = fresh(), fresh(), fresh()
     whole = run(0, n, sa, n)
     assert torch.equal(whole, run(0, n, sb, n + 3000)) and torch.equal(sa, sb)
-    cut = n // 2 // 128 * 128
+    cut = n // 2 // 64 * 64
     if cut:
         assert torch.equal(whole, torch.cat([run(0, cut, sc, cut), run(cut, n, sc, n - cut)])) and torch.equal(sa, sc)
     d = lambda t: t.double().cpu()

@@ -133,12 +133,22 @@ short_conv_vec_kernel(const TP* __restrict__ in, int ld, int col0, int C, const 
     const int first = blockIdx.z * CONV_RUN, c = 8 * (blockIdx.x * CONV_VEC_THREADS + threadIdx.x);
     if (n <= 0 || first >= n || c >= C) return;
     float wt[TAPS][8], ib[8], bs[8];
+    {
+        float flat[8 * TAPS], part[8];                                // the channels' taps lie in a row
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        ib[i] = in_bias ? in_bias[c + i] : 0.f;
-        bs[i] = bias ? bias[c + i] : 0.f;
+        for (int q = 0; q < TAPS; ++q) {
+            load8(w + (size_t)c * TAPS + 8 * q, part);
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) wt[j][i] = w[(size_t)(c + i) * TAPS + j];
+            for (int i = 0; i < 8; ++i) flat[8 * q + i] = part[i];
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            ib[i] = bs[i] = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) wt[j][i] = flat[i * TAPS + j];
+        }
+        if (in_bias) load8(in_bias + c, ib);
+        if (bias) load8(bias + c, bs);
     }
     pdl_wait();
     float* st = state + (long long)slots[b] * state_stride + c;
@@ -209,7 +219,7 @@ extern "C" int vl_short_conv(const void* in, int dtype, int ld, int col0, int C,
     cudaStream_t s = (cudaStream_t)stream;
     const int runs = (longest + CONV_RUN - 1) / CONV_RUN;
     if (out && taps <= 4 && C % 8 == 0 && ld % 8 == 0 && col0 % 8 == 0 && state_stride % 4 == 0 && B <= 65535 && runs <= 65535 &&
-        (((uintptr_t)in | (uintptr_t)out | (uintptr_t)state) & 15) == 0) {
+        (((uintptr_t)in | (uintptr_t)out | (uintptr_t)state | (uintptr_t)w | (uintptr_t)bias | (uintptr_t)in_bias) & 15) == 0) {
 #define CONV_TRY(TP, TO)                                                                                                               \
         return launch_short_conv_vec<TP, TO>((const TP*)in, ld, col0, C, w, bias, in_bias, taps, state, state_stride, cu, slots, B,   \
                                              longest, (TO*)out, act, s)
