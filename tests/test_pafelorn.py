@@ -728,7 +728,7 @@ def test_one_key_that_stands_out_at_every_edge(dtype, H_, G_, D_, page, n, windo
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("kind", ["min_gru", "gated_lru"])
-@pytest.mark.parametrize("C,blocks", [(18, 3), (64, 1), (160, 5), (300, 2)])
+@pytest.mark.parametrize("C,blocks", [(18, 3), (64, 1), (160, 5), (300, 2), (35, 5), (1, 1)])
 def test_element_wise_recurrences(dtype, kind, C, blocks):
     """The scan alone: states carried over single tokens, short portions and portions of several stretches, in slots used in
     another order; the neighbours of its state columns are left alone."""

@@ -1510,7 +1510,7 @@ def short_conv(x, col0, C, weight, bias, state, state_off, cu, slots, out, act=T
                                              _ptr(in_bias), taps,
                                              sp, stride, _ptr(cu), _ptr(slots), B, int(longest or max(x.shape[0], 1)), _ptr(out),
                                              dtype_code(out.dtype) if out is not None else F32, int(bool(act)), _stream()), "vl_short_conv")
-    wide = (out is not None and taps <= 4 and C % 8 == 0 and x.shape[1] % 8 == 0 and col0 % 8 == 0 and stride % 4 == 0
+    wide = (out is not None and taps <= 4 and C % 4 == 0 and x.shape[1] % 4 == 0 and col0 % 4 == 0 and stride % 4 == 0
             and (x.data_ptr() | out.data_ptr() | sp | weight.data_ptr() | (_ptr(bias) or 0) | (_ptr(in_bias) or 0)) % 16 == 0)       # (csrc/recurrent.cu: one launch for any step)
     if out is not None and not wide and int(longest or x.shape[0]) > 64:
         global launch_count

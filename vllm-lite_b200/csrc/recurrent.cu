@@ -116,12 +116,17 @@ short_conv_kernel(const TP* __restrict__ in, int ld, int col0, int C, const floa
     }
 }
 
-// The same with 16-byte accesses, for 1 to 4 taps, channels in eights and everything on 16-byte boundaries: a thread owns 8
+// The same with 8- and 16-byte accesses, for 1 to 4 taps, channels in fours and everything on 16-byte boundaries: a thread owns 4
 // channels and CONV_RUN neighbouring tokens of one request, whose rows (and the taps - 1 before them) are loaded together and
 // pass through a window in registers; a channel's sum runs over the taps in the same order.  The thread of a request's first
 // tokens alone touches the state: it reads the old rows, then leaves the portion's last inputs, so one launch serves any step.
 #define CONV_RUN 8
 #define CONV_VEC_THREADS 128
+template <typename T> __device__ __forceinline__ void conv_load4(const T* p, float* v) {
+    const float4 q = Quad<T>::load(p);
+    v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+}
+template <typename T> __device__ __forceinline__ void conv_store4(T* p, const float* v) { Quad<T>::store(p, make_float4(v[0], v[1], v[2], v[3])); }
 template <typename TP, typename TO, int TAPS>
 __global__ void __launch_bounds__(CONV_VEC_THREADS)
 short_conv_vec_kernel(const TP* __restrict__ in, int ld, int col0, int C, const float* __restrict__ w,
@@ -130,77 +135,71 @@ short_conv_vec_kernel(const TP* __restrict__ in, int ld, int col0, int C, const 
     constexpr int BACK = TAPS - 1;
     pdl_launch_dependents();
     const int b = blockIdx.y, s0 = cu[b], n = cu[b + 1] - s0;
-    const int first = blockIdx.z * CONV_RUN, c = 8 * (blockIdx.x * CONV_VEC_THREADS + threadIdx.x);
+    const int first = blockIdx.z * CONV_RUN, c = 4 * (blockIdx.x * CONV_VEC_THREADS + threadIdx.x);
     if (n <= 0 || first >= n || c >= C) return;
-    float wt[TAPS][8], ib[8], bs[8];
+    float wt[TAPS][4], ib[4] = {0.f, 0.f, 0.f, 0.f}, bs[4] = {0.f, 0.f, 0.f, 0.f};
     {
-        float flat[8 * TAPS], part[8];                                // the channels' taps lie in a row
+        float flat[4 * TAPS];                                         // the channels' taps lie in a row
 #pragma unroll
-        for (int q = 0; q < TAPS; ++q) {
-            load8(w + (size_t)c * TAPS + 8 * q, part);
+        for (int q = 0; q < TAPS; ++q) conv_load4(w + (size_t)c * TAPS + 4 * q, flat + 4 * q);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) flat[8 * q + i] = part[i];
-        }
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            ib[i] = bs[i] = 0.f;
+        for (int i = 0; i < 4; ++i)
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) wt[j][i] = flat[i * TAPS + j];
-        }
-        if (in_bias) load8(in_bias + c, ib);
-        if (bias) load8(bias + c, bs);
+        if (in_bias) conv_load4(in_bias + c, ib);
+        if (bias) conv_load4(bias + c, bs);
     }
     pdl_wait();
     float* st = state + (long long)slots[b] * state_stride + c;
     const TP* src = in + (size_t)s0 * ld + col0 + c;
     const int m = min(CONV_RUN, n - first);
-    float x[CONV_RUN + BACK][8];                                      // the rows first - BACK .. first + CONV_RUN - 1
+    float x[CONV_RUN + BACK][4];                                      // the rows first - BACK .. first + CONV_RUN - 1
 #pragma unroll
     for (int k = 0; k < CONV_RUN + BACK; ++k) {
         const int at = first - BACK + k;
         if (at < 0) {
-            load8(st + (size_t)(at + BACK) * C, x[k]);
+            conv_load4(st + (size_t)(at + BACK) * C, x[k]);
         } else if (at < first + m) {
-            load8(src + (size_t)at * ld, x[k]);
+            conv_load4(src + (size_t)at * ld, x[k]);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) x[k][i] += ib[i];
+            for (int i = 0; i < 4; ++i) x[k][i] += ib[i];
         }
     }
     if (BACK > 0 && first == 0) {                                     // the new state: the last BACK inputs of old rows and portion
-        float keep[BACK > 0 ? BACK : 1][8];
+        float keep[BACK > 0 ? BACK : 1][4];
 #pragma unroll
         for (int j = 0; j < BACK; ++j) {
             const int at = n - BACK + j;
             if (at < 0) {
-                load8(st + (size_t)(at + BACK) * C, keep[j]);
+                conv_load4(st + (size_t)(at + BACK) * C, keep[j]);
             } else {
-                load8(src + (size_t)at * ld, keep[j]);
+                conv_load4(src + (size_t)at * ld, keep[j]);
 #pragma unroll
-                for (int i = 0; i < 8; ++i) keep[j][i] += ib[i];
+                for (int i = 0; i < 4; ++i) keep[j][i] += ib[i];
             }
         }
 #pragma unroll
-        for (int j = 0; j < BACK; ++j) store8(st + (size_t)j * C, keep[j]);
+        for (int j = 0; j < BACK; ++j) conv_store4(st + (size_t)j * C, keep[j]);
     }
 #pragma unroll
     for (int k = 0; k < CONV_RUN; ++k) {
         if (k >= m) break;
-        float acc[8];
+        float acc[4];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
+        for (int i = 0; i < 4; ++i) {
             acc[i] = bs[i];
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) acc[i] += wt[j][i] * x[k + j][i];
             if (act) acc[i] = silu_f(acc[i]);
         }
-        store8(out + (size_t)(s0 + first + k) * C + c, acc);
+        conv_store4(out + (size_t)(s0 + first + k) * C + c, acc);
     }
 }
 template <typename TP, typename TO>
 static int launch_short_conv_vec(const TP* in, int ld, int col0, int C, const float* w, const float* bias, const float* in_bias, int taps,
                                  float* state, long long state_stride, const int* cu, const int* slots, int B, int longest, TO* out,
                                  int act, cudaStream_t s) {
-    const dim3 grid((C / 8 + CONV_VEC_THREADS - 1) / CONV_VEC_THREADS, B, (longest + CONV_RUN - 1) / CONV_RUN), block(CONV_VEC_THREADS);
+    const dim3 grid((C / 4 + CONV_VEC_THREADS - 1) / CONV_VEC_THREADS, B, (longest + CONV_RUN - 1) / CONV_RUN), block(CONV_VEC_THREADS);
 #define CONV_VEC(TAPS) return vl_launch(short_conv_vec_kernel<TP, TO, TAPS>, grid, block, 0, s, in, ld, col0, C, w, bias, in_bias, state, \
                                         state_stride, cu, slots, out, act)
     if (taps == 1) CONV_VEC(1);
@@ -218,7 +217,7 @@ extern "C" int vl_short_conv(const void* in, int dtype, int ld, int col0, int C,
     if (out && out_dtype != VL_F32 && out_dtype != dtype) return VL_ERR_UNSUPPORTED;       // float32, or the dtype of the rows
     cudaStream_t s = (cudaStream_t)stream;
     const int runs = (longest + CONV_RUN - 1) / CONV_RUN;
-    if (out && taps <= 4 && C % 8 == 0 && ld % 8 == 0 && col0 % 8 == 0 && state_stride % 4 == 0 && B <= 65535 && runs <= 65535 &&
+    if (out && taps <= 4 && C % 4 == 0 && ld % 4 == 0 && col0 % 4 == 0 && state_stride % 4 == 0 && B <= 65535 && runs <= 65535 &&
         (((uintptr_t)in | (uintptr_t)out | (uintptr_t)state | (uintptr_t)w | (uintptr_t)bias | (uintptr_t)in_bias) & 15) == 0) {
 #define CONV_TRY(TP, TO)                                                                                                               \
         return launch_short_conv_vec<TP, TO>((const TP*)in, ld, col0, C, w, bias, in_bias, taps, state, state_stride, cu, slots, B,   \
