@@ -321,6 +321,24 @@ def test_frequencies_slowed_down(r):
     assert got.dtype == np.float32 and np.allclose(got, want, rtol=1e-6, atol=0)
 
 
+@pytest.mark.parametrize("which", ["A", "B", "C", "D"])
+def test_cache_sizing_counts_the_buffers_of_every_mixer(which):
+    from vllm_lite_b200.cache.sizing import _mixer_width
+    from vllm_lite_b200.config import plan_from_config_json
+    for b in plan_from_config_json(CONFIGS[which])[1].layers:
+        m = b.mixer
+        if m.kind == "differential_attention":
+            P_ = -(-max(2 * m.dim, m.vdim) // 16) * 16
+            assert _mixer_width(m) >= m.num_heads * (2 * m.dim + 4 * P_ + m.vdim) + m.num_kv_heads * (2 * m.dim + m.vdim)
+        else:
+            a = m.left
+            P_ = -(-max(a.head_dim, a.v_head_dim) // 16) * 16
+            attention = (a.num_heads + a.num_kv_heads) * a.head_dim + a.num_kv_heads * a.v_head_dim + (2 + (a.gate is not None)) * a.num_heads * P_
+            assert _mixer_width(a) >= attention
+            assert _mixer_width(m.right) == (8 if m.right.kind == "gated_lru" else 4) * m.right.width
+            assert _mixer_width(m) >= _mixer_width(a) + _mixer_width(m.right)
+
+
 def test_plain_pieces_behave():
     d = lambda v: torch.tensor(v, dtype=torch.float64)
     assert P.bigram_rows([4, 2, 7], dict(buckets=10, mul_prev=3, mul_cur=5)) == [10, (12 + 10) % 10, (6 + 35) % 10]

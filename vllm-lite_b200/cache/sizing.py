@@ -48,7 +48,17 @@ def _mixer_width(mixer) -> int:
     if hasattr(mixer, "num_kv_heads") and hasattr(mixer, "head_dim"):
         hd = max(mixer.head_dim, getattr(mixer, "v_head_dim", None) or 0)
         gate = mixer.num_heads if getattr(mixer, "gate", None) else 0  # an output gate as wide as the heads
+        if getattr(mixer, "whole_norm", False) or getattr(mixer, "head_temp", None):
+            gate += mixer.num_heads                                    # the head work writes its queries to rows of their own
         return (2 * mixer.num_heads + 2 * mixer.num_kv_heads + gate) * (-(-hd // 16) * 16)
+    if hasattr(mixer, "diff"):
+        # differential attention: the stacked product, padded query rows and outputs of both maps, the combined heads
+        row = -(-max(2 * mixer.dim, mixer.vdim) // 16) * 16 + 16
+        return 6 * mixer.num_heads * row + 2 * mixer.num_kv_heads * row + mixer.num_heads * mixer.vdim
+    if hasattr(mixer, "width") and hasattr(mixer, "blocks"):           # linear recurrent unit: y, x, conv, float32 gates, gated
+        return (2 + 1 + 4 + 1) * mixer.width
+    if hasattr(mixer, "width") and not hasattr(mixer, "kv_rank"):      # minimal gated recurrence: z, x, gate, gated
+        return 4 * mixer.width
     if hasattr(mixer, "kv_rank"):
         # latent attention: both latents (and the rotated key part), the queries, their absorbed form and the context
         # (heads x cached row, the row rounded up to 16), the expanded values, the output gate
