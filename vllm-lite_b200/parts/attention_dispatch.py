@@ -101,7 +101,7 @@ def run(qkv, out, cache, group, step, spec, scale, fold=None, sinks=None, weight
             spec.num_heads, spec.num_kv_heads, spec.head_dim, scale, spec.window)
     if ops.flash_supported(qkv.dtype, spec.head_dim):
         # a window much shorter than the context: single tokens count the keys they read, so that no block is started for
-        # positions behind the window (64 tokens x 4 key heads x 4,096 positions, window 1,024: 87 -> 47 us)
+        # positions behind the window (64 tokens x 4 key heads x 4,096 positions, window 1,024: 87 -> 35 us)
         def single(tokens, context, **kw):
             short = fold is None and spec.window and 2 * int(spec.window) <= int(context) and not getattr(spec, "shared_row", False)
             if short and _merges_itself(ops, spec, tokens, spec.window):
