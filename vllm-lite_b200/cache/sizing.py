@@ -65,7 +65,8 @@ def _mixer_width(mixer) -> int:
         rot = getattr(mixer, "rot_dim", 0)
         row = -(-(mixer.kv_rank + rot) // 16) * 16
         gate = mixer.num_heads * mixer.vdim if getattr(mixer, "gate", None) else 0
-        return mixer.q_rank + mixer.kv_rank + rot + gate + mixer.num_heads * (mixer.dim + rot + 2 * row + mixer.vdim)
+        gate += mixer.num_heads if getattr(mixer, "head_gate", None) else 0
+        return mixer.q_rank + mixer.kv_rank + rot + gate + 7 + mixer.num_heads * (mixer.dim + rot + 2 * row + mixer.vdim)
     if hasattr(mixer, "state") and hasattr(mixer, "norm_groups"):       # state space: projection, convolved copy, scan, gated
         inner = mixer.num_heads * mixer.vdim
         conv = inner + 2 * mixer.groups * mixer.state
@@ -77,6 +78,12 @@ def _mixer_width(mixer) -> int:
         # time mixing: five mixes of the input, r, k, v and the raw decay in float32, the gate, the scan's result, the gated rows
         hd = mixer.num_heads * mixer.dim
         return 5 * mixer.hidden_size + 8 * hd + hd + 2 * mixer.decay_rank + 2 * hd + hd
+    if hasattr(mixer, "unit_eps") and not hasattr(mixer, "decay_rank"):
+        # delta rule with one decay per head: one product (with the gate, two numbers a head and up to 7 rows of padding), its
+        # convolved float32 copy, the scan's float32 result, the gated rows
+        hp = mixer.num_heads * mixer.vdim
+        conv = 2 * mixer.num_kv_heads * mixer.dim + hp
+        return (conv + hp + 2 * mixer.num_heads + 7) + 2 * conv + 2 * hp + hp
     if hasattr(mixer, "decay_rank"):                                    # delta rule
         hp, hd = mixer.num_heads * mixer.vdim, mixer.num_heads * mixer.dim
         conv = 2 * mixer.num_kv_heads * mixer.dim + hp
@@ -100,6 +107,8 @@ def activation_reserve(plan, max_step_tokens: int, max_requests: int, max_contex
         elif hasattr(ffn, "intermediate_size"):
             w += 3 * ffn.intermediate_size
         widest = max(widest, w)
+    if any(getattr(call, "add_embedding", False) for call in getattr(plan, "order", ())):
+        streams += 1                                          # the embedding's output is kept for the whole step
     per_token = 4 * H * (1 + (streams if streams > 1 else 0)) + itemsize * (widest + 4 * H)
     bounds, b = 1, 1024
     while b < max_context:

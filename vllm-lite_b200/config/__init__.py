@@ -9,3 +9,4 @@ from .tuzisun import TuzisunConfig  # noqa: F401,E402  (registers Tuzisun)
 from .sodonex import SodonexConfig  # noqa: F401,E402  (registers Sodonex)
 from .puturax import PuturaxConfig  # noqa: F401,E402  (registers Puturax)
 from .pafelorn import PafelornConfig  # noqa: F401,E402  (registers Pafelorn)
+from .vekusun import VekusunConfig  # noqa: F401,E402  (registers Vekusun)

@@ -134,10 +134,11 @@ extern "C" int vl_gated_act(const void* gu, void* out, int dtype, int T, int I, 
     return VL_ERR_UNSUPPORTED;
 }
 
-// A function of one argument, element by element in float32: act 16 = the square of max(v, 0), 17 = tanh(v) (the codes
-// continue those of the gated activations, which take two).
+// A function of one argument, element by element in float32: act 16 = the square of max(v, 0), 17 = tanh(v), 18 = gelu(v) =
+// v times the normal distribution function at v (the codes continue those of the gated activations, which take two).
 __device__ __forceinline__ float unary_value(float v, int act) {
     if (act == 16) { v = fmaxf(v, 0.f); return v * v; }
+    if (act == 18) return 0.5f * v * (1.0f + erff(v * 0.70710678f));     // erf(v / sqrt(2))
     return act == 17 ? tanhf(v) : v;
 }
 // VEC = 4: a thread takes four neighbouring values (one 16- or 8-byte access each way), when the buffers allow it.
@@ -157,7 +158,7 @@ __global__ void unary_act_kernel(const T* __restrict__ in, T* __restrict__ out, 
 
 extern "C" int vl_unary_act(const void* in, void* out, int dtype, long long n, int act, void* stream) {
     if (n <= 0) return VL_OK;
-    if (act != 16 && act != 17) return VL_ERR_ARGUMENT;
+    if (act < 16 || act > 18) return VL_ERR_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     const bool vec = n % 4 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0;
     const unsigned blocks = (unsigned)((n / (vec ? 4 : 1) + 255) / 256);

@@ -458,6 +458,137 @@ extern "C" int vl_rmsnorm_add(const void* y, int act_dtype, const float* bias, c
     return VL_ERR_UNSUPPORTED;
 }
 
+// The sum that a stream waits for, formed by the kernel of the norm that reads it next:
+//     x[r] <- (base or x)[r] + mult * (sa * a[r] + sb * b[r]) + add[r] + vec;      h[r] = x[r] / sqrt(mean(x[r]^2) + eps) * w
+// a, b: the results of two sub-layers side by side (activation dtype, either may be null), sa, sb one factor per column (float32,
+// null: ones); base, add: float32 rows; vec: one float32 row for all.  out null: only the sum.  rows given: output row r is made
+// from source row rows[r] and x is left as it is.  A row is kept in registers where it fits (H a multiple of 4, at most
+// 256 * 4 * VPT values); the order of the sums depends on the row length alone.
+template <typename TA>
+struct StreamSumArgs {
+    const float *base, *sa, *sb, *add, *vec;
+    const TA *a, *b;
+    float mult;
+};
+template <typename TA>
+__device__ __forceinline__ float stream_value(const StreamSumArgs<TA>& p, const float* x, size_t row, int i, int H) {
+    const size_t at = row * H + i;
+    float v = p.base ? p.base[at] : x[at];
+    if (p.a) {
+        float d = to_f32(p.a[at]) * (p.sa ? p.sa[i] : 1.f);
+        if (p.b) d += to_f32(p.b[at]) * (p.sb ? p.sb[i] : 1.f);
+        v += p.mult * d;
+    }
+    if (p.add) v += p.add[at];
+    if (p.vec) v += p.vec[i];
+    return v;
+}
+template <typename TA>
+__global__ void __launch_bounds__(256)
+stream_norm_kernel(float* __restrict__ x, const StreamSumArgs<TA> p, const int* __restrict__ rows, const float* __restrict__ w,
+                   float eps, TA* __restrict__ out, int H) {
+    __shared__ float scratch[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r = blockIdx.x;
+    const size_t src = rows ? rows[r] : r;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < H; i += 256) {
+        const float v = stream_value(p, x, src, i, H);
+        ss += v * v;
+    }
+    ss = block_sum<256>(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+    for (int i = threadIdx.x; i < H; i += 256) {
+        const float v = stream_value(p, x, src, i, H);
+        if (!rows) x[src * H + i] = v;                   // this thread alone reads or writes element i
+        if (out) out[(size_t)r * H + i] = from_f32<TA>(v * inv * w[i]);
+    }
+}
+template <typename TA, int VPT>
+__global__ void __launch_bounds__(256)
+stream_norm_vec_kernel(float* __restrict__ x, const StreamSumArgs<TA> p, const int* __restrict__ rows, const float* __restrict__ w,
+                       float eps, TA* __restrict__ out, int H) {
+    __shared__ float scratch[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r = blockIdx.x, H4 = H >> 2;
+    const size_t at = (size_t)(rows ? rows[r] : r) * H;
+    const float* from = (p.base ? p.base : x) + at;
+    float4 v[VPT];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+        const int c = threadIdx.x + 256 * i;
+        if (c < H4) {
+            v[i] = Quad<float>::load(from + 4 * c);
+            if (p.a) {
+                float4 d = Quad<TA>::load(p.a + at + 4 * c);
+                if (p.sa) {
+                    const float4 s = Quad<float>::load(p.sa + 4 * c);
+                    d.x *= s.x; d.y *= s.y; d.z *= s.z; d.w *= s.w;
+                }
+                if (p.b) {
+                    const float4 e = Quad<TA>::load(p.b + at + 4 * c);
+                    const float4 s = p.sb ? Quad<float>::load(p.sb + 4 * c) : make_float4(1.f, 1.f, 1.f, 1.f);
+                    d.x += e.x * s.x; d.y += e.y * s.y; d.z += e.z * s.z; d.w += e.w * s.w;
+                }
+                v[i].x += p.mult * d.x; v[i].y += p.mult * d.y; v[i].z += p.mult * d.z; v[i].w += p.mult * d.w;
+            }
+            if (p.add) {
+                const float4 e = Quad<float>::load(p.add + at + 4 * c);
+                v[i].x += e.x; v[i].y += e.y; v[i].z += e.z; v[i].w += e.w;
+            }
+            if (p.vec) {
+                const float4 e = Quad<float>::load(p.vec + 4 * c);
+                v[i].x += e.x; v[i].y += e.y; v[i].z += e.z; v[i].w += e.w;
+            }
+            if (!rows) Quad<float>::store(x + at + 4 * c, v[i]);
+            ss += v[i].x * v[i].x; ss += v[i].y * v[i].y; ss += v[i].z * v[i].z; ss += v[i].w * v[i].w;
+        }
+    }
+    if (!out) return;
+    const float inv = 1.0f / sqrtf(block_sum<256>(ss, scratch) / (float)H + eps);
+    TA* o = out + (size_t)r * H;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+        const int c = threadIdx.x + 256 * i;
+        if (c < H4) {
+            const float4 g = Quad<float>::load(w + 4 * c);
+            Quad<TA>::store(o + 4 * c, make_float4(v[i].x * inv * g.x, v[i].y * inv * g.y, v[i].z * inv * g.z, v[i].w * inv * g.w));
+        }
+    }
+}
+template <typename TA>
+static int launch_stream_norm(float* x, const StreamSumArgs<TA>& p, const int* rows, const float* w, float eps, TA* out, int R, int H,
+                              cudaStream_t s) {
+    const int pieces = (H / 4 + 255) / 256;
+    const bool vec = H % 4 == 0 && (((uintptr_t)x | (uintptr_t)p.base | (uintptr_t)p.sa | (uintptr_t)p.sb | (uintptr_t)p.add |
+                                     (uintptr_t)p.vec | (uintptr_t)p.a | (uintptr_t)p.b | (uintptr_t)w | (uintptr_t)out) & 15) == 0;
+#define STREAM_NORM(KERNEL) return vl_launch(KERNEL, dim3(R), dim3(256), 0, s, x, p, rows, w, eps, out, H)
+    if (vec && pieces <= 1) STREAM_NORM((stream_norm_vec_kernel<TA, 1>));
+    if (vec && pieces <= 2) STREAM_NORM((stream_norm_vec_kernel<TA, 2>));
+    if (vec && pieces <= 4) STREAM_NORM((stream_norm_vec_kernel<TA, 4>));
+    if (vec && pieces <= 8) STREAM_NORM((stream_norm_vec_kernel<TA, 8>));
+    STREAM_NORM(stream_norm_kernel<TA>);
+#undef STREAM_NORM
+}
+
+extern "C" int vl_stream_norm(float* x, const float* base, const void* a, const float* sa, const void* b, const float* sb, float mult,
+                              const float* add, const float* vec, const int* rows, const float* w, float eps, void* out, int act_dtype,
+                              int R, int H, void* stream) {
+    if (R <= 0) return VL_OK;
+    if (H <= 0 || (b && !a) || (out && !w) || (!out && rows)) return VL_ERR_ARGUMENT;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (act_dtype == VL_F32)
+        return launch_stream_norm<float>(x, StreamSumArgs<float>{base, sa, sb, add, vec, (const float*)a, (const float*)b, mult}, rows, w, eps,
+                                         (float*)out, R, H, s);
+    if (act_dtype == VL_BF16)
+        return launch_stream_norm<bf16>(x, StreamSumArgs<bf16>{base, sa, sb, add, vec, (const bf16*)a, (const bf16*)b, mult}, rows, w, eps,
+                                        (bf16*)out, R, H, s);
+    return VL_ERR_UNSUPPORTED;
+}
+
 extern "C" int vl_embed(const int* ids, const void* table, int table_dtype, float* x,
                         int T, int H, int V, float scale, unsigned* err, void* stream) {
     if (T <= 0) return VL_OK;

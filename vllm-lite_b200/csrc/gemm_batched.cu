@@ -19,6 +19,10 @@ static inline bool vl_batched_simt_only() {
     return v && v[0] == '1';
 }
 
+// `gate` (optional): row m of batch b is multiplied by sigmoid(gate[m * gate_ld + b]) before it is rounded (an attention's output
+// gate with one number per head, applied by the product that makes the heads' values).
+__device__ __forceinline__ float gb_sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
+
 #define GB_BN 64
 #define GB_BK 16
 
@@ -26,7 +30,7 @@ template <typename T, typename TW, typename TC, int BM>
 __global__ void __launch_bounds__(256)
 gemm_batched_nt_kernel(const T* __restrict__ A, const TW* __restrict__ W, TC* __restrict__ C, int M, int N, int K,
                        int lda, int ldw, int ldc, long long a_bs, long long w_bs, long long c_bs,
-                       const int* __restrict__ tile_group, long long w_gs) {
+                       const int* __restrict__ tile_group, long long w_gs, const T* __restrict__ gate, int gate_ld) {
     constexpr int TM = BM / 16;
     __shared__ float As[GB_BK][BM + 4];
     __shared__ float Ws[GB_BK][GB_BN + 4];
@@ -81,10 +85,11 @@ gemm_batched_nt_kernel(const T* __restrict__ A, const TW* __restrict__ W, TC* __
     for (int i = 0; i < TM; ++i) {
         const int m = m0 + ty * TM + i;
         if (m >= M) continue;
+        const float open = gate ? gb_sigmoid(to_f32(gate[(size_t)m * gate_ld + blockIdx.z])) : 1.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) Cb[(size_t)m * ldc + n] = from_f32<TC>(acc[i][j]);
+            if (n < N) Cb[(size_t)m * ldc + n] = from_f32<TC>(acc[i][j] * open);
         }
     }
 }
@@ -148,7 +153,7 @@ gemm_batched_bf16_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict_
                              int lda, int ldw, int ldc, long long a_bs, long long w_bs, long long c_bs,
                              const int* __restrict__ tile_group, long long w_gs,
                              const int* __restrict__ row_index, int index_div, const float* __restrict__ row_scale,
-                             int act, float alpha, float limit, float shift, int nst) {
+                             int act, float alpha, float limit, float shift, const bf16* __restrict__ gate, int gate_ld, int nst) {
     constexpr int WARPS_M = BM / 16, WARPS_N = 4 / WARPS_M, WN = GM_BN / WARPS_N, NT = WN / 8;
     // the ring is larger than the 48 KB a kernel may declare: dynamic shared memory
     extern __shared__ __align__(16) unsigned char gm_smem[];
@@ -237,6 +242,7 @@ gemm_batched_bf16_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict_
             const int p = row_index ? row_index[m] : m;
             scale = p >= 0 ? row_scale[p] : 0.f;
         }
+        if (gate) scale = gb_sigmoid(to_f32(gate[(size_t)m * gate_ld + blockIdx.z]));
         TC* crow = Cb + (size_t)m * ldc;
         if (act == GM_ACT_NONE || act >= GM_ACT_UNARY) {
 #pragma unroll
@@ -401,58 +407,59 @@ template <typename TC>
 static int launch_batched_mma(const bf16* A, const bf16* W, TC* C, int M, int N, int K, int lda, int ldw, int ldc,
                               long long a_bs, long long w_bs, long long c_bs, int batch, const int* tile_group,
                               long long w_gs, int bm, const int* row_index, int index_div, const float* row_scale,
-                              int act, float alpha, float limit, float shift, cudaStream_t s) {
+                              int act, float alpha, float limit, float shift, const bf16* gate, int gate_ld, cudaStream_t s) {
     dim3 grid((N + GM_BN - 1) / GM_BN, (M + bm - 1) / bm, batch);
     if (grid.y > 65535 || grid.z > 65535) return VL_ERR_UNSUPPORTED;
     if (bm == 64)
         return launch_mma_kernel<64, TC>(grid, s, K, A, W, C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, tile_group, w_gs,
-                                           row_index, index_div, row_scale, act, alpha, limit, shift);
+                                           row_index, index_div, row_scale, act, alpha, limit, shift, gate, gate_ld);
     return launch_mma_kernel<16, TC>(grid, s, K, A, W, C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, tile_group, w_gs,
-                                       row_index, index_div, row_scale, act, alpha, limit, shift);
+                                       row_index, index_div, row_scale, act, alpha, limit, shift, gate, gate_ld);
 }
 
 template <typename T, typename TC>
 static int launch_batched(const T* A, const T* W, TC* C, int M, int N, int K, int lda, int ldw, int ldc,
                           long long a_bs, long long w_bs, long long c_bs, int batch, const int* tile_group,
-                          long long w_gs, int bm, cudaStream_t s) {
+                          long long w_gs, int bm, const T* gate, int gate_ld, cudaStream_t s) {
     dim3 grid((N + GB_BN - 1) / GB_BN, (M + bm - 1) / bm, batch);
     if (grid.y > 65535 || grid.z > 65535) return VL_ERR_UNSUPPORTED;
     if (bm == 64)
         return vl_launch(gemm_batched_nt_kernel<T, T, TC, 64>, grid, dim3(256), 0, s, A, W, C, M, N, K, lda, ldw, ldc,
-                         a_bs, w_bs, c_bs, tile_group, w_gs);
+                         a_bs, w_bs, c_bs, tile_group, w_gs, gate, gate_ld);
     return vl_launch(gemm_batched_nt_kernel<T, T, TC, 16>, grid, dim3(256), 0, s, A, W, C, M, N, K, lda, ldw, ldc,
-                     a_bs, w_bs, c_bs, tile_group, w_gs);
+                     a_bs, w_bs, c_bs, tile_group, w_gs, gate, gate_ld);
 }
 
 // bm: rows per tile, 64 or 16.  With tile_group, M is the padded number of sorted rows (a multiple of bm).
 // c_dtype: the operands' dtype, or float32 (the sums as they are).
 extern "C" int vl_gemm_batched_nt(const void* A, const void* W, void* C, int dtype, int c_dtype, int M, int N, int K,
                                   int lda, int ldw, int ldc, long long a_bs, long long w_bs, long long c_bs,
-                                  int batch, const int* tile_group, long long w_gs, int bm, void* stream) {
+                                  int batch, const int* tile_group, long long w_gs, int bm, const void* gate, int gate_ld, void* stream) {
     if (M <= 0 || N <= 0 || batch <= 0) return VL_OK;
     if (K <= 0 || lda < K || ldw < K || ldc < N || (bm != 64 && bm != 16)) return VL_ERR_ARGUMENT;
     if (tile_group && M % bm) return VL_ERR_ARGUMENT;
+    if (gate && (tile_group || c_dtype != dtype || gate_ld < batch)) return VL_ERR_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     if (c_dtype != dtype && c_dtype != VL_F32) return VL_ERR_UNSUPPORTED;
     if (dtype == VL_F32)
         return launch_batched<float, float>((const float*)A, (const float*)W, (float*)C, M, N, K, lda, ldw, ldc,
-                                     a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, s);
+                                     a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, (const float*)gate, gate_ld, s);
     if (dtype == VL_BF16 && c_dtype == VL_F32) {
         if (!tile_group && M >= GW_MIN_ROWS && N >= 96 && (M + GW_BM - 1) / GW_BM <= 65535 && batch <= 65535 &&
             gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
             return launch_batched_wide((const bf16*)A, (const bf16*)W, (float*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, batch, s);
         if (gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
             return launch_batched_mma((const bf16*)A, (const bf16*)W, (float*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs,
-                                      batch, tile_group, w_gs, bm, nullptr, 1, nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f, s);
+                                      batch, tile_group, w_gs, bm, nullptr, 1, nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f, nullptr, 0, s);
         return launch_batched<bf16, float>((const bf16*)A, (const bf16*)W, (float*)C, M, N, K, lda, ldw, ldc,
-                                           a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, s);
+                                           a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, nullptr, 0, s);
     }
     if (dtype == VL_BF16) {
         if (gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
             return launch_batched_mma((const bf16*)A, (const bf16*)W, (bf16*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs,
-                                      batch, tile_group, w_gs, bm, nullptr, 1, nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f, s);
+                                      batch, tile_group, w_gs, bm, nullptr, 1, nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f, (const bf16*)gate, gate_ld, s);
         return launch_batched<bf16, bf16>((const bf16*)A, (const bf16*)W, (bf16*)C, M, N, K, lda, ldw, ldc,
-                                    a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, s);
+                                    a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, (const bf16*)gate, gate_ld, s);
     }
     return VL_ERR_UNSUPPORTED;
 }
@@ -475,11 +482,11 @@ extern "C" int vl_gemm_rows_f32w(const void* A, int a_dtype, const void* W, int 
         // both operands bfloat16: their products are exact in float32, the tensor cores add them in float32
         return launch_mma_kernel<16, float>(grid, s, Kc, (const bf16*)A, (const bf16*)W, C, M, N, Kc, K, K, N, (long long)Kc,
                                             (long long)Kc, cs, (const int*)nullptr, 0ll, (const int*)nullptr, 1,
-                                            (const float*)nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f);
+                                            (const float*)nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f, (const bf16*)nullptr, 0);
     }
 #define ROWS_CASE(TA, TWV)                                                                                          \
     return vl_launch(gemm_batched_nt_kernel<TA, TWV, float, 16>, grid, dim3(256), 0, s, (const TA*)A, (const TWV*)W, C, M, N, \
-                     Kc, K, K, N, (long long)Kc, (long long)Kc, cs, (const int*)nullptr, 0ll)
+                     Kc, K, K, N, (long long)Kc, (long long)Kc, cs, (const int*)nullptr, 0ll, (const TA*)nullptr, 0)
     if (a_dtype == VL_F32 && w_dtype == VL_F32) ROWS_CASE(float, float);
     if (a_dtype == VL_BF16 && w_dtype == VL_F32) ROWS_CASE(bf16, float);
     if (a_dtype == VL_BF16 && w_dtype == VL_BF16) ROWS_CASE(bf16, bf16);
@@ -489,7 +496,7 @@ extern "C" int vl_gemm_rows_f32w(const void* A, int a_dtype, const void* W, int 
 
 // 1 when `vl_gemm_grouped_fused` takes these sizes (bfloat16 only): rows of A and W on 16-byte boundaries.
 extern "C" int vl_gemm_grouped_fused_ok(int K, int N, int act) {
-    return K % 8 == 0 && (act == GM_ACT_NONE || act >= GM_ACT_UNARY || N % 16 == 0) && !vl_batched_simt_only();
+    return K % 8 == 0 && act <= GM_ACT_UNARY && (act == GM_ACT_NONE || act == GM_ACT_UNARY || N % 16 == 0) && !vl_batched_simt_only();
 }
 
 // The grouped product of a routed feed-forward with its neighbours folded in (bfloat16, tensor cores):
@@ -505,5 +512,5 @@ extern "C" int vl_gemm_grouped_fused(const void* A, const void* W, void* C, int 
     if (act < GM_ACT_NONE || (act > 2 && act != GM_ACT_UNARY) || ldc < (gated ? N / 2 : N)) return VL_ERR_ARGUMENT;
     if (!vl_gemm_grouped_fused_ok(K, N, act) || !gm_aligned(A, W, K, lda, K, 0, 0, w_gs)) return VL_ERR_UNSUPPORTED;
     return launch_batched_mma((const bf16*)A, (const bf16*)W, (bf16*)C, M, N, K, lda, K, ldc, 0, 0, 0, 1, tile_group, w_gs, bm,
-                              row_index, index_div, row_scale, act, alpha, limit, shift, (cudaStream_t)stream);
+                              row_index, index_div, row_scale, act, alpha, limit, shift, nullptr, 0, (cudaStream_t)stream);
 }

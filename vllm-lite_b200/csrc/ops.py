@@ -35,6 +35,8 @@ _SIGNATURES = {
     ("embed_norm", "vl_embed"): [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
     ("embed_norm", "vl_rmsnorm_add"): [c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p,
                                        c_float, c_float, c_void_p, c_void_p, c_void_p],
+    ("embed_norm", "vl_stream_norm"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p,
+                                       c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
     ("embed_norm", "vl_embed_pair"): [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_int, c_longlong,
                                       c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
     ("head_work", "vl_head_work"): [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int,
@@ -58,7 +60,7 @@ _SIGNATURES = {
     ("rope_cache", "vl_head_norm_write"): [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int,
                                            c_float, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_longlong,
                                            c_int, c_void_p, c_void_p],
-    ("latent", "vl_rope_heads"): [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
+    ("latent", "vl_rope_heads"): [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p],
     ("activation", "vl_sigmoid_gate"): [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     ("recurrent", "vl_token_shift_multi"): [c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
                                             c_void_p, c_int, c_int, c_int, c_void_p],
@@ -105,10 +107,12 @@ _SIGNATURES = {
     ("activation", "vl_scale_softcap"): [c_void_p, c_longlong, c_float, c_float, c_void_p],
     ("embed_norm", "vl_layernorm_add"): [c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p],
     ("embed_norm", "vl_layernorm_rows"): [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
-    ("latent", "vl_latent_norm_write"): [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p,
-                                         c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
+    ("latent", "vl_latent_norm_write"): [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p,
+                                         c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_float, c_int, c_int, c_int,
+                                         c_void_p, c_void_p, c_void_p],
     ("gemm_batched", "vl_gemm_batched_nt"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                             c_longlong, c_longlong, c_longlong, c_int, c_void_p, c_longlong, c_int, c_void_p],
+                                             c_longlong, c_longlong, c_longlong, c_int, c_void_p, c_longlong, c_int, c_void_p, c_int,
+                                             c_void_p],
     ("gemm_batched", "vl_gemm_grouped_fused"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
                                                 c_longlong, c_int, c_void_p, c_int, c_void_p, c_int, c_float, c_float, c_float,
                                                 c_void_p],
@@ -148,7 +152,7 @@ _SIGNATURES = {
                                      c_void_p],
     ("recurrent", "vl_delta_scan"): [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
                                      c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
-                                     c_int, c_void_p],
+                                     c_int, c_int, c_void_p],
     ("recurrent", "vl_gate_norm"): [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_float, c_void_p,
                                     c_int, c_int, c_int, c_void_p],
 }
@@ -262,6 +266,45 @@ def add_rmsnorm(x, delta, weight, eps, out, rows=None):
     _check(_fn("embed_norm", "vl_add_rmsnorm")(_ptr(x), _ptr(delta), _ptr(rows), _ptr(weight), _ptr(out),
                                                dtype_code(out.dtype), R, H, float(eps), _stream()), "vl_add_rmsnorm")
     return out
+
+
+def stream_norm(x, total, weight=None, eps=0.0, out=None, rows=None):
+    """x[r] <- (base or x)[r] + mult (a_scale a[r] + b_scale b[r]) + rows[r] + vector (`total`: a parts.base.StreamSum), and, with
+    `weight`, out[r] = x[r] / sqrt(mean(x[r]^2) + eps) * weight.  `rows` given: out[r] is made from source row rows[r] and x is left
+    as it is.  float32 arithmetic; a, b and out in one dtype.  Returns out (x without a norm)."""
+    _need(x, torch.float32, "x", 2)
+    T, H = x.shape
+    a, b = (total.a, total.b) if total.a is not None else (total.b, None)      # one sub-layer alone may be either
+    sa, sb = (total.a_scale, total.b_scale) if total.a is not None else (total.b_scale, None)
+    act = out.dtype if out is not None else (a.dtype if a is not None else torch.float32)
+    for t, n in ((a, "a"), (b, "b")):
+        if t is not None:
+            _need(t, act, n, 2)
+            if t.shape != x.shape:
+                raise KernelError(f"stream_norm: {n} has the stream's shape")
+    for t, n in ((total.base, "base"), (total.rows, "rows to add")):
+        if t is not None:
+            _need(t, torch.float32, n, 2)
+            if t.shape != x.shape:
+                raise KernelError(f"stream_norm: {n} have the stream's shape")
+    for t, n in ((sa, "a_scale"), (sb, "b_scale"), (total.vector, "vector"), (weight, "weight")):
+        if t is not None:
+            _need(t, torch.float32, n, 1)
+            if t.shape[0] != H:
+                raise KernelError(f"stream_norm: {n} has one entry per column")
+    R = T if rows is None else rows.shape[0]
+    if rows is not None:
+        _need(rows, torch.int32, "rows", 1)
+    if (out is None) != (weight is None) or (out is None and rows is not None):
+        raise KernelError("stream_norm: a norm has a weight and an output; picked rows are normed")
+    if out is not None:
+        _need(out, None, "out", 2)
+        if out.shape != (R, H):
+            raise KernelError("stream_norm: out holds one row per picked row")
+    _check(_fn("embed_norm", "vl_stream_norm")(
+        _ptr(x), _ptr(total.base), _ptr(a), _ptr(sa), _ptr(b), _ptr(sb), float(total.mult), _ptr(total.rows), _ptr(total.vector),
+        _ptr(rows), _ptr(weight), float(eps), _ptr(out), dtype_code(act), R, H, _stream()), "vl_stream_norm")
+    return out if out is not None else x
 
 
 def add_bias(y, bias):
@@ -815,7 +858,7 @@ def silu_mul(gate_up, out, group=0):
 
 ACTIVATIONS = {"silu": 0, "relu": 1, "capped_swish": 2}
 # functions of ONE argument (an expert without a gate: down(f(up h))); the codes continue the gated ones
-UNARY_ACTIVATIONS = {"relu2": 16, "tanh": 17}           # the square of max(v, 0); tanh
+UNARY_ACTIVATIONS = {"relu2": 16, "tanh": 17, "gelu": 18}           # the square of max(v, 0); tanh; v times the normal distribution function
 
 
 def _act_code(act) -> int:
@@ -947,25 +990,31 @@ def layernorm_rows(x, rows, weight, eps, out):
 
 # ---------------------------------------------------------------- latent attention
 def latent_norm_write(proj, q_rank, kv_rank, q_weight, kv_weight, eps, cq_out, slots, cache, err, rot_dim=0, rotary=None,
-                      positions=None):
+                      positions=None, kv_col=None, q_heads=None):
     """proj [T, >= q_rank + kv_rank] = [a_q | a_kv]: cq_out [T, q_rank] = rmsnorm(a_q) * q_weight; the cache row
     `slots[t]` of `cache` [pages, 1, page_size, width >= kv_rank] = rmsnorm(a_kv) * kv_weight, zero beyond kv_rank
     (slots None or negative: no write).  `rot_dim` > 0: proj carries rot_dim more columns behind a_kv, a key part that is
-    not normed; `rotary` (inv_freq float32 [rot / 2], rot) turns its first rot features by `positions`, and the part is
-    written into the cache row behind the latent."""
-    inv_freq, rot = rotary if rotary is not None else (None, 0)
+    not normed; `rotary` (inv_freq float32 [rot / 2], rot[, factor on sine and cosine]) turns its first rot features by
+    `positions`, and the part is written into the cache row behind the latent.
+    q_rank 0 (q_weight and cq_out None): no query latent; a_kv then starts at column `kv_col`, and `q_heads` = (first column,
+    stride, heads) names the rotated parts of finished query heads before it, which are turned in place."""
+    inv_freq, rot, amp = (tuple(rotary) + (1.0,))[:3] if rotary is not None else (None, 0, 1.0)
+    kv_col = q_rank if kv_col is None else int(kv_col)
+    q_col, q_stride, heads = q_heads if q_heads is not None else (0, 0, 0)
     if rot_dim:
         if rot:
             _need(inv_freq, torch.float32, "inv_freq", 1); _need(positions, torch.int32, "positions", 1)
             if inv_freq.shape[0] != rot // 2 or positions.shape[0] != proj.shape[0]:
                 raise KernelError("latent_norm_write: inv_freq holds rot / 2 numbers, positions one per token")
-        if proj.shape[1] < q_rank + kv_rank + rot_dim or (slots is not None and cache.shape[3] < kv_rank + rot_dim):
+        if proj.shape[1] < kv_col + kv_rank + rot_dim or (slots is not None and cache.shape[3] < kv_rank + rot_dim):
             raise KernelError("latent_norm_write: no room for the rotated key part")
-    _need(proj, None, "proj", 2); _need(cq_out, proj.dtype, "cq_out", 2)
-    _need(q_weight, torch.float32, "q_weight", 1); _need(kv_weight, torch.float32, "kv_weight", 1)
+    _need(proj, None, "proj", 2); _need(kv_weight, torch.float32, "kv_weight", 1)
     T = proj.shape[0]
-    if proj.shape[1] < q_rank + kv_rank or cq_out.shape != (T, q_rank) or q_weight.shape[0] != q_rank \
-            or kv_weight.shape[0] != kv_rank:
+    if q_rank:
+        _need(cq_out, proj.dtype, "cq_out", 2); _need(q_weight, torch.float32, "q_weight", 1)
+        if cq_out.shape != (T, q_rank) or q_weight.shape[0] != q_rank:
+            raise KernelError("latent_norm_write: the query latent's shapes disagree")
+    if proj.shape[1] < kv_col + kv_rank or kv_col < q_rank or kv_weight.shape[0] != kv_rank:
         raise KernelError("latent_norm_write: shapes disagree")
     width, num_slots = kv_rank, 0
     if slots is not None:
@@ -974,21 +1023,21 @@ def latent_norm_write(proj, q_rank, kv_rank, q_weight, kv_weight, eps, cq_out, s
             raise KernelError(f"latent_norm_write: cache {tuple(cache.shape)} does not hold rows of {kv_rank}")
         width, num_slots = cache.shape[3], cache.shape[0] * cache.shape[2]
     _check(_fn("latent", "vl_latent_norm_write")(
-        _ptr(proj), dtype_code(proj.dtype), proj.shape[1], T, int(q_rank), int(kv_rank), _ptr(q_weight), _ptr(kv_weight),
+        _ptr(proj), dtype_code(proj.dtype), proj.shape[1], T, int(q_rank), kv_col, int(kv_rank), _ptr(q_weight), _ptr(kv_weight),
         float(eps), _ptr(cq_out), _ptr(slots), _ptr(cache) if slots is not None else None, max(width, kv_rank + rot_dim),
-        num_slots, int(rot_dim), int(rot if rot_dim else 0), _ptr(inv_freq) if rot_dim else None,
-        _ptr(positions) if rot_dim and rot else None, _ptr(err), _stream()), "vl_latent_norm_write")
+        num_slots, int(rot_dim), int(rot if rot_dim else 0), _ptr(inv_freq) if rot_dim else None, float(amp), int(q_col), int(q_stride),
+        int(heads if rot_dim else 0), _ptr(positions) if rot_dim and rot else None, _ptr(err), _stream()), "vl_latent_norm_write")
     return cq_out
 
 
-def rope_heads(x, col0, stride, heads, inv_freq, rot, positions):
+def rope_heads(x, col0, stride, heads, inv_freq, rot, positions, amp=1.0):
     """In place on x [T, ld]: the features col0 + h * stride + [0, rot) of every head h < heads are turned by the token's
-    position (pairs (i, i + rot/2), angle = position * inv_freq[i] in float32)."""
+    position (pairs (i, i + rot/2), angle = position * inv_freq[i] in float32, sine and cosine times `amp`)."""
     _need(x, None, "x", 2); _need(inv_freq, torch.float32, "inv_freq", 1); _need(positions, torch.int32, "positions", 1)
     if inv_freq.shape[0] != rot // 2 or positions.shape[0] != x.shape[0]:
         raise KernelError("rope_heads: inv_freq holds rot / 2 numbers, positions one per token")
     _check(_fn("latent", "vl_rope_heads")(_ptr(x), dtype_code(x.dtype), x.shape[0], x.shape[1], int(col0), int(stride), int(heads),
-                                          int(rot), _ptr(inv_freq), _ptr(positions), _stream()), "vl_rope_heads")
+                                          int(rot), _ptr(inv_freq), float(amp), _ptr(positions), _stream()), "vl_rope_heads")
     return x
 
 
@@ -1032,17 +1081,24 @@ def sigmoid_gate(x, gate, gate_col=0):
     return x
 
 
-def gemm_heads(a, w, out):
-    """One product per head on column slices: a [T, H*K], w [H, N, K], out [T, H*N] (in a's dtype, or float32);
-    out[:, h*N:(h+1)*N] = a[:, h*K:(h+1)*K] @ w[h]^T.  float32 accumulation in a fixed order over K."""
+def gemm_heads(a, w, out, gate=None, gate_col=0):
+    """One product per head on column slices: a [T, >= H*K], w [H, N, K], out [T, H*N] (in a's dtype, or float32);
+    out[:, h*N:(h+1)*N] = a[:, h*K:(h+1)*K] @ w[h]^T (columns of a behind H*K are not read).  float32 accumulation in a fixed
+    order over K.  `gate` [T, ld] (in a's dtype): head h's sums are multiplied by sigmoid(gate[t, gate_col + h]) before they are rounded."""
     _need(a, None, "a", 2); _need(w, a.dtype, "w", 3); _need(out, None, "out", 2)
     H, N, K = w.shape
     T = a.shape[0]
-    if a.shape[1] != H * K or out.shape != (T, H * N):
+    if a.shape[1] < H * K or out.shape != (T, H * N):
         raise KernelError(f"gemm_heads: shapes disagree a{tuple(a.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
+    gp, gld = None, 0
+    if gate is not None:
+        _need(gate, a.dtype, "gate", 2)
+        if gate.shape[0] != T or gate_col < 0 or gate_col + H > gate.shape[1] or out.dtype != a.dtype:
+            raise KernelError("gemm_heads: the gate has one column per head, and out its dtype")
+        gp, gld = gate.data_ptr() + gate_col * gate.element_size(), gate.shape[1]
     _check(_fn("gemm_batched", "vl_gemm_batched_nt")(
-        _ptr(a), _ptr(w), _ptr(out), dtype_code(a.dtype), dtype_code(out.dtype), T, N, K, H * K, K, H * N, K, N * K, N, H, None, 0,
-        16 if T <= 16 else 64, _stream()), "vl_gemm_batched_nt")
+        _ptr(a), _ptr(w), _ptr(out), dtype_code(a.dtype), dtype_code(out.dtype), T, N, K, a.shape[1], K, H * N, K, N * K, N, H, None, 0,
+        16 if T <= 16 else 64, gp, gld, _stream()), "vl_gemm_batched_nt")
     return out
 
 
@@ -1057,7 +1113,7 @@ def gemm_grouped(rows, w, out, tile_group, bm):
         raise KernelError("gemm_grouped: shapes disagree")
     _check(_fn("gemm_batched", "vl_gemm_batched_nt")(
         _ptr(rows), _ptr(w), _ptr(out), dtype_code(rows.dtype), dtype_code(rows.dtype), cap, N, K, K, K, N, 0, 0, 0, 1, _ptr(tile_group), N * K,
-        int(bm), _stream()), "vl_gemm_batched_nt")
+        int(bm), None, 0, _stream()), "vl_gemm_batched_nt")
     return out
 
 
@@ -1551,18 +1607,21 @@ def mlstm_scan(proj, q_col, k_col, v_col, i_col, f_col, i_bias, f_bias, cap, q_s
     return o
 
 
-def delta_scan(qkv, decay, decay_col, dt_bias, A_log, proj, beta_col, q_scale, unit_eps, state, state_off, cu, slots, o, H, G, D, P):
+def delta_scan(qkv, decay, decay_col, dt_bias, A_log, proj, beta_col, q_scale, unit_eps, state, state_off, cu, slots, o, H, G, D, P,
+               head_decay=False):
+    """The gated delta rule (csrc/recurrent.cu).  `head_decay`: one raw decay (and dt_bias) per head, else one per head and key channel."""
+    per = H if head_decay else H * D
     _need(qkv, torch.float32, "qkv", 2); _need(decay, None, "decay", 2); _need(proj, decay.dtype, "proj", 2)
     _need(o, torch.float32, "o", 2); _need(dt_bias, torch.float32, "dt_bias", 1); _need(A_log, torch.float32, "A_log", 1)
     T = qkv.shape[0]
-    if decay.shape[0] != T or decay_col + H * D > decay.shape[1] or proj.shape[0] != T or o.shape != (T, H * P) or dt_bias.shape[0] != H * D \
+    if decay.shape[0] != T or decay_col + per > decay.shape[1] or proj.shape[0] != T or o.shape != (T, H * P) or dt_bias.shape[0] != per \
             or A_log.shape[0] != H or beta_col + H > proj.shape[1]:
         raise KernelError("delta_scan: shapes disagree")
     B = _seg_args(cu, slots)
     sp, stride = _state_args(state, state_off, scan_state_floats(H, D, P))
     _check(_fn("recurrent", "vl_delta_scan")(_ptr(qkv), qkv.shape[1], _ptr(decay), decay.shape[1], decay_col, _ptr(dt_bias), _ptr(A_log), _ptr(proj),
                                              dtype_code(proj.dtype), proj.shape[1], beta_col, float(q_scale), float(unit_eps),
-                                             sp, stride, _ptr(cu), _ptr(slots), B, _ptr(o), H, G, D, P, _stream()),
+                                             sp, stride, _ptr(cu), _ptr(slots), B, _ptr(o), H, G, D, P, int(bool(head_decay)), _stream()),
            "vl_delta_scan")
     return o
 

@@ -613,10 +613,11 @@ extern "C" int vl_mlstm_scan(const void* proj, int dtype, int ld, int q_col, int
 // qkv float32 [T, C]: q (G*D) | k (G*D) | v (H*P), the convolutions' output.  raw decay: columns dcol .. of `decay` (rows dld wide),
 // raw beta: column beta_col + h of `proj`.  o float32 [T, H*P].
 // Staged per token: q [D] | k [D] | decay [D] | v [CT] | beta; a warp per token then makes q and k unit vectors (q scaled),
-// the decays exp(-rate softplus(raw + bias)) and beta a sigmoid.
-template <typename TP, int ROWS, int L>
-__global__ void __launch_bounds__(RC_MAX_THREADS)
-delta_scan_kernel(const float* __restrict__ qkv, int C, const TP* __restrict__ decay, int dld, int dcol,
+// the decays exp(-rate softplus(raw + bias)) and beta a sigmoid.  HEAD: one decay per head (columns dcol + h, dt_bias [H]); a token
+// then stages one decay in place of D.
+template <typename TP, int ROWS, int L, bool HEAD>
+__device__ __forceinline__ void
+delta_scan_body(const float* __restrict__ qkv, int C, const TP* __restrict__ decay, int dld, int dcol,
                   const float* __restrict__ dt_bias,
                   const float* __restrict__ A_log, const TP* __restrict__ proj, int ld, int beta_col, float q_scale,
                   float unit_eps, float* __restrict__ state, long long state_stride, const int* __restrict__ cu,
@@ -632,7 +633,8 @@ delta_scan_kernel(const float* __restrict__ qkv, int C, const TP* __restrict__ d
     const int p0 = blockIdx.z * CT, p = p0 + col;
     const bool live = p < P;
     const int g = h / (H / G);
-    const int VEC = 3 * D + CT + 1;
+    const int ND = HEAD ? 1 : D, V0 = 2 * D + ND;              // decays of a token; where its value columns begin
+    const int VEC = V0 + CT + 1;
     float* S = scan_state<ROWS>(state, state_stride, slots[b], h);
     float s[ROWS];
 #pragma unroll
@@ -641,8 +643,8 @@ delta_scan_kernel(const float* __restrict__ qkv, int C, const TP* __restrict__ d
     auto raw = [&](int row, int e) -> float {
         const size_t t = (size_t)(s0 + row);
         if (e < 2 * D) return qkv[t * C + (e < D ? (size_t)g * D + e : (size_t)(G + g) * D + (e - D))];
-        if (e < 3 * D) return to_f32(decay[t * dld + dcol + (size_t)h * D + (e - 2 * D)]);
-        if (e < 3 * D + CT) return p0 + (e - 3 * D) < P ? qkv[t * C + (size_t)2 * G * D + (size_t)h * P + p0 + (e - 3 * D)] : 0.f;
+        if (e < V0) return to_f32(decay[t * dld + dcol + (size_t)h * ND + (e - 2 * D)]);
+        if (e < V0 + CT) return p0 + (e - V0) < P ? qkv[t * C + (size_t)2 * G * D + (size_t)h * P + p0 + (e - V0)] : 0.f;
         return to_f32(proj[t * ld + beta_col + h]);
     };
     auto finish = [&](float* buf, int m) {
@@ -656,9 +658,10 @@ delta_scan_kernel(const float* __restrict__ qkv, int C, const TP* __restrict__ d
             for (int r = lane; r < D; r += 32) {
                 v[r] *= qn;
                 v[D + r] *= kn;
-                v[2 * D + r] = expf(-rate * softplus_f(v[2 * D + r] + dt_bias[(size_t)h * D + r]));
+                if (!HEAD) v[2 * D + r] = expf(-rate * softplus_f(v[2 * D + r] + dt_bias[(size_t)h * D + r]));
             }
-            if (lane == 0) v[3 * D + CT] = sigmoid_f(v[3 * D + CT]);
+            if (HEAD && lane == 1) v[2 * D] = expf(-rate * softplus_f(v[2 * D] + dt_bias[h]));
+            if (lane == 0) v[V0 + CT] = sigmoid_f(v[V0 + CT]);
         }
     };
     float pf[RC_PREFETCH];
@@ -680,12 +683,12 @@ delta_scan_kernel(const float* __restrict__ qkv, int C, const TP* __restrict__ d
             for (int i = 0; i < ROWS; ++i) {
                 const int r = l + L * i;
                 if (r < D) {
-                    s[i] *= v[2 * D + r];
+                    s[i] *= HEAD ? v[2 * D] : v[2 * D + r];
                     back += s[i] * v[D + r];
                 }
             }
             back = group_sum<L>(back);
-            const float u = v[3 * D + CT] * (v[3 * D + col] - back);
+            const float u = v[V0 + CT] * (v[V0 + col] - back);
             float acc = 0.f;
 #pragma unroll
             for (int i = 0; i < ROWS; ++i) {
@@ -712,19 +715,39 @@ delta_scan_kernel(const float* __restrict__ qkv, int C, const TP* __restrict__ d
     for (int i = 0; i < ROWS; ++i) S[(size_t)i * NT] = s[i];
 }
 
+#define DELTA_KERNEL(NAME, HEAD)                                                                                                   \
+    template <typename TP, int ROWS, int L>                                                                                        \
+    __global__ void __launch_bounds__(RC_MAX_THREADS)                                                                              \
+    NAME(const float* __restrict__ qkv, int C, const TP* __restrict__ decay, int dld, int dcol, const float* __restrict__ dt_bias, \
+         const float* __restrict__ A_log, const TP* __restrict__ proj, int ld, int beta_col, float q_scale, float unit_eps,        \
+         float* __restrict__ state, long long state_stride, const int* __restrict__ cu, const int* __restrict__ slots,            \
+         float* __restrict__ o, int H, int G, int D, int P, int chunk) {                                                           \
+        delta_scan_body<TP, ROWS, L, HEAD>(qkv, C, decay, dld, dcol, dt_bias, A_log, proj, ld, beta_col, q_scale, unit_eps, state, \
+                                           state_stride, cu, slots, o, H, G, D, P, chunk);                                        \
+    }
+DELTA_KERNEL(delta_scan_kernel, false)
+DELTA_KERNEL(head_delta_scan_kernel, true)
+#undef DELTA_KERNEL
+
 extern "C" int vl_delta_scan(const float* qkv, int C, const void* decay, int dld, int dcol, const float* dt_bias, const float* A_log,
                              const void* proj, int dtype, int ld, int beta_col, float q_scale, float unit_eps, float* state,
                              long long state_stride, const int* cu, const int* slots, int B, float* o, int H, int G, int D,
-                             int P, void* stream) {
+                             int P, int head_decay, void* stream) {
     if (B <= 0) return VL_OK;
     if (H <= 0 || G <= 0 || H % G || D <= 0 || P <= 0 || C != 2 * G * D + H * P) return VL_ERR_ARGUMENT;
     ScanShape sh;
     if (!scan_shape(D, P, &sh)) return VL_ERR_UNSUPPORTED;
-    const int CT = sh.CT, VEC = 3 * D + CT + 1, chunk = scan_chunk(VEC, sh.threads);
+    const int CT = sh.CT, VEC = 2 * D + (head_decay ? 1 : D) + CT + 1, chunk = scan_chunk(VEC, sh.threads);
     if (!chunk) return VL_ERR_UNSUPPORTED;
     dim3 grid(H, B, sh.Z);
     const size_t smem = sizeof(float) * (size_t)2 * chunk * VEC;
     cudaStream_t s = (cudaStream_t)stream;
+    if (head_decay && dtype == VL_F32)
+        SCAN_LAUNCH(head_delta_scan_kernel, float, sh, grid, smem, s, qkv, C, (const float*)decay, dld, dcol, dt_bias, A_log,
+                    (const float*)proj, ld, beta_col, q_scale, unit_eps, state, state_stride, cu, slots, o, H, G, D, P, chunk);
+    if (head_decay && dtype == VL_BF16)
+        SCAN_LAUNCH(head_delta_scan_kernel, bf16, sh, grid, smem, s, qkv, C, (const bf16*)decay, dld, dcol, dt_bias, A_log,
+                    (const bf16*)proj, ld, beta_col, q_scale, unit_eps, state, state_stride, cu, slots, o, H, G, D, P, chunk);
     if (dtype == VL_F32)
         SCAN_LAUNCH(delta_scan_kernel, float, sh, grid, smem, s, qkv, C, (const float*)decay, dld, dcol, dt_bias, A_log,
                     (const float*)proj, ld, beta_col, q_scale, unit_eps, state, state_stride, cu, slots, o, H, G, D, P, chunk);

@@ -132,7 +132,7 @@ class CallCache:
 @dataclass
 class Residual:
     x: torch.Tensor                           # float32 [T, H]
-    pending: Optional[torch.Tensor] = None    # not yet added into x
+    pending: Optional[object] = None          # not yet added into x: a tensor in the activation dtype, or a `StreamSum`
     normed: Optional["ScaledRows"] = None     # output of the norm `normed_for` on x, in factored form
     normed_for: object = None
     cast: Optional[torch.Tensor] = None       # x in the activation dtype, when the kernel that last wrote x left it
@@ -141,9 +141,28 @@ class Residual:
                                               # together with the read that a following block of the same kind asks for
 
     def settle(self):
-        """Bring `x` up to date (blocks that keep several streams write back lazily)."""
+        """Bring `x` up to date (blocks that keep several streams write back lazily; a `StreamSum` waits for the norm
+        that reads the stream next)."""
         if self.deferred is not None:
             self.deferred(None)
+        if isinstance(self.pending, StreamSum):
+            from ..csrc import ops
+            ops.stream_norm(self.x, self.pending)
+            self.pending = None
+
+    def add_before_next(self, rows=None, vector=None):
+        """Have `rows` (float32 [T, H]) and `vector` (float32 [H]) added to the stream before it is read next."""
+        if rows is None and vector is None:
+            return
+        if self.normed is not None:
+            raise NotImplementedError("an addition to a stream whose next norm was left in factored form")
+        if self.deferred is not None or (isinstance(self.pending, StreamSum) and
+                                         (self.pending.rows is not None or self.pending.vector is not None)):
+            self.settle()
+        if not isinstance(self.pending, StreamSum):
+            self.pending = StreamSum(a=self.pending)
+        self.pending.rows, self.pending.vector = rows, vector
+        self.cast = None
 
 
 @dataclass
@@ -182,6 +201,21 @@ class ScaledPair:
     a_weight: Optional[torch.Tensor] = None
     b_weight: Optional[torch.Tensor] = None
     eps: float = 0.0
+
+
+@dataclass
+class StreamSum:
+    """What the stream x still lacks: x <- (base or x) + mult * (a_scale * a + b_scale * b) + rows + vector, the scales per channel
+    (float32 [H], None: ones), in float32.  It waits as `Residual.pending` for the norm that reads the stream next, whose kernel
+    forms the sum on its way (`ops.stream_norm`); a block that does not say `takes_sum` is handed the finished stream."""
+    a: Optional[torch.Tensor] = None          # [T, H], activation dtype
+    a_scale: Optional[torch.Tensor] = None
+    b: Optional[torch.Tensor] = None
+    b_scale: Optional[torch.Tensor] = None
+    mult: float = 1.0
+    base: Optional[torch.Tensor] = None       # float32 [T, H]: where the stream's values are until it is first written
+    rows: Optional[torch.Tensor] = None       # float32 [T, H]
+    vector: Optional[torch.Tensor] = None     # float32 [H]
 
 
 def sub_weights(weights: dict, prefix: str) -> dict:

@@ -11,7 +11,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import StreamSink, prefixed, sub_weights
+from .base import StreamSink, StreamSum, prefixed, sub_weights
 from .registry import BLOCKS, FEED_FORWARDS, MIXERS, NORMS
 from .spec import BlockSpec
 
@@ -225,6 +225,63 @@ def _exact(weights, prefix, norm_spec):
     if getattr(norm_spec, "tensor", "weight") == "":
         return {"": weights[prefix]} if prefix in weights else {}
     return sub_weights(weights, prefix)
+
+
+@BLOCKS.register("shared_norm")
+class SharedNormBlock:
+    """h = norm1(x); x += m (s1 * mixer(h) + s2 * ffn(h)) (m = `spec.residual_mult`, s1 and s2 one factor per channel): both
+    sub-layers read one norm's output.  The sum is left to the norm that reads the stream next (`StreamSum`), so a block
+    launches nothing for it; that norm's kernel also adds what the model puts between two calls.  A block without a
+    feed-forward (`spec.ffn` None) is its mixer alone."""
+
+    takes_sum = True
+
+    @staticmethod
+    def declare(spec: BlockSpec) -> dict:
+        from .spec import TensorDecl
+        norm1, mixer, _, ffn = spec.names
+        size = (spec.norm1.size,)
+        d = prefixed(NORMS.get(spec.norm1.kind).declare(spec.norm1), norm1)
+        d.update(prefixed(MIXERS.get(spec.mixer.kind).declare(spec.mixer), mixer))
+        if spec.scales is not None:
+            d[spec.scales[0]] = TensorDecl(size, init="norm")
+        if spec.ffn is not None:
+            d.update(prefixed(FEED_FORWARDS.get(spec.ffn.kind).declare(spec.ffn), ffn))
+            if spec.scales is not None:
+                d[spec.scales[1]] = TensorDecl(size, init="norm")
+        return d
+
+    @staticmethod
+    def cache_need(spec: BlockSpec):
+        return MIXERS.get(spec.mixer.kind).cache_need(spec.mixer)
+
+    def __init__(self, spec: BlockSpec, weights: dict, ctx):
+        self.spec = spec
+        norm1, mixer, _, ffn = spec.names
+        self.norm1 = NORMS.get(spec.norm1.kind)(spec.norm1, _exact(weights, norm1, spec.norm1), ctx)
+        if not getattr(self.norm1, "takes_sum", False):
+            raise TypeError(f"norm kind {spec.norm1.kind!r} cannot form the stream's sum as it reads (takes_sum)")
+        self.mixer = MIXERS.get(spec.mixer.kind)(spec.mixer, sub_weights(weights, mixer), ctx)
+        self.ffn = None
+        if spec.ffn is not None:
+            self.ffn = FEED_FORWARDS.get(spec.ffn.kind)(spec.ffn, sub_weights(weights, ffn), ctx)
+        scale = lambda i: weights[spec.scales[i]].to(device=ctx.device, dtype=torch.float32).contiguous()
+        self.mixer_scale = self.ffn_scale = None
+        if spec.scales is not None:
+            self.mixer_scale = scale(0)
+            self.ffn_scale = scale(1) if self.ffn is not None else None
+        self.mult = float(spec.residual_mult)
+        self.graph_safe = bool(getattr(self.mixer, "graph_safe", False)
+                               and (self.ffn is None or getattr(self.ffn, "graph_safe", False)))
+
+    def __call__(self, residual, step, cache):
+        if residual.normed is not None:
+            raise NotImplementedError("a shared-norm block after a block that leaves a norm's output in factored form")
+        h = self.norm1(residual.x, residual.pending, step, tag="norm1")
+        residual.cast = None
+        y = self.mixer(h, step, cache)
+        z = self.ffn(h, step) if self.ffn is not None else None
+        residual.pending = StreamSum(y, self.mixer_scale, z, self.ffn_scale, self.mult)
 
 
 @BLOCKS.register("hyper_connection")

@@ -22,8 +22,14 @@ part for all heads; both are rotated by the position and the score is scale * (q
 row is then [c | k_rot]; the query the kernels see is [a_h | q_rot] (the per-head matrix of the absorb step is
 [[W_uk^T, 0], [0, I]]: the identity block hands the rotated part through exactly), and the expand step reads the
 first kv_rank columns of the attention's result alone (zero columns in the per-head matrix).
+The kernels pair feature i with i + dim/2; an encoding that pairs 2i with 2i + 1 is served by reordering the rows of the
+matrices that make both rotated parts when they are bound (q . k does not change when both are reordered alike).
 An output gate (`gate`) multiplies the concatenated heads by sigmoid(W_g h); W_g is stacked under the two
-down-projections, so it costs no product of its own.
+down-projections, so it costs no product of its own.  With one number per head (`head_gate`) the expand step's product
+multiplies its sums by it, so it costs no kernel either.
+
+Without a query latent (`q_rank` 0) the queries are one more block of rows of that first product, and the kernel that norms the
+latent and writes the cache turns their rotated parts too: two launches before the absorb step instead of four.
 """
 from __future__ import annotations
 
@@ -32,7 +38,7 @@ from collections import namedtuple
 import torch
 
 from ..cache.spec import PagedLatent
-from .linear import Linear
+from .linear import Linear, stacked
 from .registry import MIXERS
 from .spec import LatentAttentionSpec, TensorDecl
 
@@ -48,9 +54,13 @@ def padded_rank(kv_rank: int) -> int:
 
 
 def check_latent_sizes(spec: LatentAttentionSpec):
-    for name in ("hidden_size", "num_heads", "dim", "vdim", "q_rank", "kv_rank"):
+    for name in ("hidden_size", "num_heads", "dim", "vdim", "kv_rank"):
         if getattr(spec, name) <= 0:
             raise ValueError(f"latent attention: {name} must be positive, got {getattr(spec, name)}")
+    if spec.q_rank < 0:
+        raise ValueError(f"latent attention: q_rank {spec.q_rank} is negative (0: no query latent)")
+    if spec.gate is not None and spec.head_gate is not None:
+        raise ValueError("latent attention: one output gate, per element (gate) or per head (head_gate)")
     if spec.rot_dim < 0 or (spec.rot_dim > 0) != (spec.position is not None):
         raise ValueError("latent attention: a rotated part (rot_dim) and a position encoding come together")
     if spec.position is not None and (spec.position.dim > spec.rot_dim or spec.position.dim % 2):
@@ -62,6 +72,13 @@ def check_latent_sizes(spec: LatentAttentionSpec):
         raise ValueError(f"window {spec.window} must be positive (None reads every earlier key)")
 
 
+def half_order(pairs_interleaved: int, part: int) -> list:
+    """The order of a part's features in which the first `pairs_interleaved` features, paired 2i with 2i + 1, are paired
+    i with i + half."""
+    n = pairs_interleaved
+    return list(range(0, n, 2)) + list(range(1, n, 2)) + list(range(n, part))
+
+
 @MIXERS.register("latent_attention")
 class LatentAttention:
     graph_safe = True
@@ -70,8 +87,8 @@ class LatentAttention:
     def declare(spec: LatentAttentionSpec) -> dict:
         dq, dqn, uq, dkv, dkvn, uk, uv, o, sink = spec.names
         H = spec.num_heads
-        d = {dq: TensorDecl((spec.q_rank, spec.hidden_size)), dqn: TensorDecl((spec.q_rank,), init="norm"),
-             uq: TensorDecl((H * (spec.dim + spec.rot_dim), spec.q_rank)),
+        d = {} if not spec.q_rank else {dq: TensorDecl((spec.q_rank, spec.hidden_size)), dqn: TensorDecl((spec.q_rank,), init="norm")}
+        d = {**d, uq: TensorDecl((H * (spec.dim + spec.rot_dim), spec.q_rank or spec.hidden_size)),
              dkv: TensorDecl((spec.kv_rank + spec.rot_dim, spec.hidden_size)), dkvn: TensorDecl((spec.kv_rank,), init="norm"),
              uk: TensorDecl((H * spec.dim, spec.kv_rank)), uv: TensorDecl((H * spec.vdim, spec.kv_rank)),
              o: TensorDecl((spec.hidden_size, H * spec.vdim))}
@@ -79,6 +96,8 @@ class LatentAttention:
             d[sink] = TensorDecl((H,))
         if spec.gate is not None:
             d[spec.gate] = TensorDecl((H * spec.vdim, spec.hidden_size))
+        if spec.head_gate is not None:
+            d[spec.head_gate] = TensorDecl((H, spec.hidden_size))
         return d
 
     @staticmethod
@@ -92,19 +111,29 @@ class LatentAttention:
         dq, dqn, uq, dkv, dkvn, uk, uv, o, sink = spec.names
         H, D, V, R, P = spec.num_heads, spec.dim, spec.vdim, spec.kv_rank, spec.rot_dim
         self.rank = padded_rank(R + P)
-        down = [weights[dq], weights[dkv]] + ([weights[spec.gate]] if spec.gate is not None else [])
-        self.down = Linear(torch.cat(down, dim=0).contiguous())
-        self.gate_col = spec.q_rank + R + P if spec.gate is not None else None
+        w_uq, w_dkv = weights[uq], weights[dkv]
+        if spec.position is not None and spec.position.interleaved:
+            order = torch.tensor(half_order(spec.position.dim, P), device=w_dkv.device)
+            w_dkv = torch.cat([w_dkv[:R], w_dkv[R:][order]], dim=0)
+            heads = w_uq.view(H, D + P, -1)
+            w_uq = torch.cat([heads[:, :D], heads[:, D:][:, order]], dim=1).reshape(w_uq.shape)
+        # columns of the first product: queries or their latent, the key/value latent (and rotated key part), the gate
+        first = weights[dq] if spec.q_rank else w_uq
+        gate = spec.gate if spec.gate is not None else spec.head_gate
+        self.down = Linear(stacked([first, w_dkv] + ([weights[gate]] if gate is not None else [])))
+        self.kv_col = first.shape[0]
+        self.gate_col = self.kv_col + R + P
         self.rotary = None
         if spec.position is not None:
             from .registry import POSITIONS
             table = POSITIONS.get(spec.position.kind)(spec.position, {}, ctx)
-            self.rotary = table.fused_rotary()           # (inv_freq, rotated features)
-            if self.rotary is None:
+            ask = getattr(table, "scaled_rotary", None)
+            if ask is None:
                 raise TypeError(f"position kind {spec.position.kind!r} offers no table of inverse frequencies")
-        self.q_norm = weights[dqn].to(device=ctx.device, dtype=torch.float32).contiguous()
+            self.rotary = ask()                          # (inv_freq, rotated features, factor on sine and cosine)
+        self.q_norm = weights[dqn].to(device=ctx.device, dtype=torch.float32).contiguous() if spec.q_rank else None
         self.kv_norm = weights[dkvn].to(device=ctx.device, dtype=torch.float32).contiguous()
-        self.uq = Linear(weights[uq])
+        self.uq = Linear(w_uq.contiguous()) if spec.q_rank else None
         # a_h = W_uk[h]^T q_h: per head a [rank, dim] matrix (the transpose, rows beyond kv_rank zero)
         wk = weights[uk].view(H, D, R)
         absorb = torch.zeros((H, self.rank, D + P), dtype=wk.dtype, device=wk.device)
@@ -130,17 +159,27 @@ class LatentAttention:
         H = s.num_heads
         group = step.groups[cache.group]
         proj = self.down(h, step, "latent.down")
-        cq = ws.get(tag + "latent.cq", (T, s.q_rank), self.dtype)
-        ops.latent_norm_write(proj, s.q_rank, s.kv_rank, self.q_norm, self.kv_norm, s.eps, cq,
-                              group.slots if cache.writes else None, cache.k, step.err, rot_dim=s.rot_dim,
-                              rotary=self.rotary, positions=step.positions)
-        q = self.uq(cq, step, "latent.q")
-        if self.rotary is not None and self.rotary[1] > 0:
-            ops.rope_heads(q, s.dim, s.dim + s.rot_dim, H, self.rotary[0], self.rotary[1], step.positions)
+        slots = group.slots if cache.writes else None
+        write = dict(rot_dim=s.rot_dim, rotary=self.rotary, positions=step.positions)
+        if s.q_rank:
+            cq = ws.get(tag + "latent.cq", (T, s.q_rank), self.dtype)
+            ops.latent_norm_write(proj, s.q_rank, s.kv_rank, self.q_norm, self.kv_norm, s.eps, cq, slots, cache.k, step.err, **write)
+            q = self.uq(cq, step, "latent.q")
+            if self.rotary is not None and self.rotary[1] > 0:
+                ops.rope_heads(q, s.dim, s.dim + s.rot_dim, H, self.rotary[0], self.rotary[1], step.positions, self.rotary[2])
+        else:
+            turned = (s.dim, s.dim + s.rot_dim, H) if s.rot_dim else None
+            ops.latent_norm_write(proj, 0, s.kv_rank, None, self.kv_norm, s.eps, None, slots, cache.k, step.err,
+                                  kv_col=self.kv_col, q_heads=turned, **write)
+            q = proj                                     # the queries are its first columns
         qa = ops.gemm_heads(q, self.absorb, ws.get(tag + "latent.qa", (T, H * self.rank), self.dtype))
         ctx = ws.get(tag + "latent.ctx", (T, H * self.rank), self.dtype)
         attention_dispatch.run(qa, ctx, cache, group, step, self.layout, self.scale, sinks=self.sinks)
-        v = ops.gemm_heads(ctx, self.expand, ws.get(tag + "latent.v", (T, H * s.vdim), self.dtype))
-        if self.gate_col is not None:
+        v = ws.get(tag + "latent.v", (T, H * s.vdim), self.dtype)
+        if s.head_gate is not None:
+            ops.gemm_heads(ctx, self.expand, v, gate=proj, gate_col=self.gate_col)
+        else:
+            ops.gemm_heads(ctx, self.expand, v)
+        if s.gate is not None:
             ops.sigmoid_gate(v, proj, self.gate_col)
         return self.o(v, step, "latent.o")

@@ -13,6 +13,16 @@ import torch
 from .base import ScaledRows, StreamSink
 
 
+def stacked(weights, multiple: int = 8) -> torch.Tensor:
+    """Matrices with the same input, one under the other, and rows of zeros up to a multiple of `multiple` rows: the rows of
+    the product then start on 16-byte boundaries, and whoever reads its columns never looks at the last ones."""
+    rows = sum(w.shape[0] for w in weights)
+    fill = -rows % multiple
+    if fill:
+        weights = list(weights) + [weights[0].new_zeros((fill, weights[0].shape[1]))]
+    return torch.cat(weights, dim=0).contiguous()
+
+
 class Linear:
     def __init__(self, weight: torch.Tensor, bias: torch.Tensor = None):
         if weight.dim() != 2 or not weight.is_contiguous():

@@ -7,7 +7,7 @@ from __future__ import annotations
 import torch
 
 from ..cache.spec import widened
-from .base import BuildContext, Residual, prefixed, sub_weights
+from .base import BuildContext, Residual, StreamSum, prefixed, sub_weights
 from .registry import BLOCKS, EMBEDDINGS, HEADS, NORMS
 from .spec import ModelPlan, TensorDecl
 
@@ -20,6 +20,7 @@ def declare_model(plan: ModelPlan) -> dict:
         d.update(prefixed(BLOCKS.get(block.kind).declare(block), plan.layer_prefix.format(i)))
     d.update(prefixed(NORMS.get(plan.final_norm.kind).declare(plan.final_norm), plan.final_norm_prefix))
     d.update(prefixed(HEADS.get(head.kind).declare(head), plan.head_prefix))
+    d.update({name: TensorDecl((rows, plan.hidden_size)) for name, rows in plan.stream_tables})
     return d
 
 
@@ -60,6 +61,10 @@ class CausalLM:
         self.final_norm = NORMS.get(plan.final_norm.kind)(plan.final_norm,
                                                           sub_weights(weights, plan.final_norm_prefix), ctx)
         self.head = HEADS.get(head.kind)(head, sub_weights(weights, plan.head_prefix), ctx, embedding=self.embedding)
+        # rows that are added to the stream between two calls, in float32 like the stream
+        self.stream_tables = {name: weights[name].to(device=ctx.device, dtype=torch.float32).contiguous()
+                              for name, _ in plan.stream_tables}
+        self.keeps_embedding = any(call.add_embedding for call in plan.order)
         self.graph_safe = all(getattr(part, "graph_safe", False) for part in [self.embedding, self.head] + self.layers)
 
     def forward(self, step, caches, watch=None) -> torch.Tensor:
@@ -67,29 +72,39 @@ class CausalLM:
         the running order with the stream brought up to date (a reader for tests and comparisons)."""
         ws = step.workspace
         x = ws.get(step.tag + "residual", (step.num_tokens, self.plan.hidden_size), torch.float32)
+        # the embedding's output is kept apart when a later call adds it again: the stream then starts as a sum with that base
+        first = ws.get(step.tag + "embedded", tuple(x.shape), torch.float32) if self.keeps_embedding else x
         if getattr(self.embedding, "keeps_state", False):
-            self.embedding(step, x, caches[len(self.plan.order)])
+            self.embedding(step, first, caches[len(self.plan.order)])
         else:
-            self.embedding(step, x)
+            self.embedding(step, first)
         residual = Residual(x)
+        if self.keeps_embedding:
+            residual.pending = StreamSum(base=first)
         order = self.plan.order
         for i, (call, cache) in enumerate(zip(order, caches)):
             layer = self.layers[call.layer]
-            if residual.deferred is not None and not getattr(layer, "takes_deferred", False):
+            residual.add_before_next(first if call.add_embedding else None,
+                                     self.stream_tables[call.add_row[0]][call.add_row[1]] if call.add_row is not None else None)
+            if (residual.deferred is not None and not getattr(layer, "takes_deferred", False)) or \
+                    (isinstance(residual.pending, StreamSum) and not getattr(layer, "takes_sum", False)):
                 residual.settle()
             if getattr(layer, "chains_norms", False):
                 # a block may leave the next block's first norm in factored form (parts/base.py, ScaledRows)
                 nxt = self.layers[order[i + 1].layer] if i + 1 < len(order) else None
+                if nxt is not None and (order[i + 1].add_embedding or order[i + 1].add_row is not None):
+                    nxt = None
                 ask = getattr(nxt, "input_norm_for_fusion", None)
                 layer(residual, step, cache, next_norm=ask(step.num_tokens) if ask else None)
             else:
                 layer(residual, step, cache)
             if watch is not None:
+                residual.settle()
                 if residual.pending is not None or residual.normed is not None:
                     raise NotImplementedError("watching a model whose blocks leave their results pending")
-                residual.settle()
                 watch(i, residual.x)
-        residual.settle()
+        if residual.deferred is not None or not getattr(self.final_norm, "takes_sum", False):
+            residual.settle()
         R = step.logit_rows.shape[0]
         if R == 0:
             return ws.get(step.tag + "logits", (0, self.plan.vocab_size), torch.float32)

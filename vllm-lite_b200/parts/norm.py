@@ -56,10 +56,15 @@ class RmsNorm:
         kernel norms every head while it rotates it)."""
         return self.weight, self.spec.eps
 
+    takes_sum = True           # `delta` may be a `StreamSum`: the kernel forms the stream's new values as it reads
+
     def __call__(self, x, delta, step, rows=None, tag="norm"):
         from ..csrc import ops
+        from .base import StreamSum
         R = x.shape[0] if rows is None else rows.shape[0]
         out = step.workspace.get(step.tag + tag, (R, self.spec.size), self.dtype)
+        if isinstance(delta, StreamSum):
+            return ops.stream_norm(x, delta, self.weight, self.spec.eps, out, rows=rows)
         return ops.add_rmsnorm(x, delta, self.weight, self.spec.eps, out, rows=rows)
 
 

@@ -13,9 +13,9 @@ from __future__ import annotations
 import torch
 
 from ..cache.spec import FixedState
-from .linear import Linear
+from .linear import Linear, stacked
 from .registry import MIXERS
-from .spec import DeltaRuleSpec, MatrixMemorySpec, StateSpaceSpec, TensorDecl, TimeMixSpec
+from .spec import DeltaRuleSpec, HeadDeltaSpec, MatrixMemorySpec, StateSpaceSpec, TensorDecl, TimeMixSpec
 
 
 def _f32(t, ctx):
@@ -179,6 +179,62 @@ class DeltaRule:
         gated = ws.get(tag + "dr.gated", (T, H * P), self.dtype)
         ops.gate_norm(o, up, H * D, "sigmoid", False, self.norm, s.eps, gated, P)
         return self.o_proj(gated, step, "dr.out")
+
+
+@MIXERS.register("head_delta")
+class HeadDelta:
+    """The delta rule with one decay per head and a silu output gate (`HeadDeltaSpec`): everything the input is multiplied by
+    is one product, [q | k | v | g | b | a]; the short convolution reads its first three blocks of columns, the scan the two
+    numbers per head, the norm the gate."""
+    graph_safe = True
+
+    @staticmethod
+    def declare(s: HeadDeltaSpec) -> dict:
+        q, k, v, conv, b, a_log, norm, a, dt_bias, g, o = s.names
+        H, G, D, P, W = s.num_heads, s.num_kv_heads, s.dim, s.vdim, s.hidden_size
+        return {q: TensorDecl((G * D, W)), k: TensorDecl((G * D, W)), v: TensorDecl((H * P, W)),
+                q + conv: TensorDecl((G * D, s.conv), init="conv"), k + conv: TensorDecl((G * D, s.conv), init="conv"),
+                v + conv: TensorDecl((H * P, s.conv), init="conv"), b: TensorDecl((H, W)),
+                a_log: TensorDecl((H,), init="unit"), norm: TensorDecl((P,), init="norm"), a: TensorDecl((H, W)),
+                dt_bias: TensorDecl((H,), init="unit"), g: TensorDecl((H * P, W)), o: TensorDecl((W, H * P))}
+
+    @staticmethod
+    def _conv_channels(s):
+        return 2 * s.num_kv_heads * s.dim + s.num_heads * s.vdim
+
+    @staticmethod
+    def cache_need(s: HeadDeltaSpec):
+        from ..csrc import ops
+        return FixedState(((s.conv - 1) * HeadDelta._conv_channels(s) + ops.scan_state_floats(s.num_heads, s.dim, s.vdim),))
+
+    def __init__(self, s: HeadDeltaSpec, weights: dict, ctx):
+        from ..csrc import ops
+        if s.num_heads % s.num_kv_heads or s.conv < 1:
+            raise ValueError(f"delta rule: {s.num_kv_heads} key heads do not divide {s.num_heads} heads, or no tap")
+        ops.scan_lanes(s.dim)
+        self.spec, self.dtype = s, ctx.dtype
+        q, k, v, conv, b, a_log, norm, a, dt_bias, g, o = s.names
+        self.in_proj = Linear(stacked([weights[n] for n in (q, k, v, g, b, a)]))
+        self.o_proj = Linear(weights[o])
+        self.conv = _f32(torch.cat([weights[q + conv], weights[k + conv], weights[v + conv]], dim=0), ctx)
+        self.a_log, self.dt_bias, self.norm = _f32(weights[a_log], ctx), _f32(weights[dt_bias], ctx), _f32(weights[norm], ctx)
+
+    def __call__(self, h, step, cache):
+        from ..csrc import ops
+        s, ws, tag = self.spec, step.workspace, step.tag
+        H, G, D, P = s.num_heads, s.num_kv_heads, s.dim, s.vdim
+        C = self._conv_channels(s)
+        T = h.shape[0]
+        proj = self.in_proj(h, step, "hd.in")
+        qkv = ws.get(tag + "hd.qkv", (T, C), torch.float32)
+        ops.short_conv(proj, 0, C, self.conv, None, cache.state, 0, step.cu_seqlens, step.state_slots, qkv,
+                       longest=step.max_query_len)
+        o = ws.get(tag + "hd.o", (T, H * P), torch.float32)
+        ops.delta_scan(qkv, proj, C + H * P + H, self.dt_bias, self.a_log, proj, C + H * P, D ** -0.5, s.unit_eps, cache.state,
+                       (s.conv - 1) * C, step.cu_seqlens, step.state_slots, o, H, G, D, P, head_decay=True)
+        gated = ws.get(tag + "hd.gated", (T, H * P), self.dtype)
+        ops.gate_norm(o, proj, C, "silu", False, self.norm, s.eps, gated, P)
+        return self.o_proj(gated, step, "hd.out")
 
 
 @MIXERS.register("time_mix")

@@ -65,6 +65,18 @@ class RotaryScaling:
 
 
 @dataclass(frozen=True)
+class YarnScaling:
+    """The same by how often a frequency turns within the `original` context (YaRN): with n = rotary_dim and
+    c(t) = n ln(original / (2 pi t)) / (2 ln theta) (the feature index whose pair turns t times), low = max(floor(c(fast)), 0),
+    high = min(ceil(c(slow)), n - 1), r_i = clamp((i - low) / max(high - low, 0.001), 0, 1): f_i becomes
+    r_i f_i / factor + (1 - r_i) f_i, and sine and cosine are multiplied by 0.1 ln(factor) + 1."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
 class RotarySpec:
     """Rotary position encoding of the first `rotary_dim` features of each head; inv_freq[i] =
     theta^(-2i / rotary_dim).  Feature i turns with feature i + rotary_dim/2 (rotate-half), or, when
@@ -74,7 +86,7 @@ class RotarySpec:
     rotary_dim: Optional[int] = None
     kind: str = "rotary"
     interleaved: bool = False
-    scaling: Optional[RotaryScaling] = None
+    scaling: Optional[object] = None        # RotaryScaling or YarnScaling
 
     @property
     def dim(self) -> int:
@@ -229,7 +241,9 @@ class LatentAttentionSpec:
     (W_uq has heads * (dim + rot_dim) rows), W_dkv has rot_dim more rows behind the latent's, which are NOT normed and
     are ONE more key part shared by all heads; `position` turns the first `position.dim` features of both parts, and the
     score is scale * (q . k + q_rot . k_rot).  The cached row is then [c | rotated key part].
-    `gate` (a tensor name): the concatenated heads times sigmoid(W_g h), W_g [heads * vdim, hidden], before W_o."""
+    `gate` (a tensor name): the concatenated heads times sigmoid(W_g h), W_g [heads * vdim, hidden], before W_o.
+    `head_gate` (a tensor name): head h's values times sigmoid(W_g h)_h, W_g [heads, hidden].
+    `q_rank` 0: no query latent, q = W_uq h (the tensor `uq` is then [heads * (dim + rot_dim), hidden]; dq and its norm do not exist)."""
     hidden_size: int
     num_heads: int
     dim: int
@@ -245,6 +259,7 @@ class LatentAttentionSpec:
     rot_dim: int = 0
     position: Optional[RotarySpec] = None
     gate: Optional[str] = None
+    head_gate: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -252,8 +267,8 @@ class GatedMlpSpec:
     """down(act(gate(h)) * up(h)) with a choice of activation ("silu", "relu", or "capped_swish": g' = min(g, limit),
     u' = clamp(u, -limit, limit), g' sigmoid(alpha g') (u' + up_shift)) and optional bias vectors on all
     three projections.  `names`: (gate, up, down) relative to the part's prefix; a bias is `<name><bias_suffix>`.
-    `gated` False: down(f(up(h))) with f a function of one argument ("relu2": the square of max(v, 0)); there is no gate
-    matrix and no bias.
+    `gated` False: down(f(up(h))) with f a function of one argument ("relu2": the square of max(v, 0); "gelu": v times the
+    normal distribution function at v); there is no gate matrix and no bias.
     Activation "poly_norm" (ungated) takes the whole row: c_0 N(z) + c_1 N(z^2) + c_2 N(z^3) + c_3, powers element by element,
     N(v) = v / sqrt(mean(v^2) + eps) over the row; its four numbers are the tensor `coef`."""
     hidden_size: int
@@ -383,6 +398,27 @@ class DeltaRuleSpec:
     unit_eps: float = 1e-6
     names: Tuple[str, ...] = ("q", "k", "v", ".conv", "b", "A_log", "norm", "a1", "a2", "dt_bias", "g1", "g2", "o")
     kind: str = "delta_rule"
+
+
+@dataclass(frozen=True)
+class HeadDeltaSpec:
+    """Gated delta rule with ONE decay per head.
+
+    q = W_q h, k = W_k h (kv_heads x dim), v = W_v h (heads x vdim), each through a causal convolution of `conv` taps
+    (no bias) and silu; head h uses q/k head floor(h / (heads / kv_heads)); q, k -> x / sqrt(sum x^2 + unit_eps), q also times
+    dim^-1/2; beta = sigmoid(W_b h), g = exp(-exp(A_log) softplus(W_a h + dt_bias)), both one number a head;
+    S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; out = W_o (rms_head(o) * norm * silu(W_g h)), norm of vdim
+    entries shared by heads.  `names`: (q, k, v, conv suffix, b, A_log, norm, a, dt_bias, g, o)."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    eps: float
+    unit_eps: float = 1e-6
+    names: Tuple[str, ...] = ("q", "k", "v", ".conv", "b", "A_log", "norm", "a", "dt_bias", "g", "o")
+    kind: str = "head_delta"
 
 
 @dataclass(frozen=True)
@@ -524,7 +560,9 @@ class BlockSpec:
     x_t <- sum_s mix_q[s, t] x_s + out_q[t] y; the single stream is the sum of the copies.  `hyper`: the two
     sub-layers' `HyperConnectionSpec`; `hyper_prefixes`: where their tensors lie.  `ffn` may be None.
     kind "sandwich": x += post1(mixer(norm1(x))); x += post2(ffn(norm2(x))): a norm before and a norm after every
-    sub-layer (`post_norms`, their tensors under `post_names`); `ffn` may be None."""
+    sub-layer (`post_norms`, their tensors under `post_names`); `ffn` may be None.
+    kind "shared_norm": h = norm1(x); x += m (s1 * mixer(h) + s2 * ffn(h)): both sub-layers read ONE norm's output; m =
+    `residual_mult`; `scales`: the names of s1 and s2 [hidden], None: ones; `ffn` may be None (and norm2 is unused)."""
     mixer: object
     ffn: object
     norm1: NormSpec
@@ -538,6 +576,7 @@ class BlockSpec:
     names: Tuple[str, str, str, str] = ("input_layernorm.", "self_attn.", "post_attention_layernorm.", "mlp.")
     post_norms: Optional[Tuple[NormSpec, NormSpec]] = None     # sandwich: the norms on the two sub-layers' outputs
     post_names: Tuple[str, str] = ("post_mixer_norm.", "post_mlp_norm.")
+    scales: Optional[Tuple[str, str]] = None                   # shared_norm: per-channel factors on the two sub-layers' results
 
 
 @dataclass(frozen=True)
@@ -547,9 +586,14 @@ class LayerCall:
     `layer` indexes `ModelPlan.layers` (the weights).  `cache_of`, when set, is
     the index of an EARLIER entry of the order whose cache this call reads
     instead of writing one of its own.
+    What is added to the stream right before this call: `add_embedding`, the embedding's output (the stream as it was before the
+    first call); then `add_row` = (table, row), a row of a table of the model (`ModelPlan.stream_tables`).  A layer named by several
+    calls runs each time from a cache or state of the call's own.
     """
     layer: int
     cache_of: Optional[int] = None
+    add_embedding: bool = False
+    add_row: Optional[Tuple[str, int]] = None
 
 
 @dataclass(frozen=True)
@@ -575,6 +619,8 @@ class ModelPlan:
     head: Optional[object] = None
     # names of stored tensors that the model does not bind and that the loader passes over
     unused_tensors: Tuple[str, ...] = ()
+    # (tensor name, rows): tables [rows, hidden] whose rows `LayerCall.add_row` adds to the stream
+    stream_tables: Tuple[Tuple[str, int], ...] = ()
 
     @property
     def embedding_spec(self):
@@ -594,4 +640,8 @@ class ModelPlan:
                     raise ValueError(f"order[{i}].cache_of={call.cache_of} must name an earlier entry")
                 if self.order[call.cache_of].cache_of is not None:
                     raise ValueError(f"order[{i}].cache_of={call.cache_of} names an entry that owns no cache")
+            if call.add_row is not None:
+                rows = dict(self.stream_tables).get(call.add_row[0])
+                if rows is None or not 0 <= call.add_row[1] < rows:
+                    raise ValueError(f"order[{i}].add_row={call.add_row} names no row of the plan's stream tables")
         return self
