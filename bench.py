@@ -431,7 +431,8 @@ TIMED_OPS = ("paged_attention", "flash_prefill", "flash_prefill_tc5", "flash_dec
              "moe_gather", "moe_combine", "gated_act", "silu_mul", "scale_softcap", "embed", "cast", "add_bias",
              "hc_step", "dyt_rows", "short_conv", "ssd_scan", "mlstm_scan", "delta_scan", "gate_norm", "scaled_sum",
              "token_shift", "rows_norm_rope_write", "conv_rows_norm_rope_write", "rmsnorm_add", "unary_act",
-             "head_norm_write", "rope_heads", "sigmoid_gate", "token_shift_multi", "decay_scan", "decay_from_raw", "head_work", "combine_maps", "linear_scan", "poly_norm", "embed_pair")
+             "head_norm_write", "rope_heads", "sigmoid_gate", "token_shift_multi", "decay_scan", "decay_from_raw", "head_work", "combine_maps", "linear_scan", "poly_norm", "embed_pair",
+             "stream_norm", "delta_chunks", "delta_step")
 
 
 def kikepel_config(size, layers):
@@ -1149,6 +1150,169 @@ def pafelorn_roofline(size, layers, context, results, pk):
     return roof
 
 
+# ---------------------------------------------------------------------------------------------------
+# --vekusun: the Vekusun decoder (mixer and feed-forward side by side on one norm, a stretch of layers run twice; latent attention
+# with a query latent and a sink, or with a rotated part and a gate per head; the delta rule with one decay per head; erf gelu or
+# silu experts) beside the Qwen3 decoder at equal width, number of layer runs, heads and active feed-forward width
+# ---------------------------------------------------------------------------------------------------
+# name: (width, heads, q/k heads of the delta rule, head, rotated part, query latent, latent without positions, latent beside the
+#        rotated part, taps, dense ff, expert ff, experts, top, vocab)
+VEKUSUN_SIZES = {"2k": (2048, 16, 8, 128, 64, 768, 256, 192, 4, 8192, 1024, 32, 4, 65536),
+                 "4k": (4096, 32, 16, 128, 64, 1536, 256, 192, 4, 12288, 1408, 64, 6, 65536),
+                 "2k-h64": (2048, 32, 16, 64, 32, 512, 128, 96, 4, 8192, 1024, 32, 4, 65536)}
+VEKUSUN_LOOP = (1, 3, 2)
+
+
+def vekusun_config(size, layers):
+    W, H, G, D, rot, qr, kr, kr2, taps, ff, eff, E, top, vocab = VEKUSUN_SIZES[size]
+    delta = dict(heads=H, kv_heads=G, dim=D, vdim=D, conv=taps)
+    one = dict(heads=H, dim=D, vdim=D, q_rank=qr, kv_rank=kr, scale=D ** -0.5)
+    two = dict(heads=H, dim=D, rot_dim=rot, vdim=D, kv_rank=kr2, scale=(D + rot) ** -0.5,
+               rot=dict(dims=rot, base=500000.0, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0)))
+    dense = dict(kind="dense", ff=ff)
+    moe = dict(kind="moe", expert=dict(ff=eff), router=dict(experts=E, top=top))
+    kinds = [("delta", delta, dense), ("latent_attention", one, moe), ("latent_attention_2", two, dense), ("delta", delta, moe)]
+    start, stop, times = VEKUSUN_LOOP
+    return dict(architecture="Vekusun", vocab=vocab, width=W, norm=dict(eps=1e-6), logit_softcap=30.0, residual_mult=0.5,
+                loop=dict(start=start, stop=stop, times=times), max_position_embeddings=16384,
+                layers=[dict(type=kinds[i % 4][0], mixer=kinds[i % 4][1], mlp=kinds[i % 4][2]) for i in range(layers)])
+
+
+def vekusun_runs(layers):
+    """The kinds (0..3 as in `vekusun_config`) of the layers in running order."""
+    start, stop, times = VEKUSUN_LOOP
+    return [i % 4 for i in list(range(start)) + list(range(start, stop)) * times + list(range(stop, layers))]
+
+
+def vekusun_bench(args):
+    import torch
+    from vllm_lite_b200.engine import LLMEngine, StepEntry, random_model
+    size, layers = args.vekusun, args.layers or 8
+    W, H, G, D, rot, qr, kr, kr2, taps, ff, eff, E, top, vocab = VEKUSUN_SIZES[size]
+    context, pk, runs = args.context, peaks(), len(vekusun_runs(args.layers or 8))
+    warmup = max(args.warmup, 3)
+    qwen = dict(QWEN3_8B, num_hidden_layers=runs, hidden_size=W, num_attention_heads=H, num_key_value_heads=max(1, H // 4),
+                head_dim=D, intermediate_size=top * eff, vocab_size=vocab, max_position_embeddings=16384)
+    apart = lambda k: "+sink" if k.get("sinks") is not None else ""
+    results = {}
+    for name, cfg in (("vekusun", vekusun_config(size, layers)), ("qwen3", qwen)):
+        _, plan, weights = random_model(cfg, seed=0, dtype="bfloat16", device="cuda:0")
+        for key in weights:                               # corrections smaller than the scores: the tokens spread over the experts
+            if key.endswith(".correction"):
+                weights[key] = weights[key] * 0.01
+        slack = 256
+        pages = 64 * (-(-(context + slack) // args.block_size) + 1) + PREFILL_TOKENS // args.block_size + 64
+        engine = LLMEngine(plan=plan, weights=weights, dtype="bfloat16", kv_blocks=pages, block_size=args.block_size,
+                           max_batch_size=64, max_num_batched_tokens=PREFILL_TOKENS, prefill_chunk_size=PREFILL_TOKENS,
+                           max_model_len=context + slack)
+        del weights
+        runner, sampler = engine.runner, engine.sampler
+        for t in runner.storage.paged:
+            t.normal_()
+        res = {}
+        clocks = ClockSampler().start()
+        w0 = time.time()
+        pms = prefill_run(runner, vocab)
+        res["prefill"] = {"tokens": PREFILL_TOKENS, "ms": round(pms, 3), "tokens_per_s": round(PREFILL_TOKENS / pms * 1e3, 1)}
+        for b in (8, 64):
+            ms, launches, _ = decode_run(runner, sampler, b, context, warmup, args.steps, "random", vocab, f"d{b}.")
+            res[f"decode_b{b}"] = {"ms_per_step": round(ms, 4), "tokens_per_s": round(b * 1e3 / ms, 1), "launches": round(launches)}
+        clocks.stop()
+        res["clocks"] = clocks.summary(w0, time.time())
+        gen = torch.Generator().manual_seed(5)
+        prompt = torch.randint(0, vocab, (PREFILL_TOKENS,), generator=gen).tolist()
+        res["kernels_prefill"] = timed_step(runner, [StepEntry("kp", prompt, [PREFILL_TOKENS - 1])], apart)
+        runner.release("kp")
+        ids = [f"kd{i}" for i in range(64)]
+        for rid in ids:
+            runner.cache.admit(rid)
+            runner.cache.append(rid, context - 1)
+        runner.storage.zero_slots(runner.cache.take_fresh_slots())
+        res["kernels_decode_b64"] = timed_step(runner, [StepEntry(rid, [i], [0]) for i, rid in enumerate(ids)], apart)
+        for rid in ids:
+            runner.release(rid)
+        runner.check_device_errors()
+        res["weights_GB"] = round(sum(p.numel() * p.element_size() for p in _tensors_of(runner.model)) / 1e9, 2)
+        results[name] = res
+        del engine, runner, sampler
+        torch.cuda.empty_cache()
+    print(json.dumps({"vekusun_bench": size, "layers": layers, "layer_runs": runs, "context": context, "steps": args.steps,
+                      "warmup": warmup, "dtype": "bf16", "data": "synthetic (random weights, uniform token ids)",
+                      "config": {"vekusun": dict(zip(("width", "heads", "delta_kv_heads", "head", "rot_dim", "q_rank", "kv_rank", "kv_rank_rotated",
+                                                      "taps", "dense_ff", "expert_ff", "experts", "top", "vocab"), VEKUSUN_SIZES[size])),
+                                 "qwen3": {k_: qwen[k_] for k_ in ("num_hidden_layers", "hidden_size", "num_attention_heads",
+                                                                    "num_key_value_heads", "head_dim", "intermediate_size", "vocab_size")}},
+                      "results": results, "roofline": vekusun_roofline(size, layers, context, results, pk)}))
+    return 0
+
+
+def vekusun_roofline(size, layers, context, results, pk):
+    """The new kernels against their rooflines, beside the like kernels of the closest model: algorithmic bytes or flops over
+    the launches' time between CUDA events."""
+    W, H, G, D, rot, qr, kr, kr2, taps, ff, eff, E, top, vocab = VEKUSUN_SIZES[size]
+    T, B = PREFILL_TOKENS, 64
+    vk, q = results["vekusun"], results["qwen3"]
+    us = lambda res, step, names: sum(res[step].get(n, [0, 0.0])[1] for n in names)
+    count = lambda res, step, name: res[step].get(name, [0, 0.0])[0]
+    tf = lambda flops, micro: round(flops / (micro * 1e-6) / 1e12, 1) if micro else None
+    gb = lambda nbytes, micro: round(nbytes / (micro * 1e-6) / 1e9, 1) if micro else None
+    each = lambda micro, n: round(micro / n, 1) if n else None
+    att = ("paged_attention", "flash_prefill", "flash_prefill_tc5", "flash_decode")
+    kinds = vekusun_runs(layers)
+    n = [kinds.count(k) for k in range(4)]
+    n_delta, n_moe, n_dense = n[0] + n[3], n[1] + n[3], n[0] + n[2]
+    row1, row2 = kr, kr2 + rot                                    # cached rows
+    causal = T * (T + 1) // 2
+    roof = {"peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"], "source": pk["source"]}}
+    for step, fig in (("kernels_prefill", "attention_prefill_tflops"), ("kernels_decode_b64", "attention_decode_gbs")):
+        r = {}
+        for label, suffix, k, row in (("latent, sink", "+sink", n[1], row1), ("latent, rotated", "", n[2], row2)):
+            t = us(vk, step, tuple(a + suffix for a in att))
+            r[label] = tf(k * causal * H * 4.0 * row, t) if step == "kernels_prefill" else gb(k * B * context * 2.0 * row, t)
+            if step != "kernels_prefill":
+                r[label + ", tflops"] = tf(k * B * context * H * 4.0 * row, t)
+            r[label + ", us a layer"] = each(t, k)
+        t = us(q, step, att)
+        kv = max(1, H // 4)
+        r["qwen3"] = tf(len(kinds) * causal * H * 4.0 * D, t) if step == "kernels_prefill" else gb(len(kinds) * B * context * 4.0 * kv * D, t)
+        r["qwen3, us a layer"] = each(t, len(kinds))
+        roof[fig] = r
+    C = 2 * G * D + H * D
+    for step, rows, reqs in (("kernels_prefill", T, 1), ("kernels_decode_b64", B, B)):
+        r = {}
+        r["delta_rule_us_a_layer"] = each(us(vk, step, ("delta_scan", "delta_chunks", "delta_step")), n_delta)
+        state = reqs * H * D * D * 8.0
+        t = us(vk, step, ("delta_scan", "delta_chunks", "delta_step"))
+        r["delta_rule_gbs"] = gb(n_delta * (rows * (C + H * D) * 4.0 + state), t)
+        r["delta_rule_tflops (8 multiply-adds a state element and token)"] = tf(n_delta * rows * H * 8.0 * D * D, t)
+        r["short_conv_gbs"] = gb(n_delta * rows * C * 6.0, us(vk, step, ("short_conv",)))
+        r["gate_norm_gbs"] = gb(n_delta * rows * H * D * 8.0, us(vk, step, ("gate_norm",)))
+        r["stream_norm_gbs"] = gb(len(kinds) * rows * W * 14.0, us(vk, step, ("stream_norm",)))
+        r["qwen3_add_rmsnorm_gbs"] = gb(count(q, step, "add_rmsnorm") * rows * W * 12.0, us(q, step, ("add_rmsnorm",)))
+        r["latent_norm_write_gbs"] = gb(rows * 4.0 * (n[1] * (qr + kr) + n[2] * (H * rot + kr2 + rot)), us(vk, step, ("latent_norm_write",)))
+        r["qwen3_qk_norm_rope_write_gbs"] = gb(count(q, step, "qk_norm_rope_write") * rows * (H + 2 * max(1, H // 4)) * D * 4.0,
+                                               us(q, step, ("qk_norm_rope_write",)))
+        r["gelu_gbs"] = gb(n_dense * rows * ff * 4.0, us(vk, step, ("unary_act",)))
+        t = us(vk, step, ("gemm_heads",))
+        flops = rows * H * 2.0 * (n[1] * 2 * D * row1 + n[2] * ((D + rot) * row2 + D * row2))
+        nbytes = n[1] * 2 * (H * D * row1 + rows * H * (D + row1)) * 2.0 + n[2] * 2.0 * (H * (2 * D + rot) * row2 + rows * H * (2 * D + rot + 2 * row2))
+        r["head_products"] = {"tflops": tf(flops, t), "gbs": gb(nbytes, t), "us_a_layer": each(t, n[1] + n[2])}
+        r["us_a_step"] = {k_: vk[step][k_][1] for k_ in vk[step]}
+        r["qwen3_us_a_step"] = {k_: q[step][k_][1] for k_ in q[step]}
+        roof[step] = r
+    grouped = ("gemm_grouped", "gemm_grouped_fused", "gemm_grouped_tc5")
+    q_layer = (H + 2 * max(1, H // 4)) * D * W + W * H * D + 3 * W * top * eff
+    roof["expert_products_prefill_tflops"] = {
+        "vekusun": tf(n_moe * 2.0 * T * top * 3 * W * eff, us(vk, "kernels_prefill", grouped)),
+        "qwen3 (all dense products of the layers)": tf(len(kinds) * 2.0 * T * q_layer, us(q, "kernels_prefill", ("gemm_bf16_tc5", "gemm_bf16_tc5_pair", "library_mm")))}
+    v_layers = n_delta * (C + 2 * H * D) * W + n[1] * ((qr + kr) * W + H * D * qr + H * D * W) + n[2] * ((H * (D + rot) + row2) * W + H * D * W) + n_dense * 2 * W * ff
+    roof["dense_products_prefill_tflops"] = {"vekusun": tf(2.0 * T * v_layers, us(vk, "kernels_prefill", ("gemm_bf16_tc5", "gemm_bf16_tc5_pair", "library_mm")))}
+    roof["expert_products_decode_gbs"] = {
+        "vekusun (experts that 64 tokens can reach)": gb(n_moe * min(E, B * top) * 3.0 * W * eff * 2, us(vk, "kernels_decode_b64", grouped)),
+        "qwen3 (all products)": gb(q["weights_GB"] * 1e9 - 2.0 * vocab * W * 2, us(q, "kernels_decode_b64", ("library_mm", "gemm_bf16_small_m")))}
+    return roof
+
+
 def _tensors_of(model):
     """Every device tensor that the parts of a model hold (weights as they are resident)."""
     import torch
@@ -1204,6 +1368,9 @@ def main(argv=None):
     ap.add_argument("--pafelorn", default=None, choices=sorted(PAFELORN_SIZES), metavar="SIZE",
                     help="instead of the default workload: the Pafelorn decoder at layer sizes " + ", ".join(sorted(PAFELORN_SIZES))
                          + " beside the Qwen3 decoder at equal width, depth, heads and active feed-forward width")
+    ap.add_argument("--vekusun", default=None, choices=sorted(VEKUSUN_SIZES), metavar="SIZE",
+                    help="instead of the default workload: the Vekusun decoder at layer sizes " + ", ".join(sorted(VEKUSUN_SIZES))
+                         + " beside the Qwen3 decoder at equal width, number of layer runs, heads and active feed-forward width")
     ap.add_argument("--kikepel", default=None, choices=sorted(KIKEPEL_SIZES), metavar="SIZE",
                     help="instead of the default workload: the Kikepel decoder at layer sizes " + ", ".join(sorted(KIKEPEL_SIZES))
                          + " beside the Qwen3 decoder at equal width, depth and heads: prefill of 2,048 tokens, decode at batch 8 "
@@ -1228,6 +1395,8 @@ def main(argv=None):
         return puturax_bench(args)
     if args.pafelorn:
         return pafelorn_bench(args)
+    if args.vekusun:
+        return vekusun_bench(args)
     import torch
     from vllm_lite_b200.csrc import ops
     from vllm_lite_b200.engine import LLMEngine, random_model

@@ -83,7 +83,9 @@ def _mixer_width(mixer) -> int:
         # convolved float32 copy, the scan's float32 result, the gated rows
         hp = mixer.num_heads * mixer.vdim
         conv = 2 * mixer.num_kv_heads * mixer.dim + hp
-        return (conv + hp + 2 * mixer.num_heads + 7) + 2 * conv + 2 * hp + hp
+        # ... and, in chunks of 64 tokens, per head two matrices of 64 numbers a row of the state, one of 64 x 64, the chunk's state
+        chunks = 2 * mixer.num_heads * (mixer.dim + mixer.vdim + 64 + 3 + mixer.dim * mixer.vdim // 64)
+        return (conv + hp + 2 * mixer.num_heads + 7) + 2 * conv + 2 * hp + hp + chunks
     if hasattr(mixer, "decay_rank"):                                    # delta rule
         hp, hd = mixer.num_heads * mixer.vdim, mixer.num_heads * mixer.dim
         conv = 2 * mixer.num_kv_heads * mixer.dim + hp

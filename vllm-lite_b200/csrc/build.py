@@ -24,7 +24,7 @@ CSRC = Path(__file__).resolve().parent
 ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 NVCC_FLAGS = ARCH_FLAGS + ["-O3", "-lineinfo", "-std=c++17", "--shared", "-Xcompiler", "-fPIC"]
 SOURCES = ("embed_norm", "rope_cache", "attention", "activation", "gemm_f32", "gemm_bf16", "gemm_tc5", "gemm_tc5_pair", "sampling", "hyper", "recurrent",
-           "memprobe", "latent", "gemm_batched", "moe", "gemm_tc5_grouped", "head_work", "linear_scan")
+           "memprobe", "latent", "gemm_batched", "moe", "gemm_tc5_grouped", "head_work", "linear_scan", "delta")
 # sources compiled once per value of a constant; the values here are what build_all() prepares,
 # any other allowed value is compiled when a model first needs it
 VARIANTS = {"flash_attn": [{"FA_HD": 128}, {"FA_HD": 64}, {"FA_HD": 32}, {"FA_HD": 16}],

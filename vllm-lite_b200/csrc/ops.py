@@ -153,6 +153,12 @@ _SIGNATURES = {
     ("recurrent", "vl_delta_scan"): [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
                                      c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
                                      c_int, c_int, c_void_p],
+    ("delta", "vl_delta_step"): [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
+                                 c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
+                                 c_int, c_int, c_void_p],
+    ("delta", "vl_delta_chunks"): [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
+                                   c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
+                                   c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     ("recurrent", "vl_gate_norm"): [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_float, c_void_p,
                                     c_int, c_int, c_int, c_void_p],
 }
@@ -1624,6 +1630,67 @@ def delta_scan(qkv, decay, decay_col, dt_bias, A_log, proj, beta_col, q_scale, u
                                              sp, stride, _ptr(cu), _ptr(slots), B, _ptr(o), H, G, D, P, int(bool(head_decay)), _stream()),
            "vl_delta_scan")
     return o
+
+
+# the delta rule with one decay per head (csrc/delta.cu)
+DELTA_CHUNK, DELTA_MIN_CHUNK, DELTA_MAX = 64, 16, 128
+
+
+def head_delta_ok(D, P) -> bool:
+    """Whether csrc/delta.cu takes a state of D rows and P columns per head (rows on 16-byte boundaries, at most 128 x 128); the
+    state then lies row by row (H * D * P floats).  Other sizes run `delta_scan`, which keeps its own layout."""
+    return 0 < D <= DELTA_MAX and 0 < P <= DELTA_MAX and D % 4 == 0 and P % 4 == 0
+
+
+def _head_delta_args(qkv, proj, a_col, b_col, gate_col, dt_bias, A_log, norm, state, state_off, cu, slots, out, H, G, D, P):
+    _need(qkv, torch.float32, "qkv", 2); _need(proj, None, "proj", 2); _need(out, proj.dtype, "out", 2)
+    for t, n, size in ((dt_bias, "dt_bias", H), (A_log, "A_log", H), (norm, "norm", P)):
+        _need(t, torch.float32, n, 1)
+        if t.shape[0] != size:
+            raise KernelError(f"head delta: {n} has {size} entries")
+    T, C = qkv.shape
+    if proj.shape[0] != T or out.shape != (T, H * P) or C != 2 * G * D + H * P or not head_delta_ok(D, P) or H % G:
+        raise KernelError("head delta: shapes disagree")
+    if min(a_col, b_col, gate_col) < 0 or max(a_col + H, b_col + H, gate_col + H * P) > proj.shape[1]:
+        raise KernelError("head delta: a column range leaves the rows")
+    B = _seg_args(cu, slots)
+    sp, stride = _state_args(state, state_off, H * D * P)
+    return B, sp, stride
+
+
+def delta_step(qkv, proj, a_col, b_col, gate_col, dt_bias, A_log, q_scale, unit_eps, norm, eps, state, state_off, cu, slots, out, H, G, D, P):
+    """out [T, H P] = rms_head(o) * norm * silu(gate) of the delta rule with one decay per head, for the requests of the step that
+    bring fewer than DELTA_MIN_CHUNK tokens (the others' rows and states are left alone).  qkv: what the convolution leaves;
+    raw decays, raw betas and the gate are columns of `proj`."""
+    B, sp, stride = _head_delta_args(qkv, proj, a_col, b_col, gate_col, dt_bias, A_log, norm, state, state_off, cu, slots, out, H, G, D, P)
+    _check(_fn("delta", "vl_delta_step")(
+        _ptr(qkv), qkv.shape[1], _ptr(proj), dtype_code(proj.dtype), proj.shape[1], int(a_col), int(b_col), int(gate_col), _ptr(dt_bias),
+        _ptr(A_log), float(q_scale), float(unit_eps), _ptr(norm), float(eps), sp, stride, _ptr(cu), _ptr(slots), B, _ptr(out), H, G, D, P,
+        DELTA_MIN_CHUNK - 1, _stream()), "vl_delta_step")
+    return out
+
+
+def delta_chunk_floats(chunks, H, D, P) -> int:
+    """Floats of the scratch that `delta_chunks` needs for so many chunks (csrc/delta.cu)."""
+    c = DELTA_CHUNK
+    return chunks * H * (D * c + P * c + c * c + 3 * c + D * P)
+
+
+def delta_chunks(qkv, proj, a_col, b_col, gate_col, dt_bias, A_log, q_scale, unit_eps, norm, eps, state, state_off, cu, slots, chunks, scratch,
+                 u, out, H, G, D, P):
+    """The same for the requests that bring DELTA_MIN_CHUNK tokens or more, in chunks of 64 tokens.  `chunks`: a bound on the
+    chunks of the step; scratch float32 of `delta_chunk_floats`; u float32 [T, H P]."""
+    global launch_count
+    B, sp, stride = _head_delta_args(qkv, proj, a_col, b_col, gate_col, dt_bias, A_log, norm, state, state_off, cu, slots, out, H, G, D, P)
+    _need(scratch, torch.float32, "scratch"); _need(u, torch.float32, "u", 2)
+    if scratch.numel() < delta_chunk_floats(chunks, H, D, P) or u.shape != out.shape:
+        raise KernelError("delta_chunks: the scratch is too small")
+    _check(_fn("delta", "vl_delta_chunks")(
+        _ptr(qkv), qkv.shape[1], _ptr(proj), dtype_code(proj.dtype), proj.shape[1], int(a_col), int(b_col), int(gate_col), _ptr(dt_bias),
+        _ptr(A_log), float(q_scale), float(unit_eps), _ptr(norm), float(eps), sp, stride, _ptr(cu), _ptr(slots), B, int(chunks), _ptr(scratch),
+        _ptr(u), _ptr(out), H, G, D, P, 2 * sm_pairs(), _stream()), "vl_delta_chunks")
+    launch_count += 2             # three launches
+    return out
 
 
 def token_shift_multi(h, mu, state, state_off, cu, slots, req_index, positions, out):

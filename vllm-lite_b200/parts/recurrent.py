@@ -184,9 +184,18 @@ class DeltaRule:
 @MIXERS.register("head_delta")
 class HeadDelta:
     """The delta rule with one decay per head and a silu output gate (`HeadDeltaSpec`): everything the input is multiplied by
-    is one product, [q | k | v | g | b | a]; the short convolution reads its first three blocks of columns, the scan the two
-    numbers per head, the norm the gate."""
+    is one product, [q | k | v | g | b | a]; the short convolution reads its first three blocks of columns, the recurrence the two
+    numbers per head and, in its own epilogue, the norm's gate (csrc/delta.cu: single tokens walk, longer portions run in
+    chunks whose insides are matrix products).  Sizes that csrc/delta.cu does not take run the scan of csrc/recurrent.cu and
+    the gated norm behind it; which of the two depends on the sizes alone, and so does the layout of the state."""
     graph_safe = True
+
+    @staticmethod
+    def _state_floats(s) -> int:
+        from ..csrc import ops
+        if ops.head_delta_ok(s.dim, s.vdim):
+            return s.num_heads * s.dim * s.vdim
+        return ops.scan_state_floats(s.num_heads, s.dim, s.vdim)
 
     @staticmethod
     def declare(s: HeadDeltaSpec) -> dict:
@@ -204,8 +213,7 @@ class HeadDelta:
 
     @staticmethod
     def cache_need(s: HeadDeltaSpec):
-        from ..csrc import ops
-        return FixedState(((s.conv - 1) * HeadDelta._conv_channels(s) + ops.scan_state_floats(s.num_heads, s.dim, s.vdim),))
+        return FixedState(((s.conv - 1) * HeadDelta._conv_channels(s) + HeadDelta._state_floats(s),))
 
     def __init__(self, s: HeadDeltaSpec, weights: dict, ctx):
         from ..csrc import ops
@@ -229,10 +237,22 @@ class HeadDelta:
         qkv = ws.get(tag + "hd.qkv", (T, C), torch.float32)
         ops.short_conv(proj, 0, C, self.conv, None, cache.state, 0, step.cu_seqlens, step.state_slots, qkv,
                        longest=step.max_query_len)
-        o = ws.get(tag + "hd.o", (T, H * P), torch.float32)
-        ops.delta_scan(qkv, proj, C + H * P + H, self.dt_bias, self.a_log, proj, C + H * P, D ** -0.5, s.unit_eps, cache.state,
-                       (s.conv - 1) * C, step.cu_seqlens, step.state_slots, o, H, G, D, P, head_decay=True)
         gated = ws.get(tag + "hd.gated", (T, H * P), self.dtype)
+        b_col, a_col = C + H * P, C + H * P + H
+        if ops.head_delta_ok(D, P):
+            args = (qkv, proj, a_col, b_col, C, self.dt_bias, self.a_log, D ** -0.5, s.unit_eps, self.norm, s.eps, cache.state,
+                    (s.conv - 1) * C, step.cu_seqlens, step.state_slots)
+            B = step.cu_seqlens.shape[0] - 1
+            if step.max_query_len >= ops.DELTA_MIN_CHUNK:
+                chunks = T // ops.DELTA_CHUNK + B
+                scratch = ws.get(tag + "hd.chunks", (ops.delta_chunk_floats(chunks, H, D, P),), torch.float32)
+                ops.delta_chunks(*args, chunks, scratch, ws.get(tag + "hd.u", (T, H * P), torch.float32), gated, H, G, D, P)
+            if step.max_query_len < ops.DELTA_MIN_CHUNK or B > 1:
+                ops.delta_step(*args, gated, H, G, D, P)
+            return self.o_proj(gated, step, "hd.out")
+        o = ws.get(tag + "hd.o", (T, H * P), torch.float32)
+        ops.delta_scan(qkv, proj, a_col, self.dt_bias, self.a_log, proj, b_col, D ** -0.5, s.unit_eps, cache.state,
+                       (s.conv - 1) * C, step.cu_seqlens, step.state_slots, o, H, G, D, P, head_decay=True)
         ops.gate_norm(o, proj, C, "silu", False, self.norm, s.eps, gated, P)
         return self.o_proj(gated, step, "hd.out")
 
