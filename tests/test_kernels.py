@@ -419,7 +419,8 @@ def test_paged_attention_ragged(kernel, dtype, nq, nkv, hd, page, window):
 
 @pytest.mark.parametrize("nq,nkv,hd,page,window", [(2, 1, 64, 16, 0), (6, 2, 64, 8, 37), (5, 5, 64, 64, 0),
                                                    (4, 2, 128, 16, 0), (8, 1, 128, 32, 150), (3, 3, 128, 128, 0),
-                                                   (32, 8, 128, 16, 0)])
+                                                   (32, 8, 128, 16, 0), (3, 1, 192, 16, 0), (4, 2, 192, 64, 90),
+                                                   (6, 1, 256, 8, 0), (2, 2, 256, 128, 150), (16, 1, 256, 64, 0)])
 @pytest.mark.parametrize("order", ["shuffled", "in a row", "runs"])
 def test_flash_tc5_prefill(nq, nkv, hd, page, window, order):
     """The tcgen05 kernel on a ragged batch: a whole prompt of several tiles, a continuation that

@@ -48,95 +48,114 @@ static bool delta_sizes_ok(int H, int G, int D, int P, int C) {
 
 // ------------------------------------------------------------------------------------------ few tokens
 #define STEP_ROWS 8                   // rows of the state a thread holds (four columns each)
+// How the threads lie over a state of D rows and U = P / 4 units of four columns: a warp covers LU neighbouring units of 32 / LU rows,
+// UG warps side by side cover the units, WR of them one under the other the rows (STEP_ROWS rows a thread).
+struct StepShape { int LU, UG, WR; };
+static inline StepShape step_shape(int D, int U) {
+    int LU = 1;
+    while (LU < U && LU < 8) LU <<= 1;
+    const int rows = 32 / LU * STEP_ROWS;
+    return StepShape{LU, (U + LU - 1) / LU, (D + rows - 1) / rows};
+}
 template <typename TP>
 __global__ void __launch_bounds__(512, 2)
 delta_step_kernel(const float* __restrict__ qkv, int C, const TP* __restrict__ proj, int ld, int a_col, int b_col, int gate_col,
                   const float* __restrict__ dt_bias, const float* __restrict__ A_log, float q_scale, float unit_eps,
                   const float* __restrict__ norm, float eps, float* __restrict__ state, long long state_stride,
                   const int* __restrict__ cu, const int* __restrict__ slots, TP* __restrict__ out, int H, int G, int D, int P,
-                  int longest) {
-    __shared__ __align__(16) float sq[DELTA_MAX], sk[DELTA_MAX], su[DELTA_MAX];
+                  int longest, int LU, int UG, int WR) {
+    __shared__ __align__(16) float sq[DELTA_MAX], sk[DELTA_MAX], su[DELTA_MAX], part[2][4][DELTA_MAX];
     __shared__ float s_g, s_beta, s_qk;
-    extern __shared__ __align__(16) float part[];                  // [2][row groups][P]
     pdl_launch_dependents();
     pdl_wait();
     const int h = blockIdx.x, b = blockIdx.y;
     const int s0 = cu[b], n = cu[b + 1] - s0;
     if (n <= 0 || n > longest) return;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int U = P >> 2, RG = blockDim.x / U;
-    const int unit = tid % U, rg = tid / U;
-    const bool live = rg < RG;
+    const int U = P >> 2, RG = WR * (32 / LU);
+    const int unit = (warp % UG) * LU + lane % LU, wr = warp / UG, rg = wr * (32 / LU) + lane / LU;
+    const bool live = unit < U;
     float* S = state + (long long)slots[b] * state_stride + (size_t)h * D * P + 4 * unit;
     float4 s[STEP_ROWS];
 #pragma unroll
     for (int i = 0; i < STEP_ROWS; ++i) {
         const int r = rg + RG * i;
-        s[i] = (live && r < D) ? ld4(S + (size_t)r * P) : make_float4(0.f, 0.f, 0.f, 0.f);
+        s[i] = (live && r < D) ? ld4(S + r * P) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     const int g = h / (H / G);
     for (int t = 0; t < n; ++t) {
         const float* row = qkv + (size_t)(s0 + t) * C;
         const TP* prow = proj + (size_t)(s0 + t) * ld;
-        if (warp == 0) {                                          // unit vectors, their product, the two numbers of the head
-            float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f), z = v;
+        if (warp == 0) {                                          // unit vectors, their product; what the epilogue will need
+            float4 q = v, k = v;
             if (4 * lane < D) { q = ld4(row + (size_t)g * D + 4 * lane); k = ld4(row + (size_t)(G + g) * D + 4 * lane); }
+            if (lane < U) {
+                v = ld4(row + (size_t)2 * G * D + (size_t)h * P + 4 * lane);
+                z = Quad<TP>::load(prow + gate_col + (size_t)h * P + 4 * lane);
+            }
             const float qn = q_scale / sqrtf(warp_sum(dot4(q, q)) + unit_eps), kn = 1.f / sqrtf(warp_sum(dot4(k, k)) + unit_eps);
             q.x *= qn; q.y *= qn; q.z *= qn; q.w *= qn;
             k.x *= kn; k.y *= kn; k.z *= kn; k.w *= kn;
-            const float qk = warp_sum(dot4(q, k));
             if (4 * lane < D) { st4(sq + 4 * lane, q); st4(sk + 4 * lane, k); }
-            if (lane == 0) {
-                s_qk = qk;
-                s_g = expf(-expf(A_log[h]) * dl_softplus(to_f32(prow[a_col + h]) + dt_bias[h]));
-                s_beta = dl_sigmoid(to_f32(prow[b_col + h]));
-            }
+            const float qk = warp_sum(dot4(q, k));
+            if (lane == 0) s_qk = qk;
+        }
+        if (tid == blockDim.x - 1) {                              // the two numbers of the head (the last warp, or the only one)
+            s_g = expf(-expf(A_log[h]) * dl_softplus(to_f32(prow[a_col + h]) + dt_bias[h]));
+            s_beta = dl_sigmoid(to_f32(prow[b_col + h]));
         }
         __syncthreads();
         float4 w = make_float4(0.f, 0.f, 0.f, 0.f), r4 = w;
 #pragma unroll
         for (int i = 0; i < STEP_ROWS; ++i) {
             const int r = rg + RG * i;
-            if (live && r < D) {
+            if (r < D) {
                 const float kr = sk[r], qr = sq[r];
                 w.x += s[i].x * kr; w.y += s[i].y * kr; w.z += s[i].z * kr; w.w += s[i].w * kr;
                 r4.x += s[i].x * qr; r4.y += s[i].y * qr; r4.z += s[i].z * qr; r4.w += s[i].w * qr;
             }
         }
-        if (live) {
-            st4(part + (size_t)rg * P + 4 * unit, w);
-            st4(part + (size_t)(RG + rg) * P + 4 * unit, r4);
+        for (int o = LU; o < 32; o <<= 1) {                       // the warp's rows of a unit
+            w.x += __shfl_xor_sync(0xffffffffu, w.x, o); w.y += __shfl_xor_sync(0xffffffffu, w.y, o);
+            w.z += __shfl_xor_sync(0xffffffffu, w.z, o); w.w += __shfl_xor_sync(0xffffffffu, w.w, o);
+            r4.x += __shfl_xor_sync(0xffffffffu, r4.x, o); r4.y += __shfl_xor_sync(0xffffffffu, r4.y, o);
+            r4.z += __shfl_xor_sync(0xffffffffu, r4.z, o); r4.w += __shfl_xor_sync(0xffffffffu, r4.w, o);
+        }
+        if (live && lane < LU) {
+            st4(&part[0][wr][4 * unit], w);
+            st4(&part[1][wr][4 * unit], r4);
         }
         __syncthreads();
         const float gt = s_g;
         if (warp == 0) {
             float4 u = make_float4(0.f, 0.f, 0.f, 0.f), o = u;
             if (lane < U) {
-                for (int i = 0; i < RG; ++i) {
-                    const float4 a = ld4(part + (size_t)i * P + 4 * lane), c = ld4(part + (size_t)(RG + i) * P + 4 * lane);
+                for (int i = 0; i < WR; ++i) {
+                    const float4 a = ld4(&part[0][i][4 * lane]), c = ld4(&part[1][i][4 * lane]);
                     u.x += a.x; u.y += a.y; u.z += a.z; u.w += a.w;
                     o.x += c.x; o.y += c.y; o.z += c.z; o.w += c.w;
                 }
-                const float4 v = ld4(row + (size_t)2 * G * D + (size_t)h * P + 4 * lane);
                 const float be = s_beta, qk = s_qk;
                 u.x = be * (v.x - gt * u.x); u.y = be * (v.y - gt * u.y); u.z = be * (v.z - gt * u.z); u.w = be * (v.w - gt * u.w);
                 o.x = gt * o.x + qk * u.x; o.y = gt * o.y + qk * u.y; o.z = gt * o.z + qk * u.z; o.w = gt * o.w + qk * u.w;
                 st4(su + 4 * lane, u);
             }
+            __syncwarp();
             const float inv = 1.f / sqrtf(warp_sum(dot4(o, o)) / (float)P + eps);
             if (lane < U) {
-                const float4 nw = ld4(norm + 4 * lane), z = Quad<TP>::load(prow + gate_col + (size_t)h * P + 4 * lane);
+                const float4 nw = ld4(norm + 4 * lane);
                 Quad<TP>::store(out + (size_t)(s0 + t) * H * P + (size_t)h * P + 4 * lane,
                                 make_float4(o.x * inv * nw.x * dl_silu(z.x), o.y * inv * nw.y * dl_silu(z.y),
                                             o.z * inv * nw.z * dl_silu(z.z), o.w * inv * nw.w * dl_silu(z.w)));
             }
         }
         __syncthreads();
-        const float4 u = ld4(su + 4 * unit);
+        const float4 u = live ? ld4(su + 4 * unit) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
         for (int i = 0; i < STEP_ROWS; ++i) {
             const int r = rg + RG * i;
-            if (live && r < D) {
+            if (r < D) {
                 const float kr = sk[r];
                 s[i].x = gt * s[i].x + kr * u.x; s[i].y = gt * s[i].y + kr * u.y;
                 s[i].z = gt * s[i].z + kr * u.z; s[i].w = gt * s[i].w + kr * u.w;
@@ -147,7 +166,7 @@ delta_step_kernel(const float* __restrict__ qkv, int C, const TP* __restrict__ p
 #pragma unroll
     for (int i = 0; i < STEP_ROWS; ++i) {
         const int r = rg + RG * i;
-        if (live && r < D) st4(S + (size_t)r * P, s[i]);
+        if (live && r < D) st4(S + r * P, s[i]);
     }
 }
 
@@ -159,15 +178,12 @@ extern "C" int vl_delta_step(const float* qkv, int C, const void* proj, int dtyp
     if (!delta_sizes_ok(H, G, D, P, C)) return VL_ERR_UNSUPPORTED;
     if (ld % 4 || gate_col % 4 || state_stride % 4 || (((uintptr_t)qkv | (uintptr_t)proj | (uintptr_t)state | (uintptr_t)out | (uintptr_t)norm) & 15))
         return VL_ERR_ARGUMENT;
-    const int U = P / 4;
-    int threads = U * ((D + STEP_ROWS - 1) / STEP_ROWS);          // enough row groups that a thread holds at most STEP_ROWS rows
-    threads = (threads + 31) / 32 * 32;
-    if (threads > 512) return VL_ERR_UNSUPPORTED;
-    const size_t smem = sizeof(float) * (size_t)2 * (threads / U) * P;
+    const StepShape sh = step_shape(D, P / 4);                    // (at most 16 warps, four rows of them)
     cudaStream_t s = (cudaStream_t)stream;
 #define DELTA_STEP(TP)                                                                                                              \
-    return vl_launch(delta_step_kernel<TP>, dim3(H, B), dim3(threads), smem, s, qkv, C, (const TP*)proj, ld, a_col, b_col, gate_col, \
-                     dt_bias, A_log, q_scale, unit_eps, norm, eps, state, state_stride, cu, slots, (TP*)out, H, G, D, P, longest)
+    return vl_launch(delta_step_kernel<TP>, dim3(H, B), dim3(32 * sh.UG * sh.WR), 0, s, qkv, C, (const TP*)proj, ld, a_col, b_col, gate_col, \
+                     dt_bias, A_log, q_scale, unit_eps, norm, eps, state, state_stride, cu, slots, (TP*)out, H, G, D, P, longest,  \
+                     sh.LU, sh.UG, sh.WR)
     if (dtype == VL_F32) DELTA_STEP(float);
     if (dtype == VL_BF16) DELTA_STEP(bf16);
 #undef DELTA_STEP

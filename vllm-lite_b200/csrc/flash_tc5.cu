@@ -1,5 +1,5 @@
 // bfloat16 attention of prompt portions over the paged cache on the 5th-generation tensor cores
-// (tcgen05.mma, accumulators in TMEM), compiled for one head size: -DFA_HD=64 or 128.
+// (tcgen05.mma, accumulators in TMEM), compiled for one head size: -DFA_HD=64, 128, 192 or 256.
 //
 // The function is that of csrc/attention.cu and csrc/flash_attn.cu: a query at absolute position p
 // of a request reads the keys lo..p of that request from its pages (lo = 0 or p - window + 1),
@@ -27,7 +27,8 @@
 //   warp 6, one thread   issues O += P_j V_j (M 128, N = head size, K 64; V is read as stored, i.e.
 //        with its N index contiguous) once P_j lies in shared memory.
 // Two blocks fit on an SM (112 KB of shared memory and 256 TMEM columns each at head size 128):
-// one block's softmax runs beside the other's products.
+// one block's softmax runs beside the other's products.  Heads of 192 and 256 (the cached rows of a latent attention) take
+// 160 to 208 KB and 512 columns: one block per SM, whose own two score buffers keep the tensor core ahead of the softmax.
 // A row keeps a stale maximum until the true one exceeds it by more than 8 (in log2 units): the
 // probabilities then reach 2^8 at most, and output and sum are scaled alike, so the quotient is the
 // same; the decision is taken row by row, so a row's result does not depend on its neighbours.
@@ -50,7 +51,8 @@ using namespace tc5;
 
 namespace {
 constexpr int HD = FA_HD;
-static_assert(HD == 64 || HD == 128, "this kernel is built for head sizes 64 and 128");
+static_assert(HD == 64 || HD == 128 || HD == 192 || HD == 256, "this kernel is built for head sizes of 64, 128, 192 and 256");
+constexpr int BLOCKS_PER_SM = HD <= 128 ? 2 : 1;
 constexpr int BM = 128, BN = 64, CB = HD / 64;       // CB: blocks of 64 columns (one swizzled row) per head
 constexpr int NTHREADS = 224;
 constexpr unsigned ROW_BYTES = 128;
@@ -59,7 +61,7 @@ constexpr unsigned KV_STAGE = BN * HD * 2;           // CB blocks of [64 rows][1
 constexpr unsigned P_BYTES = BM * BN * 2;            // [128 rows][128 bytes]
 constexpr unsigned TILE_BYTES = Q_BYTES + 4 * KV_STAGE + P_BYTES;
 constexpr unsigned SMEM_BYTES = TILE_BYTES + 160;    // + barriers; two blocks per SM only without any slack
-constexpr unsigned TMEM_COLS = 256;                  // scores 2 x 64, output HD (a power of two >= their sum)
+constexpr unsigned TMEM_COLS = HD <= 128 ? 256 : 512;   // scores 2 x 64, output HD (a power of two >= their sum)
 constexpr unsigned O_COL = 2 * BN;
 constexpr float RESCALE_ABOVE = 8.0f;
 
@@ -121,7 +123,7 @@ __device__ __forceinline__ unsigned swizzled(int row, int chunk) {
 // tiles[i] = {row of the block table, index of the tile's first token in the step, tokens (<= 128),
 // position of the first}
 template <bool SIG, bool SHAPED>
-__global__ void __launch_bounds__(NTHREADS, 2)
+__global__ void __launch_bounds__(NTHREADS, BLOCKS_PER_SM)
 flash_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                  const __grid_constant__ CUtensorMap pages_k, const __grid_constant__ CUtensorMap pages_v, int use_pages,
                  const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out,

@@ -299,7 +299,8 @@ static int launch_mma_kernel(dim3 grid, cudaStream_t s, int K, Args... args) {
 template <typename TC>
 __global__ void __launch_bounds__(256)
 gemm_batched_bf16_wide_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W, TC* __restrict__ C, int M, int N, int K,
-                              int lda, int ldw, int ldc, long long a_bs, long long w_bs, long long c_bs, int nst) {
+                              int lda, int ldw, int ldc, long long a_bs, long long w_bs, long long c_bs,
+                              const bf16* __restrict__ gate, int gate_ld, int nst) {
     extern __shared__ __align__(16) unsigned char gw_smem[];
     bf16 (*As)[GW_BM][GM_LDS] = reinterpret_cast<bf16 (*)[GW_BM][GM_LDS]>(gw_smem);
     bf16 (*Ws)[GW_BN][GM_LDS] = reinterpret_cast<bf16 (*)[GW_BN][GM_LDS]>(gw_smem + (size_t)nst * GW_BM * GM_LDS * sizeof(bf16));
@@ -364,11 +365,12 @@ gemm_batched_bf16_wide_kernel(const bf16* __restrict__ A, const bf16* __restrict
         for (int half = 0; half < 2; ++half) {
             const int m = m0 + wm * 32 + i * 16 + g + half * 8;
             if (m >= M) continue;
+            const float open = gate ? gb_sigmoid(to_f32(gate[(size_t)m * gate_ld + blockIdx.z])) : 1.f;
             TC* crow = Cb + (size_t)m * ldc;
 #pragma unroll
             for (int nt = 0; nt < 8; ++nt) {
                 const int n = n0 + wn * 64 + nt * 8 + t2;
-                const float v0 = acc[i][nt][2 * half], v1 = acc[i][nt][2 * half + 1];
+                const float v0 = acc[i][nt][2 * half] * open, v1 = acc[i][nt][2 * half + 1] * open;
                 if (even && n + 1 < N) {
                     if (sizeof(TC) == 4) {
                         *reinterpret_cast<float2*>(crow + n) = make_float2(v0, v1);
@@ -386,7 +388,7 @@ gemm_batched_bf16_wide_kernel(const bf16* __restrict__ A, const bf16* __restrict
 #define GW_MIN_ROWS 512
 template <typename TC>
 static int launch_batched_wide(const bf16* A, const bf16* W, TC* C, int M, int N, int K, int lda, int ldw, int ldc, long long a_bs,
-                               long long w_bs, long long c_bs, int batch, cudaStream_t s) {
+                               long long w_bs, long long c_bs, int batch, const bf16* gate, int gate_ld, cudaStream_t s) {
     const dim3 grid((N + GW_BN - 1) / GW_BN, (M + GW_BM - 1) / GW_BM, batch);
     const int KT = (K + GM_BK - 1) / GM_BK, nst = KT < 2 ? 2 : (KT > GW_NST ? GW_NST : KT);
     const size_t stage = (size_t)(GW_BM + GW_BN) * GM_LDS * sizeof(bf16);
@@ -396,7 +398,8 @@ static int launch_batched_wide(const bf16* A, const bf16* W, TC* C, int M, int N
         if (e != cudaSuccess) return (int)e;
         ready = true;
     }
-    return vl_launch(gemm_batched_bf16_wide_kernel<TC>, grid, dim3(256), nst * stage, s, A, W, C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, nst);
+    return vl_launch(gemm_batched_bf16_wide_kernel<TC>, grid, dim3(256), nst * stage, s, A, W, C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, gate,
+                     gate_ld, nst);
 }
 
 static bool gm_aligned(const void* A, const void* W, int K, int lda, int ldw, long long a_bs, long long w_bs, long long w_gs) {
@@ -447,7 +450,7 @@ extern "C" int vl_gemm_batched_nt(const void* A, const void* W, void* C, int dty
     if (dtype == VL_BF16 && c_dtype == VL_F32) {
         if (!tile_group && M >= GW_MIN_ROWS && N >= 96 && (M + GW_BM - 1) / GW_BM <= 65535 && batch <= 65535 &&
             gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
-            return launch_batched_wide((const bf16*)A, (const bf16*)W, (float*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, batch, s);
+            return launch_batched_wide((const bf16*)A, (const bf16*)W, (float*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, batch, nullptr, 0, s);
         if (gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
             return launch_batched_mma((const bf16*)A, (const bf16*)W, (float*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs,
                                       batch, tile_group, w_gs, bm, nullptr, 1, nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f, nullptr, 0, s);
@@ -455,6 +458,10 @@ extern "C" int vl_gemm_batched_nt(const void* A, const void* W, void* C, int dty
                                            a_bs, w_bs, c_bs, batch, tile_group, w_gs, bm, nullptr, 0, s);
     }
     if (dtype == VL_BF16) {
+        if (!tile_group && M >= GW_MIN_ROWS && N >= 96 && (M + GW_BM - 1) / GW_BM <= 65535 && batch <= 65535 &&
+            gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
+            return launch_batched_wide((const bf16*)A, (const bf16*)W, (bf16*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs, batch,
+                                       (const bf16*)gate, gate_ld, s);
         if (gm_aligned(A, W, K, lda, ldw, a_bs, w_bs, w_gs) && !vl_batched_simt_only())
             return launch_batched_mma((const bf16*)A, (const bf16*)W, (bf16*)C, M, N, K, lda, ldw, ldc, a_bs, w_bs, c_bs,
                                       batch, tile_group, w_gs, bm, nullptr, 1, nullptr, GM_ACT_NONE, 0.f, 0.f, 0.f, (const bf16*)gate, gate_ld, s);

@@ -683,10 +683,15 @@ FLASH_TC5_TILE = 128
 
 
 def flash_tc5_supported(dtype, head_dim, page_size) -> bool:
-    """The tcgen05 attention kernel takes bfloat16, head sizes 64 and 128, and pages of a multiple of
+    """The attention kernels that bring their tiles by TMA take bfloat16, head sizes 64 and 128, and pages of a multiple of
     8 positions that divide 64 or are a multiple of it."""
     return (dtype == torch.bfloat16 and head_dim in (64, 128) and page_size % 8 == 0
             and (64 % page_size == 0 if page_size < 64 else page_size % 64 == 0))
+
+
+def flash_prefill_tc5_supported(dtype, head_dim, page_size) -> bool:
+    """The tcgen05 kernel of prompt portions also takes heads of 192 and 256 (one block per SM instead of two)."""
+    return flash_tc5_supported(dtype, 64 if head_dim in (192, 256) else head_dim, page_size)
 
 
 def flash_prefill_tc5(qkv, out, k_cache, v_cache, block_table, tiles, num_heads, num_kv_heads, head_dim, scale, window, err,
@@ -703,7 +708,7 @@ def flash_prefill_tc5(qkv, out, k_cache, v_cache, block_table, tiles, num_heads,
     mode, mask_chunk, gate_stride = _check_variant(qkv, num_heads, weighting, mask_chunk, head_bias, gate, sinks)
     if out.shape != (qkv.shape[0], num_heads * head_dim) or tiles.shape[1] != 4:
         raise KernelError("flash_prefill_tc5: shapes disagree")
-    if not flash_tc5_supported(qkv.dtype, head_dim, k_cache.shape[2]):
+    if not flash_prefill_tc5_supported(qkv.dtype, head_dim, k_cache.shape[2]):
         raise KernelError(f"flash_prefill_tc5: head size {head_dim} / page size {k_cache.shape[2]} not taken")
     _check(_fn("flash_tc5", "vl_flash_prefill_tc5", {"FA_HD": head_dim})(
         _ptr(qkv), qkv.shape[1], _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1],

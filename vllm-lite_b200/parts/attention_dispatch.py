@@ -112,7 +112,7 @@ def run(qkv, out, cache, group, step, spec, scale, fold=None, sinks=None, weight
         if step.query_tiles is not None:
             tile_args = (qkv, out, cache.k, cache.v, group.block_table, step.query_tiles,
                          spec.num_heads, spec.num_kv_heads, spec.head_dim, scale, spec.window, step.err)
-            if step.max_query_len > 64 and ops.flash_tc5_supported(qkv.dtype, spec.head_dim, group.page_size):
+            if step.max_query_len > 64 and ops.flash_prefill_tc5_supported(qkv.dtype, spec.head_dim, group.page_size):
                 ops.flash_prefill_tc5(*tile_args, sinks=sinks)
             else:
                 ops.flash_prefill(*tile_args, tile_rows=QUERY_TILE, sinks=sinks)
@@ -138,7 +138,7 @@ def _run_variant(ops, q, out, cache, group, step, spec, scale, weighting, chunk,
                 ops, spec, step.single_tokens.shape[0], step.single_context, chunk)):
             tile_args = (q, out, cache.k, cache.v, group.block_table, step.query_tiles, spec.num_heads, spec.num_kv_heads,
                          spec.head_dim, scale, spec.window, step.err)
-            if step.max_query_len > 64 and ops.flash_tc5_supported(q.dtype, spec.head_dim, group.page_size):
+            if step.max_query_len > 64 and ops.flash_prefill_tc5_supported(q.dtype, spec.head_dim, group.page_size):
                 ops.flash_prefill_tc5(*tile_args, sinks=sinks, **variant)
             else:
                 ops.flash_prefill(*tile_args, tile_rows=QUERY_TILE, sinks=sinks, **variant)
@@ -174,7 +174,7 @@ def _run_shaped(ops, q, out, cache, group, step, spec, scale, sinks, weighting, 
         if step.query_tiles is not None:
             tile_args = (q, out, cache.k, cache.v, group.block_table, step.query_tiles, spec.num_heads, spec.num_kv_heads,
                          spec.head_dim, scale, spec.window, step.err)
-            if step.max_query_len > 64 and ops.flash_tc5_supported(q.dtype, spec.head_dim, group.page_size):
+            if step.max_query_len > 64 and ops.flash_prefill_tc5_supported(q.dtype, spec.head_dim, group.page_size):
                 ops.flash_prefill_tc5(*tile_args, sinks=sinks, **shape)
             else:
                 ops.flash_prefill(*tile_args, tile_rows=QUERY_TILE, sinks=sinks, **shape)
