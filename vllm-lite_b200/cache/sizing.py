@@ -63,7 +63,8 @@ def _mixer_width(mixer) -> int:
         # latent attention: both latents (and the rotated key part), the queries, their absorbed form and the context
         # (heads x cached row, the row rounded up to 16), the expanded values, the output gate
         rot = getattr(mixer, "rot_dim", 0)
-        row = -(-(mixer.kv_rank + rot) // 16) * 16
+        step = 16 if mixer.kv_rank + rot <= 256 else 64
+        row = -(-(mixer.kv_rank + rot) // step) * step
         gate = mixer.num_heads * mixer.vdim if getattr(mixer, "gate", None) else 0
         gate += mixer.num_heads if getattr(mixer, "head_gate", None) else 0
         return mixer.q_rank + mixer.kv_rank + rot + gate + 7 + mixer.num_heads * (mixer.dim + rot + 2 * row + mixer.vdim)

@@ -22,12 +22,13 @@
 // softmax of its own; the 16 partial results are merged in group order.  Which
 // keys a group sees and the order of every sum depend on positions alone, so a
 // token's output does not depend on how the batch was cut.
-// head_dim: multiples of 16 up to 256.
+// head_dim: multiples of 16 up to 256; the kernel of one token and head also multiples of 64 up to 576.
 #include "common.cuh"
 
 #define ATT_THREADS 128
 #define ATT_GROUPS 16
 #define ATT_MAX_HD 256
+#define ATT_MAX_WIDE_HD 576          // vl_paged_attention alone, in steps of 64 from 256 on (wide latent rows)
 
 template <typename T> struct Pair;
 template <> struct Pair<float> {
@@ -194,6 +195,7 @@ static int launch_paged_attention(int R, dim3 grid, cudaStream_t s, const T* q, 
     switch (R) {
         ATT_CASE(1) ATT_CASE(2) ATT_CASE(3) ATT_CASE(4) ATT_CASE(5) ATT_CASE(6) ATT_CASE(7) ATT_CASE(8)
         ATT_CASE(9) ATT_CASE(10) ATT_CASE(11) ATT_CASE(12) ATT_CASE(13) ATT_CASE(14) ATT_CASE(15) ATT_CASE(16)
+        ATT_CASE(20) ATT_CASE(24) ATT_CASE(28) ATT_CASE(32) ATT_CASE(36)
         default: return VL_ERR_UNSUPPORTED;
     }
 #undef ATT_CASE
@@ -211,7 +213,7 @@ extern "C" int vl_paged_attention(const void* q, int q_stride, void* out, int dt
     if (T <= 0) return VL_OK;
     if (keep < 0 || (keep > 0 && chunk > 0)) return VL_ERR_ARGUMENT;
     if ((dist_a == nullptr) != (dist_b == nullptr) || softcap < 0.f) return VL_ERR_ARGUMENT;
-    if (hd <= 0 || hd % 16 || hd > ATT_MAX_HD) return VL_ERR_UNSUPPORTED;
+    if (hd <= 0 || hd % 16 || hd > ATT_MAX_WIDE_HD || (hd > ATT_MAX_HD && hd % 64)) return VL_ERR_UNSUPPORTED;
     if (nq <= 0 || nkv <= 0 || nq % nkv || page_size <= 0 || max_blocks <= 0) return VL_ERR_ARGUMENT;
     if ((mode != ATT_SOFTMAX && mode != ATT_SIGMOID) || chunk < 0 || (mode == ATT_SIGMOID && sinks)) return VL_ERR_ARGUMENT;
     if (gate && gate_stride < nq) return VL_ERR_ARGUMENT;

@@ -42,7 +42,8 @@ from .linear import Linear, stacked
 from .registry import MIXERS
 from .spec import LatentAttentionSpec, TensorDecl
 
-MAX_LATENT = 256            # widest cached row the attention kernels take
+FAST_LATENT = 256           # widest cached row the tensor-core attention kernels take
+MAX_LATENT = 576            # widest one any kernel takes (csrc/attention.cu: a token and head a block)
 
 # what the attention dispatcher reads of a mixer's description
 # (shared_row: keys and values are the same rows of one shared head, which the choice of the decode chunks may use)
@@ -50,7 +51,9 @@ HeadLayout = namedtuple("HeadLayout", "num_heads num_kv_heads head_dim window sh
 
 
 def padded_rank(kv_rank: int) -> int:
-    return -(-kv_rank // 16) * 16
+    """The cached row's width: a multiple of 16, beyond FAST_LATENT of 64."""
+    step = 16 if kv_rank <= FAST_LATENT else 64
+    return -(-kv_rank // step) * step
 
 
 def check_latent_sizes(spec: LatentAttentionSpec):
