@@ -554,6 +554,14 @@ LATENT = [("one", 3, 10, 14, 24, 18, None, 8), ("one", 8, 32, 48, 96, 128, None,
           ("two", 6, 12, 20, 0, 224, rot(32, 2000.0, (8.0, 40, 4.0, 1.0)), 64), ("two", 3, 20, 12, 0, 300, rot(20, 500.0, (4.0, 300, 16.0, 2.0)), 16)]
 
 
+def score_scale(spread, dim, q_rank, kv_rank, r, W):
+    """The scale that gives scores of about this standard deviation, for inputs of variance 1 and weights of 0.2."""
+    var = dim * 0.2 ** 4 * (q_rank or W) * kv_rank
+    if r is not None:
+        var += r["dims"] * (0.2 ** 2 * W * P.magnitude(r) ** 2) ** 2
+    return spread / math.sqrt(var)
+
+
 def latent_part(kind, heads, dim, vdim, q_rank, kv_rank, r, W, dtype, scale, seed, edit=None):
     from vllm_lite_b200.config.vekusun import VekusunLayer, _mixer, _rotation
     m = dict(heads=heads, dim=dim, vdim=vdim, kv_rank=kv_rank, scale=scale)
@@ -573,49 +581,46 @@ def latent_part(kind, heads, dim, vdim, q_rank, kv_rank, r, W, dtype, scale, see
 @pytest.mark.parametrize("kind,heads,dim,vdim,q_rank,kv_rank,r,page", LATENT)
 def test_latent_attention_in_portions(dtype, kind, heads, dim, vdim, q_rank, kv_rank, r, page):
     """Whole mixers over shuffled pages, portions and single tokens mixed; scores sharp enough that for most queries one key, as
-    often as not hundreds of positions back, takes most of the weight."""
+    often as not hundreds of positions back, takes most of the weight; sinks from nothing to most of the denominator."""
     W = 64
-    sharp = 5.0 / math.sqrt(dim + (r["dims"] if r else 0))
+    spread = 6.0 if dtype == torch.float32 else 3.0            # bfloat16 rounds scores in proportion to their size
 
-    def strong(t):
-        for n in ("uq", "q", "uk"):
-            if n in t:
-                t[n] = (t[n].float() * 2.0).to(dtype)
+    def sinks(t):
         if "sink" in t:
             t["sink"] = torch.linspace(-2.0, 6.0, heads).to(dtype)
 
-    part, tensors, plain = latent_part(kind, heads, dim, vdim, q_rank, kv_rank, r, W, dtype, sharp, 81, strong)
+    part, tensors, plain = latent_part(kind, heads, dim, vdim, q_rank, kv_rank, r, W, dtype,
+                                       score_scale(spread, dim, q_rank, kv_rank, r, W), 81, sinks)
     pages = Pages(part.rank, page, 2, max(TOTAL), dtype)
     h = [rand((TOTAL[b], W), 82 + b, dtype) for b in (0, 1)]
     got = in_portions(part, h, CUTS, dtype, pages=pages)
     for b in (0, 1):
-        # sharp scores magnify the rounding of the latent rows and queries in bfloat16
-        close(got[b], plain(h[b]), dtype, f"{kind} of request {b}", tol=4e-5 if dtype == torch.float32 else 9e-2)
+        close(got[b], plain(h[b]), dtype, f"{kind} of request {b}", tol=4e-5 if dtype == torch.float32 else 6e-2)
 
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("case", [0, 1, 3, 5, 6, 9, 10])
 def test_one_far_key_among_hundreds(dtype, case):
-    """One token far back whose latent points where the last queries look: without it (its row replaced) the output is another;
-    the engine's has it, in a long portion and in single tokens, also at the first position and at pages' borders."""
+    """Every key but one the same: with another token in that one place the outputs of queries hundreds of positions on are
+    others, and the engine's are the right ones, in a long portion and in single tokens, at the first position and at pages' borders."""
     kind, heads, dim, vdim, q_rank, kv_rank, r, page = LATENT[case]
     W, n = 64, 340
-    part, tensors, plain = latent_part(kind, heads, dim, vdim, q_rank, kv_rank, r, W, dtype, 1.0, 91)
+    part, tensors, plain = latent_part(kind, heads, dim, vdim, q_rank, kv_rank, r, W, dtype,
+                                       score_scale(4.0 if dtype == torch.float32 else 2.5, dim, q_rank, kv_rank, r, W), 91)
     base = rand((n, W), 92, torch.float32)
     for far in (0, page - 1, page, 64, 129):
         h = base.clone()
         h[far] = 3.0 * rand((W,), 93)
-        # queries from position 200 on look for it: ask the plain implementation which scale makes it stand out
         h = h.to(dtype)
         without = h.clone()
         without[far] = base[(far + 7) % n].to(dtype)
         want, other = plain(h), plain(without)
         moved = (want - other).abs().amax(-1)[200:]
-        assert float(moved.max()) > 0.02 * float(want.abs().max())
+        assert float(moved.max()) > 0.01 * float(want.abs().max())
         pages = Pages(part.rank, page, 1, n, dtype, seed=far)
         got = in_portions(part, [h], ([200], [100], [1], [39]), dtype, pages=pages)
-        close(got[0], want, dtype, f"far key {far}", tol=4e-5 if dtype == torch.float32 else 4e-2)
+        close(got[0], want, dtype, f"far key {far}", tol=4e-5 if dtype == torch.float32 else 6e-2)
         if dtype == torch.float32:
             assert float((got[0].double().cpu() - other).abs().max()) > 100 * float((got[0].double().cpu() - want).abs().max())
 
