@@ -27,6 +27,7 @@
 #define VL_DEV_IN_GEMM_TC5_PAIR 0x800u
 #define VL_DEV_IN_FLASH_TC5 0x1000u
 #define VL_DEV_IN_FLASH_DECODE_TMA 0x2000u
+#define VL_DEV_IN_DELTA 0x4000u
 // ... and, in the two tcgen05 products, which waits gave up in the block (shifted left by 16):
 // 1 a free stage (copying thread), 2 a free accumulator, 4 a filled stage (both: issuing thread),
 // 8 a complete accumulator (epilogue)

@@ -155,7 +155,7 @@ _SIGNATURES = {
                                      c_int, c_int, c_void_p],
     ("delta", "vl_delta_step"): [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
                                  c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
-                                 c_int, c_int, c_void_p],
+                                 c_int, c_int, c_int, c_void_p, c_void_p],
     ("delta", "vl_delta_chunks"): [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
                                    c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
                                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -1663,7 +1663,7 @@ def _head_delta_args(qkv, proj, a_col, b_col, gate_col, dt_bias, A_log, norm, st
     return B, sp, stride
 
 
-def delta_step(qkv, proj, a_col, b_col, gate_col, dt_bias, A_log, q_scale, unit_eps, norm, eps, state, state_off, cu, slots, out, H, G, D, P):
+def delta_step(qkv, proj, a_col, b_col, gate_col, dt_bias, A_log, q_scale, unit_eps, norm, eps, state, state_off, cu, slots, out, H, G, D, P, err=None):
     """out [T, H P] = rms_head(o) * norm * silu(gate) of the delta rule with one decay per head, for the requests of the step that
     bring fewer than DELTA_MIN_CHUNK tokens (the others' rows and states are left alone).  qkv: what the convolution leaves;
     raw decays, raw betas and the gate are columns of `proj`."""
@@ -1671,7 +1671,7 @@ def delta_step(qkv, proj, a_col, b_col, gate_col, dt_bias, A_log, q_scale, unit_
     _check(_fn("delta", "vl_delta_step")(
         _ptr(qkv), qkv.shape[1], _ptr(proj), dtype_code(proj.dtype), proj.shape[1], int(a_col), int(b_col), int(gate_col), _ptr(dt_bias),
         _ptr(A_log), float(q_scale), float(unit_eps), _ptr(norm), float(eps), sp, stride, _ptr(cu), _ptr(slots), B, _ptr(out), H, G, D, P,
-        DELTA_MIN_CHUNK - 1, _stream()), "vl_delta_step")
+        DELTA_MIN_CHUNK - 1, 2 * sm_pairs(), _ptr(err), _stream()), "vl_delta_step")
     return out
 
 

@@ -248,7 +248,7 @@ class HeadDelta:
                 scratch = ws.get(tag + "hd.chunks", (ops.delta_chunk_floats(chunks, H, D, P),), torch.float32)
                 ops.delta_chunks(*args, chunks, scratch, ws.get(tag + "hd.u", (T, H * P), torch.float32), gated, H, G, D, P)
             if step.max_query_len < ops.DELTA_MIN_CHUNK or B > 1:
-                ops.delta_step(*args, gated, H, G, D, P)
+                ops.delta_step(*args, gated, H, G, D, P, err=step.err)
             return self.o_proj(gated, step, "hd.out")
         o = ws.get(tag + "hd.o", (T, H * P), torch.float32)
         ops.delta_scan(qkv, proj, a_col, self.dt_bias, self.a_log, proj, b_col, D ** -0.5, s.unit_eps, cache.state,
