@@ -600,6 +600,56 @@ def test_latent_attention_in_portions(dtype, kind, heads, dim, vdim, q_rank, kv_
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("q_rank,kv_rank,rot_dim,dims,heads,dim", [(2048, 64, 0, 0, 0, 0), (1024, 512, 64, 64, 0, 0), (72, 40, 24, 16, 0, 0), (0, 96, 32, 32, 5, 24),
+                                                                   (0, 200, 16, 16, 3, 8), (0, 24, 40, 16, 2, 16), (0, 18, 6, 4, 3, 10)])
+def test_norm_rotation_and_cache_row_of_a_token(dtype, q_rank, kv_rank, rot_dim, dims, heads, dim):
+    """Both forms of the kernel (eight numbers a thread, one): the query latent or the finished query heads before the key and value
+    latent, the rotated key part behind it (only its first features turned), sine and cosine with a factor, zeros behind."""
+    pos, page, amp = [0, 1, 7, 130, 1000], 4, 1.25
+    T, kv_col = len(pos), q_rank or heads * (dim + rot_dim)
+    width = -(-(kv_rank + rot_dim) // 16) * 16 + 16
+    ld = -(-(kv_col + kv_rank + rot_dim + 3) // 8) * 8
+    proj = rand((T, ld), 100, dtype, 1.5)
+    wq, wkv = rand((max(q_rank, 1),), 101) + 1, rand((kv_rank,), 102) + 1
+    r = rot(dims, 300.0) if dims else None
+    inv = torch.tensor(P.frequencies(r), dtype=torch.float32, device=DEV) if dims else None
+    cache = torch.full((2, 1, page, width), 9.0, dtype=dtype, device=DEV)
+    slots = [6, 1, 4, -1, 7]
+    cq = torch.empty((T, q_rank), dtype=dtype, device=DEV) if q_rank else None
+    e = torch.zeros(1, dtype=torch.int32, device=DEV)
+    p64 = proj.double().cpu()
+    ops().latent_norm_write(proj, q_rank, kv_rank, wq if q_rank else None, wkv, 1e-5, cq, ints(slots), cache, e, rot_dim=rot_dim,
+                            rotary=(inv, dims, amp) if dims else None, positions=ints(pos), kv_col=kv_col,
+                            q_heads=(dim, dim + rot_dim, heads) if heads else None)
+    assert int(e.item()) == 0
+
+    def turned(x):                                  # pairs i, i + dims / 2
+        a = torch.tensor(pos, dtype=torch.float64)[:, None] * torch.tensor(P.frequencies(r))
+        c, s, h = (amp * torch.cos(a)).view(T, *[1] * (x.dim() - 2), -1), (amp * torch.sin(a)).view(T, *[1] * (x.dim() - 2), -1), dims // 2
+        return torch.cat([x[..., :h] * c - x[..., h:dims] * s, x[..., h:dims] * c + x[..., :h] * s, x[..., dims:]], -1)
+
+    tol = 2e-5 if dtype == torch.float32 else 1e-2
+    if q_rank:
+        close(cq, P.rms_norm(p64[:, :q_rank], wq.cpu(), 1e-5), dtype, "query latent", tol=tol)
+    if heads:
+        q = p64[:, :kv_col].reshape(T, heads, dim + rot_dim)
+        want = torch.cat([q[..., :dim], turned(q[..., dim:])], -1).reshape(T, kv_col)
+        close(proj[:, :kv_col], want, dtype, "query heads", tol=10 * tol)
+    want = P.rms_norm(p64[:, kv_col:kv_col + kv_rank], wkv.cpu(), 1e-5)
+    key = p64[:, kv_col + kv_rank:kv_col + kv_rank + rot_dim]
+    for t, s in enumerate(slots):
+        if s < 0:
+            continue
+        row = cache[s // page, 0, s % page]
+        close(row[:kv_rank], want[t], dtype, "cached latent", tol=tol)
+        if rot_dim:
+            close(row[kv_rank:kv_rank + rot_dim], turned(key)[t], dtype, "cached key part", tol=10 * tol)
+        assert float(row[kv_rank + rot_dim:].abs().max()) == 0.0
+    assert float(cache[0, 0, 3, 0]) == 9.0                           # slot 3 belongs to nobody
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("case", [0, 1, 3, 5, 6, 9, 10])
 def test_one_far_key_among_hundreds(dtype, case):
     """Every key but one the same: with another token in that one place the outputs of queries hundreds of positions on are
