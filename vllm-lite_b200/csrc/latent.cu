@@ -227,14 +227,16 @@ extern "C" int vl_latent_norm_write(void* proj, int dtype, int ld, int T, int q_
         return VL_ERR_ARGUMENT;
     if (rot / 2 > LATENT_MAX_PAIRS) return VL_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-    const bool vec = ((ld | q_rank | kv_col | kv_rank | row_width | rot_dim | (rot / 2) | (q_heads > 0 ? q_col | q_stride : 0)) & 7) == 0 &&
+    // (float32 steps keep the one form whose sums do not depend on such boundaries)
+    const bool vec = dtype == VL_BF16 && ((ld | q_rank | kv_col | kv_rank | row_width | rot_dim | (rot / 2) | (q_heads > 0 ? q_col | q_stride : 0)) & 7) == 0 &&
                      kv_rank <= 1024 && (((uintptr_t)proj | (uintptr_t)cq_out | (uintptr_t)cache) & 15) == 0;
-#define LATENT_WRITE(TT)                                                                                                             \
-    return vl_launch(vec ? latent_norm_write_vec_kernel<TT> : latent_norm_write_kernel<TT>, dim3(T), dim3(128), 0, s, (TT*)proj, ld, q_rank, kv_col, kv_rank, wq, wkv, eps,   \
+#define LATENT_WRITE(KERNEL, TT)                                                                                                             \
+    return vl_launch(KERNEL<TT>, dim3(T), dim3(128), 0, s, (TT*)proj, ld, q_rank, kv_col, kv_rank, wq, wkv, eps,   \
                      (TT*)cq_out, slots, (TT*)cache, row_width, num_slots, rot_dim, rot, inv_freq, amp, q_col, q_stride, q_heads,    \
                      positions, err)
-    if (dtype == VL_F32) LATENT_WRITE(float);
-    if (dtype == VL_BF16) LATENT_WRITE(bf16);
+    if (dtype == VL_F32) LATENT_WRITE(latent_norm_write_kernel, float);
+    if (vec) LATENT_WRITE(latent_norm_write_vec_kernel, bf16);
+    if (dtype == VL_BF16) LATENT_WRITE(latent_norm_write_kernel, bf16);
 #undef LATENT_WRITE
     return VL_ERR_UNSUPPORTED;
 }
